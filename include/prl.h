@@ -681,6 +681,24 @@ int prl_sublayer_close(const float* y0, int64_t ld0, int32_t n_split0, const flo
                        int64_t ld1, int32_t n_split1, const float* gain1, float s1, const float* post_gain,
                        const float* bias, int32_t add, const float* next_gain, float eps, int32_t n, int32_t W, float* x,
                        void* xa, int32_t f32, prl_stream_t stream);
+/* x += sum y0 slices + sum y1 choices (y1 [top][n][W] or NULL; where sel >= experts the slice is wsel * xa instead);
+ * xa = T(norm_next(x)): the close of a layer whose mixer and routed feed-forward read one normed input */
+int prl_joint_close(const float* y0, int32_t n_split0, const float* y1, int32_t top, const int32_t* sel, const float* wsel,
+                    int32_t experts, const float* next_gain, float eps, int32_t n, int32_t W, float* x, void* xa, int32_t f32,
+                    prl_stream_t stream);
+/* out[n][F] = T(act): act 0 relu(P[off + c])^2, act 1 gelu_tanh(P[off + c]) * P[off + F + c]; off_gate >= 0: times
+ * sigmoid(P[off_gate]) */
+int prl_ff_act(const float* P, int64_t ld, int32_t off, int32_t n, int32_t F, int32_t act, int32_t off_gate, void* out,
+               int32_t f32, prl_stream_t stream);
+/* C = A1 B1^T + A2 B2^T in one accumulation (two branches of one residual): many rows, and the token step's split-K form */
+int prl_gemm_tn_dual(const void* A1_bf16, const void* B1_bf16, int64_t K1, const void* A2_bf16, const void* B2_bf16, int64_t K2,
+                     int64_t M, int64_t N, float* C, int64_t ldc, prl_stream_t stream);
+int prl_gemm_dual_split_k(int64_t M, int64_t N, int64_t K1, int64_t K2);
+int prl_gemm_bf16_dual(const void* W1, const void* X1, int64_t K1, const void* W2, const void* X2, int64_t K2, int64_t M,
+                       int64_t N, int32_t split_k, float* partials, prl_stream_t stream);
+/* gate_up GEMM with gelu(gate) * up (tanh form) in its epilogue */
+int prl_gemm_geglu_f32(const void* X_bf16, int64_t ldx, const void* W_gate_up_bf16, int64_t ldw, int64_t M, int64_t I, int64_t K,
+                       void* act_bf16, int64_t ld_act, prl_stream_t stream);
 /* attention front end with per-head unit norms (biases and gains nullable); off_v < 0: the value is the key as
  * projected (with its bias, before its norm) */
 int prl_qk_headnorm_cache(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, int32_t off_v, int32_t n, int32_t H,
@@ -737,6 +755,16 @@ int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is
 int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
                  int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
                  int64_t max_tiles, int64_t N, int64_t K, float* C, int64_t ldc, int32_t c_perm, prl_stream_t stream);
+/* choice from ready logits: outputs ranked by softmax share + correction (nullable) inside the `keep` best of `groups`
+ * equal groups, weighted by the share alone; outputs experts .. outputs - 1 hand the input through (no rows) */
+int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
+                   int32_t top, int32_t groups, int32_t keep, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta,
+                   int32_t* tiles, prl_stream_t stream);
+/* prl_moe_gemm with act[s] = relu(product)^2 * wsel[pair] written in sorted order in A's type (the second product's operand) */
+int prl_moe_gemm_relu2(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                       int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
+                       int64_t max_tiles, int64_t N, int64_t K, const float* wsel, void* act, int64_t ld_act,
+                       prl_stream_t stream);
 int prl_moe_glu(const float* gate_up, int64_t ld, int64_t pairs, int32_t F, const int32_t* perm, const float* wsel,
                 float limit, float beta, void* out, int32_t f32, prl_stream_t stream);
 

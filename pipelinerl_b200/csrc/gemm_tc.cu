@@ -137,6 +137,9 @@ struct GemmParams {
   // gated activation of the epilogue: glu_limit == 0: SiLU(gate) * up; glu_limit > 0: the clamped form of the hybrid decoders,
   // g = min(gate, limit), u = clamp(up, +-limit), act = g * sigmoid(glu_beta * g) * (u + 1)
   float glu_limit, glu_beta;
+  // two products in one accumulation (split_k, no lo part): k-blocks >= dual_kb are k-blocks (kb - dual_kb) of a second
+  // weight (the map in the lo weight's place) and a second activation.  0 = off
+  int dual_kb;
 };
 
 template <int kNTile>
@@ -153,7 +156,8 @@ struct SmemLayout {
 template <int kNTile, bool kHead>
 __global__ void __launch_bounds__(kThreads, 2)
 gemm_swapab_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_wlo,
-                   const __grid_constant__ CUtensorMap tm_x, GemmParams p, int n_stages) {
+                   const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_x2, GemmParams p,
+                   int n_stages) {
   using L = SmemLayout<kNTile>;
   extern __shared__ uint8_t smem_raw[];
   pdl_launch_dependents();  // let the next kernel start its own prologue / weight prefetch as early as possible
@@ -197,7 +201,9 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
       const int kcoord = (kb_begin + i) * kBlockK;
       const int wc0 = p.tiled ? 0 : kcoord;
       const int wc1 = p.tiled ? (n_tile * p.kblocks + kb_begin + i) * kBlockM : n0;
-      if (p.swiglu_I) {   // tm_w boxes are 64 rows here: gate half, then up half of the same 64 features
+      if (p.dual_kb && kb_begin + i >= p.dual_kb) {
+        ptx::tma_load_2d(a_dst, &tm_wlo, kcoord - p.dual_kb * kBlockK, n0, full_bar(i), ptx::kEvictFirst);
+      } else if (p.swiglu_I) {   // tm_w boxes are 64 rows here: gate half, then up half of the same 64 features
         ptx::tma_load_2d(a_dst, &tm_w, wc0, n_tile * 64, full_bar(i), ptx::kEvictFirst);
         ptx::tma_load_2d(a_dst + L::kABytes / 2, &tm_w, wc0, (int)p.swiglu_I + n_tile * 64, full_bar(i), ptx::kEvictFirst);
       } else {
@@ -224,7 +230,9 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
       pdl_wait();
       for (int i = 0; i < pre; ++i) {
         const uint32_t b_dst = smem_base + (uint32_t)(i * stage_bytes) + L::kABytes * (lo ? 2 : 1);
-        ptx::tma_load_2d(b_dst, &tm_x, (kb_begin + i) * kBlockK, m0, full_bar(i), ptx::kEvictLast);
+        const bool second = p.dual_kb && kb_begin + i >= p.dual_kb;
+        ptx::tma_load_2d(b_dst, second ? &tm_x2 : &tm_x, (kb_begin + i - (second ? p.dual_kb : 0)) * kBlockK, m0, full_bar(i),
+                         ptx::kEvictLast);
       }
       for (int i = pre; i < n_kb; ++i) {
         const int s = i % n_stages;
@@ -235,7 +243,11 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         const int kcoord = (kb_begin + i) * kBlockK;
         const int wc0 = p.tiled ? 0 : kcoord;
         const int wc1 = p.tiled ? (n_tile * p.kblocks + kb_begin + i) * kBlockM : n0;
-        if (p.swiglu_I) {
+        const bool second = p.dual_kb && kb_begin + i >= p.dual_kb;
+        const int kcoord2 = second ? kcoord - p.dual_kb * kBlockK : kcoord;
+        if (second) {
+          ptx::tma_load_2d(a_dst, &tm_wlo, kcoord2, n0, full_bar(s), ptx::kEvictFirst);
+        } else if (p.swiglu_I) {
           ptx::tma_load_2d(a_dst, &tm_w, wc0, n_tile * 64, full_bar(s), ptx::kEvictFirst);
           ptx::tma_load_2d(a_dst + L::kABytes / 2, &tm_w, wc0, (int)p.swiglu_I + n_tile * 64, full_bar(s), ptx::kEvictFirst);
         } else {
@@ -246,7 +258,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
           ptx::tma_load_2d(a_dst + L::kABytes, &tm_wlo, wc0, wc1, full_bar(s), ptx::kEvictFirst);
           b_dst += L::kABytes;
         }
-        ptx::tma_load_2d(b_dst, &tm_x, kcoord, m0, full_bar(s), ptx::kEvictLast);
+        ptx::tma_load_2d(b_dst, second ? &tm_x2 : &tm_x, kcoord2, m0, full_bar(s), ptx::kEvictLast);
       }
     }
   } else if (warp == 1) {
@@ -454,7 +466,7 @@ __global__ void __launch_bounds__(128) head_combine_kernel(const HeadPart* __res
 
 template <int kNTile>
 int launch_gemm(const CUtensorMap& tw, const CUtensorMap& twl, const CUtensorMap& tx, const GemmParams& p,
-                cudaStream_t stream) {
+                cudaStream_t stream, const CUtensorMap* tx2 = nullptr) {
   using L = SmemLayout<kNTile>;
   const bool lo = p.has_lo != 0;
   int n_stages = L::stages(lo);
@@ -469,7 +481,7 @@ int launch_gemm(const CUtensorMap& tw, const CUtensorMap& twl, const CUtensorMap
   PRL_CUDA(ensure_smem(kernel, smem, smem_attr[p.head ? 1 : 0]));
   const int64_t feat_tiles = p.swiglu_I ? p.swiglu_I / 64 : (p.N + kBlockM - 1) / kBlockM;
   dim3 grid((unsigned)(feat_tiles * ((p.M + kNTile - 1) / kNTile)), (unsigned)p.split_k, 1);
-  PRL_CUDA(launch_pdl(kernel, grid, dim3(kThreads), (size_t)smem, stream, tw, twl, tx, p, n_stages));
+  PRL_CUDA(launch_pdl(kernel, grid, dim3(kThreads), (size_t)smem, stream, tw, twl, tx, tx2 ? *tx2 : tx, p, n_stages));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -764,6 +776,43 @@ static int gemm_splitk_impl(const void* W, const void* W_lo, const void* X, int6
     case 64: return launch_gemm<64>(tw, twl, tx, p, stream);
     case 128: return launch_gemm<128>(tw, twl, tx, p, stream);
     default: return launch_gemm<256>(tw, twl, tx, p, stream);
+  }
+}
+
+// Token-step form of prl_gemm_tn_dual (M <= 128): partials[split][M][N] of X1[M, K1] * W1[N, K1]^T + X2[M, K2] * W2[N, K2]^T.  One weight
+// stream over both matrices, so that two narrow output projections fill the SMs together.  split_k <= 0: chosen here; the
+// number of slices is returned by prl_gemm_dual_split_k(M, N, K1, K2).
+extern "C" int prl_gemm_dual_split_k(int64_t M, int64_t N, int64_t K1, int64_t K2) {
+  return prl_gemm_auto_split_k(M, N, ((K1 + kBlockK - 1) / kBlockK + (K2 + kBlockK - 1) / kBlockK) * kBlockK);
+}
+
+extern "C" int prl_gemm_bf16_dual(const void* W1, const void* X1, int64_t K1, const void* W2, const void* X2, int64_t K2, int64_t M,
+                                  int64_t N, int32_t split_k, float* partials, prl_stream_t stream_) {
+  PRL_CHECK_ARG(W1 && X1 && W2 && X2 && partials, "prl_gemm_bf16_dual: NULL argument");
+  PRL_CHECK_ARG(M >= 1 && M <= 128 && N >= 1 && K1 >= 8 && K2 >= 8 && K1 % 8 == 0 && K2 % 8 == 0 && !g_tiled_weights,
+                "prl_gemm_bf16_dual: need 1 <= M <= 128 and K1, K2 multiples of 8 (M=%lld N=%lld K1=%lld K2=%lld)", (long long)M,
+                (long long)N, (long long)K1, (long long)K2);
+  const int kb1 = (int)((K1 + kBlockK - 1) / kBlockK), kb2 = (int)((K2 + kBlockK - 1) / kBlockK);
+  if (split_k <= 0) split_k = prl_gemm_dual_split_k(M, N, K1, K2);
+  PRL_CHECK_ARG(split_k <= kb1 + kb2, "prl_gemm_bf16_dual: split_k %d > k-blocks %d", split_k, kb1 + kb2);
+  const int nt = pick_ntile(M);
+  GemmParams p = {};
+  p.M = M; p.N = N; p.K = K1 + K2; p.kblocks = kb1 + kb2; p.split_k = split_k; p.partials = partials; p.dual_kb = kb1;
+  CUtensorMap tw, tw2, tx, tx2;
+  int rc = make_weight_tmap(&tw, W1, N, K1, 0);
+  if (rc) return rc;
+  rc = make_weight_tmap(&tw2, W2, N, K2, 0);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tx, X1, (uint64_t)K1, (uint64_t)M, (uint64_t)K1 * 2, kBlockK, (uint32_t)nt);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tx2, X2, (uint64_t)K2, (uint64_t)M, (uint64_t)K2 * 2, kBlockK, (uint32_t)nt);
+  if (rc) return rc;
+  cudaStream_t stream = (cudaStream_t)stream_;
+  switch (nt) {
+    case 16: return launch_gemm<16>(tw, tw2, tx, p, stream, &tx2);
+    case 32: return launch_gemm<32>(tw, tw2, tx, p, stream, &tx2);
+    case 64: return launch_gemm<64>(tw, tw2, tx, p, stream, &tx2);
+    default: return launch_gemm<128>(tw, tw2, tx, p, stream, &tx2);
   }
 }
 

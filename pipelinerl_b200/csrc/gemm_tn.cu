@@ -36,8 +36,9 @@ constexpr int kGroupM = 8;      // row tiles per raster super-group
 struct TnParams {
   int64_t M, N, K;
   int kblocks;
-  int k_wrap;        // k-blocks >= k_wrap read B from the SECOND tensor map and A from k-block (kb - k_wrap): C = A B^T + A B2^T
-                     // in one accumulation (fp32-equivalent lm_head: B = bf16 hi part, B2 = bf16 lo residual)
+  int k_wrap;        // k-blocks >= k_wrap are k-blocks (kb - k_wrap) of the SECOND pair of tensor maps: C = A B^T + A2 B2^T in one
+                     // accumulation (fp32-equivalent lm_head: A2 = A, B = bf16 hi part, B2 = bf16 lo residual; two branches
+                     // that join the same sum: each with its own operand and weight)
   int m_tiles, n_tiles;
   int a_mn, b_mn;    // operand stored MN-major: A as [K, M] / B as [K, N] row-major (no transposed copy needed)
   void* C;
@@ -58,6 +59,7 @@ struct TnParams {
   // glu_limit > 0 (with swiglu_fp32): the clamped gate of the hybrid decoders instead of SiLU(gate) * up:
   // g = min(gate, limit), u = clamp(up, +-limit), act = g * sigmoid(glu_beta * g) * (u + 1)
   float glu_limit, glu_beta;
+  int glu_gelu;            // 1 (with swiglu_fp32): gelu(gate) * up, the tanh form of gelu
   // head epilogue (kHead): logits never leave TMEM/registers
   const int64_t* targets;  // [M] or NULL
   float4* head_part;       // [n_tiles, M]: (max, sum exp, sum exp*z, target logit or -inf) of one 256-column vocabulary tile
@@ -76,6 +78,11 @@ struct TnParams {
   int64_t ld_gu;
 };
 
+// 0.5 z (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
 __device__ __forceinline__ void tile_coords(int t, const TnParams& p, int& tm, int& tn) {
   const int per_group = kGroupM * p.n_tiles;
   const int g = t / per_group;
@@ -89,7 +96,7 @@ __device__ __forceinline__ void tile_coords(int t, const TnParams& p, int& tm, i
 template <bool kHead>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreadsTN, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_b,
-               const __grid_constant__ CUtensorMap tm_b2, TnParams p) {
+               const __grid_constant__ CUtensorMap tm_a2, const __grid_constant__ CUtensorMap tm_b2, TnParams p) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t smem_base = (ptx::smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t bar_base = smem_base + (uint32_t)(kStages * kStageBytes);
@@ -151,7 +158,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
           const int kk = (second ? kb - p.k_wrap : kb) * kBK;
           const CUtensorMap* tb = second ? &tm_b2 : &tm_b;
           if (!p.a_mn) {
-            ptx::tma_load_2d_2sm(a_dst, &tm_a, kk, a_row, full_bar(s), ptx::kEvictNormal);
+            ptx::tma_load_2d_2sm(a_dst, second ? &tm_a2 : &tm_a, kk, a_row, full_bar(s), ptx::kEvictNormal);
           } else {  // two 64(MN) x 64(k) boxes: inner coordinate = MN index, outer = k
             ptx::tma_load_2d_2sm(a_dst, &tm_a, a_row, kk, full_bar(s), ptx::kEvictNormal);
             ptx::tma_load_2d_2sm(a_dst + kMnChunkBytes, &tm_a, a_row + 64, kk, full_bar(s), ptx::kEvictNormal);
@@ -318,6 +325,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
               if (p.swiglu_fp32) {   // sampler prefill: identical bits to the fp32 GEMM output + silu_mul_kernel pair
                 const float g0 = __uint_as_float(rg[j + 2 * e]), g1 = __uint_as_float(rg[j + 2 * e + 1]);
                 const float u0 = __uint_as_float(ru[j + 2 * e]), u1 = __uint_as_float(ru[j + 2 * e + 1]);
+                if (p.glu_gelu) {
+                  ha[e] = __floats2bfloat162_rn(gelu_tanh(g0) * u0, gelu_tanh(g1) * u1);
+                  continue;
+                }
                 if (p.glu_limit > 0.f) {
                   const float l = p.glu_limit, b = p.glu_beta;
                   const float c0g = fminf(g0, l), c1g = fminf(g1, l);
@@ -588,7 +599,42 @@ extern "C" int prl_gemm_ex(const void* A, int64_t lda, int32_t a_mn_major, const
   const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
-  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, tb, p);
+  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta, tb, p);
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+// Two products in one accumulation, C[M, N] (fp32) = A1[M, K1] * B1[N, K1]^T + A2[M, K2] * B2[N, K2]^T: the output projections of two
+// branches that are added to the same residual.
+extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, const void* A2, const void* B2, int64_t K2, int64_t M,
+                                int64_t N, float* C, int64_t ldc, prl_stream_t stream_) {
+  PRL_CHECK_ARG(A1 && B1 && A2 && B2 && C, "prl_gemm_tn_dual: NULL argument");
+  PRL_CHECK_ARG(M >= 1 && N >= 1 && K1 >= 8 && K2 >= 8 && K1 % 8 == 0 && K2 % 8 == 0 && ldc >= N,
+                "prl_gemm_tn_dual: need M, N >= 1 and K1, K2 multiples of 8 (M=%lld N=%lld K1=%lld K2=%lld)", (long long)M, (long long)N,
+                (long long)K1, (long long)K2);
+  TnParams p = {};
+  p.M = M; p.N = N; p.K = K1 + K2;
+  p.k_wrap = (int)((K1 + kBK - 1) / kBK);
+  p.kblocks = p.k_wrap + (int)((K2 + kBK - 1) / kBK);
+  p.m_tiles = (int)((M + kTile - 1) / kTile);
+  p.n_tiles = (int)((N + kTile - 1) / kTile);
+  p.C = C; p.ldc = ldc; p.c_f32 = 1; p.alpha = 1.f;
+  CUtensorMap ta, tb, ta2, tb2;
+  int rc = make_tmap_2d_bf16(&ta, A1, (uint64_t)K1, (uint64_t)M, (uint64_t)K1 * 2, kBK, kHalf);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tb, B1, (uint64_t)K1, (uint64_t)N, (uint64_t)K1 * 2, kBK, kHalf);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&ta2, A2, (uint64_t)K2, (uint64_t)M, (uint64_t)K2 * 2, kBK, kHalf);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tb2, B2, (uint64_t)K2, (uint64_t)N, (uint64_t)K2 * 2, kBK, kHalf);
+  if (rc) return rc;
+  const int smem = kStages * kStageBytes + 1024 + 8 * (2 * kStages + 4) + 16;
+  static SmemAttr smem_attr = {};
+  PRL_CUDA(ensure_smem(gemm_tn_kernel<false>, smem, smem_attr));
+  const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
+  int clusters = num_sms() / 2;
+  if (tiles < clusters) clusters = (int)tiles;
+  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta2, tb2, p);
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -622,7 +668,7 @@ extern "C" int prl_gemm_dgrad_swiglu(const void* dY, int64_t ldy, const void* W_
   const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
-  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, tb, p);
+  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta, tb, p);
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -631,7 +677,7 @@ extern "C" int prl_gemm_dgrad_swiglu(const void* dY, int64_t ldy, const void* W_
 // gate_up (bf16 [M, 2 I], may be NULL) is written as well when the backward will need it.
 static int gemm_swiglu_impl(const void* X, int64_t ldx, const void* W, int64_t ldw, int64_t M, int64_t I, int64_t K,
                             void* act, int64_t ld_act, void* gate_up, int64_t ld_gu, int fp32_act, prl_stream_t stream_,
-                            float glu_limit = 0.f, float glu_beta = 0.f);
+                            float glu_limit = 0.f, float glu_beta = 0.f, int glu_gelu = 0);
 
 extern "C" int prl_gemm_swiglu(const void* X, int64_t ldx, const void* W, int64_t ldw, int64_t M, int64_t I, int64_t K,
                                void* act, int64_t ld_act, void* gate_up, int64_t ld_gu, prl_stream_t stream_) {
@@ -654,9 +700,15 @@ extern "C" int prl_gemm_glu_clamped_f32(const void* X, int64_t ldx, const void* 
   return gemm_swiglu_impl(X, ldx, W, ldw, M, I, K, act, ld_act, nullptr, 0, 1, stream_, limit, beta);
 }
 
+// the sampler form with gelu(gate) * up, gelu in its tanh form
+extern "C" int prl_gemm_geglu_f32(const void* X, int64_t ldx, const void* W, int64_t ldw, int64_t M, int64_t I, int64_t K, void* act,
+                                  int64_t ld_act, prl_stream_t stream_) {
+  return gemm_swiglu_impl(X, ldx, W, ldw, M, I, K, act, ld_act, nullptr, 0, 1, stream_, 0.f, 0.f, 1);
+}
+
 static int gemm_swiglu_impl(const void* X, int64_t ldx, const void* W, int64_t ldw, int64_t M, int64_t I, int64_t K,
                             void* act, int64_t ld_act, void* gate_up, int64_t ld_gu, int fp32_act, prl_stream_t stream_,
-                            float glu_limit, float glu_beta) {
+                            float glu_limit, float glu_beta, int glu_gelu) {
   PRL_CHECK_ARG(X && W && act, "prl_gemm_swiglu: NULL argument");
   PRL_CHECK_ARG(M >= 1 && I >= kHalf && I % kHalf == 0 && K >= 8, "prl_gemm_swiglu: need I %% 128 == 0 (M=%lld I=%lld K=%lld)",
                 (long long)M, (long long)I, (long long)K);
@@ -671,7 +723,7 @@ static int gemm_swiglu_impl(const void* X, int64_t ldx, const void* W, int64_t l
   p.n_tiles = (int)(I / kHalf);
   p.C = gate_up; p.ldc = ld_gu; p.alpha = 1.f;
   p.swiglu_I = I; p.swiglu_fp32 = fp32_act; p.act = (__nv_bfloat16*)act; p.ld_act = ld_act;
-  p.glu_limit = glu_limit; p.glu_beta = glu_beta;
+  p.glu_limit = glu_limit; p.glu_beta = glu_beta; p.glu_gelu = glu_gelu;
   CUtensorMap ta, tb;
   int rc = make_tmap_2d_bf16(&ta, X, (uint64_t)K, (uint64_t)M, (uint64_t)ldx * 2, kBK, kHalf);
   if (rc) return rc;
@@ -683,7 +735,7 @@ static int gemm_swiglu_impl(const void* X, int64_t ldx, const void* W, int64_t l
   const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
-  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, tb, p);
+  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta, tb, p);
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -717,7 +769,7 @@ int head_logprob_tn(const void* W, const void* W_lo, const void* X, int64_t M, i
   const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
-  gemm_tn_kernel<true><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, stream>>>(ta, tb, tb2, p);
+  gemm_tn_kernel<true><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, stream>>>(ta, tb, ta, tb2, p);
   PRL_LAUNCH_CHECK();
   head_tn_combine_kernel<<<(unsigned)((M + 3) / 4), 128, 0, stream>>>((const float4*)workspace, p.n_tiles, M,
                                                                       targets ? 1 : 0, logprob_target, entropy, lse);
@@ -765,7 +817,7 @@ extern "C" int prl_head_dlogits(const void* W, const void* W_lo, const void* X, 
   const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
-  gemm_tn_kernel<true><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, tb2, p);
+  gemm_tn_kernel<true><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta, tb2, p);
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }

@@ -346,20 +346,28 @@ __global__ void concat_rows_kernel(const T* __restrict__ a, const T* __restrict_
 //   x   = (add ? x : 0) + v + bias  (bias == NULL: none)
 //   xa  = T(x / rms(x) * next_gain) (next_gain == NULL: T(x)) -- the input of the NEXT sublayer's projection
 // y_i may arrive as split-K partial slices [n_split][n][ld] of a GEMM (or as the per-choice outputs of a routed
-// feed-forward): they are summed here in slice order.  One block per row; the row stays in shared memory.
+// feed-forward): they are summed here in slice order.  With `sel` the slices of y1 are the choices of a router some of
+// whose outputs hand the sublayer's INPUT through: where sel[k * n + row] >= experts, slice k of that row was never
+// written and wsel[k * n + row] * xa[row] (xa still holds the input: it is replaced last) stands in its place.
+// One block per row; the row stays in shared memory.
 template <typename T>
 __global__ void sublayer_close_kernel(const float* __restrict__ y0, int64_t ld0, int ns0, int64_t stride0,
                                       const float* __restrict__ gain0, float s0, const float* __restrict__ y1, int64_t ld1,
                                       int ns1, int64_t stride1, const float* __restrict__ gain1, float s1,
                                       const float* __restrict__ post_gain, const float* __restrict__ bias, int add,
-                                      const float* __restrict__ next_gain, float eps, int W, float* __restrict__ x,
-                                      T* __restrict__ xa) {
+                                      const float* __restrict__ next_gain, float eps, int W,
+                                      const int32_t* __restrict__ sel, const float* __restrict__ wsel, int experts,
+                                      float* __restrict__ x, T* __restrict__ xa) {
   pdl_wait();
   extern __shared__ float rowbuf[];    // [W] y0 (then v, then x) | [W] y1
   __shared__ float red[32];
   float* b0 = rowbuf;
   float* b1 = rowbuf + W;
   const int64_t r = blockIdx.x;
+  float w_pass = 0.f;                  // summed weight of the row's choices that hand the input through
+  if (sel)
+    for (int k = 0; k < ns1; ++k)
+      if (sel[(int64_t)k * gridDim.x + r] >= experts) w_pass += wsel[(int64_t)k * gridDim.x + r];
   float ss0 = 0.f, ss1 = 0.f;
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     float a = 0.f;
@@ -368,7 +376,13 @@ __global__ void sublayer_close_kernel(const float* __restrict__ y0, int64_t ld0,
     ss0 += a * a;
     if (y1) {
       float b = 0.f;
-      for (int k = 0; k < ns1; ++k) b += y1[k * stride1 + r * ld1 + c];
+      if (sel) {
+        for (int k = 0; k < ns1; ++k)
+          if (sel[(int64_t)k * gridDim.x + r] < experts) b += y1[k * stride1 + r * ld1 + c];
+        if (w_pass != 0.f) b = fmaf(w_pass, ldf(xa, r * W + c), b);
+      } else {
+        for (int k = 0; k < ns1; ++k) b += y1[k * stride1 + r * ld1 + c];
+      }
       b1[c] = b;
       ss1 += b * b;
     }
@@ -470,6 +484,28 @@ __global__ void act_store_kernel(const float* __restrict__ P, int64_t ld, int F,
   if (c >= F) return;
   const float z = fmaxf(P[r * ld + c], 0.f);
   stf(out, r * F + c, z * z);
+}
+
+// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) = z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
+// see prl_ff_act
+template <typename T>
+__global__ void ff_act_kernel(const float* __restrict__ P, int64_t ld, int off, int F, int act, int off_gate, T* __restrict__ out) {
+  pdl_wait();
+  const int64_t r = blockIdx.x;
+  const float* p = P + r * ld + off;
+  const float s = off_gate >= 0 ? sigmoid_f(P[r * ld + off_gate]) : 1.f;
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    const int c = blockIdx.y * 1024 + u * 256 + threadIdx.x;
+    if (c >= F) break;
+    const float z = p[c];
+    const float a = act == 1 ? gelu_tanh_f(z) * p[F + c] : fmaxf(z, 0.f) * fmaxf(z, 0.f);
+    stf(out, r * F + c, a * s);
+  }
 }
 
 // ---- matrix-memory LSTM (mLSTM) --------------------------------------------------------------------------------------
@@ -610,7 +646,8 @@ __global__ void postln_close_kernel(const float* __restrict__ y0, int64_t ld0, f
 //   v:    + bias; v_norm: each head divided by its root mean square over `vdim` (no gain); then
 //         v_blend == 1: the row's values are also written to v_first [n][G * vdim] (fp32) for later layers,
 //         v_blend == 2: v <- (1 - lambda) v + lambda v_first[row], lambda = *v_lambda.
-// q goes to the query buffer [n][H][dim], k and v into the paged cache.  One warp per head.
+// q goes to the query buffer [n][H][dim], k and v into the paged cache.  G == 0: queries only (a layer that reads another
+// layer's cache).  One warp per head.
 template <typename T>
 __global__ void attn_front_kernel(const float* __restrict__ P, int64_t ldp, int off_q, int off_k, int off_v, int H, int G,
                                   int dim, int vdim, const float* __restrict__ q_bias, const float* __restrict__ k_bias,
@@ -848,10 +885,11 @@ extern "C" int prl_concat_rows(const void* a, const void* b, int32_t n, int32_t 
   return PRL_OK;
 }
 
-extern "C" int prl_sublayer_close(const float* y0, int64_t ld0, int32_t n_split0, const float* gain0, float s0,
-                                  const float* y1, int64_t ld1, int32_t n_split1, const float* gain1, float s1,
-                                  const float* post_gain, const float* bias, int32_t add, const float* next_gain, float eps,
-                                  int32_t n, int32_t W, float* x, void* xa, int32_t f32, prl_stream_t st) {
+static int sublayer_close_impl(const float* y0, int64_t ld0, int32_t n_split0, const float* gain0, float s0,
+                               const float* y1, int64_t ld1, int32_t n_split1, const float* gain1, float s1,
+                               const float* post_gain, const float* bias, int32_t add, const float* next_gain, float eps,
+                               int32_t n, int32_t W, const int32_t* sel, const float* wsel, int32_t experts, float* x, void* xa,
+                               int32_t f32, prl_stream_t st) {
   PRL_CHECK_ARG(y0 && x && xa && n >= 1 && W >= 1 && ld0 >= W && (!y1 || ld1 >= W) && n_split0 >= 1 && (!y1 || n_split1 >= 1),
                 "prl_sublayer_close: bad argument");
   const size_t smem = 2 * (size_t)W * sizeof(float);
@@ -863,11 +901,44 @@ extern "C" int prl_sublayer_close(const float* y0, int64_t ld0, int32_t n_split0
   static SmemAttr attr_f = {}, attr_b = {};
   if (f32) {
     if (smem > 48 * 1024) PRL_CUDA(ensure_smem(sublayer_close_kernel<float>, (int)smem, attr_f));
-    PRL_CUDA(launch_pdl(sublayer_close_kernel<float>, dim3(n), dim3(th), smem, (cudaStream_t)st, y0, ld0, n_split0, st0, gain0, s0, y1, ld1, n_split1, st1, gain1, s1, post_gain, bias, add, next_gain, eps, W, x, (float*)xa));
+    PRL_CUDA(launch_pdl(sublayer_close_kernel<float>, dim3(n), dim3(th), smem, (cudaStream_t)st, y0, ld0, n_split0, st0, gain0, s0, y1, ld1, n_split1, st1, gain1, s1, post_gain, bias, add, next_gain, eps, W, sel, wsel, experts, x, (float*)xa));
   } else {
     if (smem > 48 * 1024) PRL_CUDA(ensure_smem(sublayer_close_kernel<bf16>, (int)smem, attr_b));
-    PRL_CUDA(launch_pdl(sublayer_close_kernel<bf16>, dim3(n), dim3(th), smem, (cudaStream_t)st, y0, ld0, n_split0, st0, gain0, s0, y1, ld1, n_split1, st1, gain1, s1, post_gain, bias, add, next_gain, eps, W, x, (bf16*)xa));
+    PRL_CUDA(launch_pdl(sublayer_close_kernel<bf16>, dim3(n), dim3(th), smem, (cudaStream_t)st, y0, ld0, n_split0, st0, gain0, s0, y1, ld1, n_split1, st1, gain1, s1, post_gain, bias, add, next_gain, eps, W, sel, wsel, experts, x, (bf16*)xa));
   }
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+extern "C" int prl_sublayer_close(const float* y0, int64_t ld0, int32_t n_split0, const float* gain0, float s0,
+                                  const float* y1, int64_t ld1, int32_t n_split1, const float* gain1, float s1,
+                                  const float* post_gain, const float* bias, int32_t add, const float* next_gain, float eps,
+                                  int32_t n, int32_t W, float* x, void* xa, int32_t f32, prl_stream_t st) {
+  return sublayer_close_impl(y0, ld0, n_split0, gain0, s0, y1, ld1, n_split1, gain1, s1, post_gain, bias, add, next_gain, eps, n,
+                             W, nullptr, nullptr, 0, x, xa, f32, st);
+}
+
+// The close of a layer whose mixer and routed feed-forward read ONE normed input and are both added to the residual:
+// x += sum y0 slices + sum of the routed choices (y1: [top][n][W]; NULL when the layer has none), a choice sel >= experts
+// being the layer's input itself times its weight; then the next layer's norm into xa (next_gain NULL: xa = T(x)).
+extern "C" int prl_joint_close(const float* y0, int32_t n_split0, const float* y1, int32_t top, const int32_t* sel, const float* wsel,
+                               int32_t experts, const float* next_gain, float eps, int32_t n, int32_t W, float* x, void* xa,
+                               int32_t f32, prl_stream_t st) {
+  PRL_CHECK_ARG(!y1 || (sel && wsel && experts >= 1), "prl_joint_close: routed slices need their choices and weights");
+  return sublayer_close_impl(y0, W, n_split0, nullptr, 1.f, y1, W, y1 ? top : 1, nullptr, 1.f, nullptr, nullptr, 1, next_gain, eps,
+                             n, W, y1 ? sel : nullptr, wsel, experts, x, xa, f32, st);
+}
+
+// Feed-forward activation from columns of a projection buffer: act 0: relu(z)^2, z = P[r, off + c]; act 1: gelu(gate) * up in
+// the tanh form, gate = P[r, off + c], up = P[r, off + F + c].  off_gate >= 0: times sigmoid(P[r, off_gate]) (one number
+// per row).  out [n][F] in the operand type.
+extern "C" int prl_ff_act(const float* P, int64_t ld, int32_t off, int32_t n, int32_t F, int32_t act, int32_t off_gate, void* out,
+                          int32_t f32, prl_stream_t st) {
+  PRL_CHECK_ARG(P && out && n >= 1 && F >= 1 && off >= 0 && (act == 0 || act == 1) && ld >= off + (int64_t)F * (act + 1) && ld > off_gate,
+                "prl_ff_act: bad argument");
+  dim3 grid(n, (F + 1023) / 1024);
+  if (f32) PRL_CUDA(launch_pdl(ff_act_kernel<float>, grid, dim3(256), (size_t)0, (cudaStream_t)st, P, ld, off, F, act, off_gate, (float*)out));
+  else PRL_CUDA(launch_pdl(ff_act_kernel<bf16>, grid, dim3(256), (size_t)0, (cudaStream_t)st, P, ld, off, F, act, off_gate, (bf16*)out));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -965,8 +1036,8 @@ extern "C" int prl_attn_front(const float* P, int64_t ldp, int32_t off_q, int32_
                               int32_t v_blend, const float* v_lambda, float* v_first, const int32_t* row_pos,
                               const int32_t* row_slot, const int32_t* block_table, int32_t max_blocks, int32_t page_size,
                               void* q_out, void* k_pool, void* v_pool, int32_t f32, prl_stream_t st) {
-  PRL_CHECK_ARG(P && row_pos && row_slot && block_table && q_out && k_pool && v_pool, "prl_attn_front: NULL argument");
-  PRL_CHECK_ARG(n >= 1 && H >= 1 && G >= 1 && dim >= 1 && vdim >= 1 && page_size >= 1 && max_blocks >= 1 && rot >= 0 &&
+  PRL_CHECK_ARG(P && row_pos && row_slot && block_table && q_out && (G == 0 || (k_pool && v_pool)), "prl_attn_front: NULL argument");
+  PRL_CHECK_ARG(n >= 1 && H >= 1 && G >= 0 && dim >= 1 && vdim >= 1 && page_size >= 1 && max_blocks >= 1 && rot >= 0 &&
                 rot <= dim && rot % 2 == 0 && (rot == 0 || freq) && gain_period >= 1,
                 "prl_attn_front: bad shape (H=%d G=%d dim=%d vdim=%d rot=%d)", H, G, dim, vdim, rot);
   PRL_CHECK_ARG(v_blend >= 0 && v_blend <= 2 && (v_blend == 0 || v_first) && (v_blend != 2 || v_lambda),

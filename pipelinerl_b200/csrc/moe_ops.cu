@@ -1,9 +1,12 @@
 // Routed feed-forward (mixture of experts) over a packed batch of n token rows, without a host round trip: the number
 // of rows each expert gets stays on the device, so the whole layer can sit in a CUDA graph.
 //
-//   1. route:  per row, the `top` experts with the largest router logits (ties: the lower index), each with the weight
+//   1. route:  (prl_moe_route, prl_moe_router) per row, the `top` experts with the largest router logits (ties: the lower index), each with the weight
 //              sigmoid(logit) or softmax over the chosen; an optional bias per expert joins the logits first; choice c
-//              of row t is the PAIR c * n + t.
+//              of row t is the PAIR c * n + t.  prl_moe_choose instead takes ready logits and ranks the outputs by their
+//              softmax share plus a correction (which the weights do not see), inside the best groups of outputs only;
+//              outputs past the experts ("identity") hand the input through: their pairs are chosen and weighted like
+//              the others but join no expert's rows.
 //   2. group:  a stable counting sort of the pairs by expert (one CTA): perm[s] = pair at sorted place s, and a table
 //              of row tiles (expert, first sorted place, rows <= 64) that the GEMMs walk; its length stays on the device.
 //   3. grouped GEMM (twice):  C[row] = A[row'] * W_e^T for every tile, W_e = W + e * expert_stride.  The first product
@@ -144,6 +147,72 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ 
     for (int c = 0; c < top; ++c) wsel[(int64_t)c * n + t] /= denom;
 }
 
+// Choice from ready logits, one warp per row.  s = softmax(z) over all E outputs; outputs are ranked by c = s + correction.
+// The outputs form `groups` equal groups of neighbours ranked by their best c; only the `keep` best groups are open.
+// The `top` best open outputs (ties: the lower index) are chosen, each with its weight s.
+constexpr int kChooseWarps = 4;
+__global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const float* __restrict__ logits, int64_t ld,
+                                                                       const float* __restrict__ correction, int n, int E, int top,
+                                                                       int groups, int keep, int32_t* __restrict__ sel,
+                                                                       float* __restrict__ wsel) {
+  pdl_wait();
+  extern __shared__ float csm[];                 // per warp: [E] choice scores | [groups] group scores
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * kChooseWarps + warp;
+  if (t >= n) return;
+  float* c = csm + (size_t)warp * (E + groups);
+  float* gs = c + E;
+  const float* z = logits + (int64_t)t * ld;
+  float zmax = -INFINITY;
+  for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
+  zmax = warp_max(zmax);
+  float sum = 0.f;
+  for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
+  const float inv = 1.f / warp_sum(sum);
+  for (int e = lane; e < E; e += 32) c[e] = expf(z[e] - zmax) * inv + (correction ? correction[e] : 0.f);
+  __syncwarp();
+  auto best_of = [&](const float* v, int count) {          // index of the largest entry, the lowest on a tie
+    float best = -INFINITY;
+    int arg = 0x7fffffff;
+    for (int e = lane; e < count; e += 32)
+      if (v[e] > best) { best = v[e]; arg = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+    }
+    return arg;
+  };
+  if (keep < groups) {
+    const int size = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float m = -INFINITY;
+      for (int e = 0; e < size; ++e) m = fmaxf(m, c[g * size + e]);
+      gs[g] = m;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {                       // an open group is marked by taking it out of the ranking
+      const int g = best_of(gs, groups);
+      if (lane == 0 && g < groups) gs[g] = -INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gs[e / size] != -INFINITY) c[e] = -INFINITY;     // still ranked: a closed group
+    __syncwarp();
+  }
+  for (int k = 0; k < top; ++k) {
+    const int e = best_of(c, E);
+    if (lane == 0) {
+      const bool ok = e < E;                               // always, for finite logits
+      sel[(int64_t)k * n + t] = ok ? e : 0;
+      wsel[(int64_t)k * n + t] = ok ? expf(z[e] - zmax) * inv : 0.f;
+      if (ok) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+}
+
 // meta[0] = number of tiles; tiles[3 * i + {0, 1, 2}] = expert, first sorted place, rows
 __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restrict__ sel, int pairs, int E,
                                                          int32_t* __restrict__ perm, int32_t* __restrict__ meta,
@@ -154,7 +223,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
   for (int e = tid; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int p = tid; p < pairs; p += blockDim.x) atomicAdd(&cnt[sel[p]], 1);
+  for (int p = tid; p < pairs; p += blockDim.x)
+    if (sel[p] < E) atomicAdd(&cnt[sel[p]], 1);          // a choice past the experts belongs to none of them
   __syncthreads();
   if (tid == 0) {
     int at = 0, nt = 0;
@@ -183,23 +253,27 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
   }
 }
 
-template <typename TA, typename TW>
+// RELU2: C is the next product's operand (type TA), C[row] = relu(product)^2 * wsel[pair]
+template <typename TA, typename TW, bool RELU2>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A, int64_t lda, int a_mod,
                                                        const TW* __restrict__ W, int64_t expert_stride, int64_t ldw,
                                                        const int32_t* __restrict__ perm, const int32_t* __restrict__ meta,
                                                        const int32_t* __restrict__ tiles, int N, int K,
-                                                       float* __restrict__ C, int64_t ldc, int c_perm) {
+                                                       void* __restrict__ C_v, int64_t ldc, int c_perm,
+                                                       const float* __restrict__ wsel) {
   pdl_wait();
   const int tile = blockIdx.y;
   if (tile >= meta[0]) return;
   __shared__ float As[kStepK][kTile + 4];
   __shared__ float Ws[kStepK][kTile + 4];
   __shared__ int32_t a_row[kTile], c_row[kTile];
+  __shared__ float c_w[kTile];
   const int e = tiles[3 * tile], s0 = tiles[3 * tile + 1], M = tiles[3 * tile + 2];
   const int tid = threadIdx.x;
   if (tid < kTile) {
     const int s = s0 + min(tid, M - 1);
     const int p = perm[s];
+    if constexpr (RELU2) c_w[tid] = wsel[p];
     a_row[tid] = a_mod > 0 ? p % a_mod : s;
     c_row[tid] = c_perm ? p : s;
   }
@@ -245,7 +319,13 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int nn = n0 + tn + j;
-      if (nn < N) C[row * ldc + nn] = acc[i][j];
+      if (nn >= N) continue;
+      if constexpr (RELU2) {
+        const float z = fmaxf(acc[i][j], 0.f);
+        reinterpret_cast<TA*>(C_v)[row * ldc + nn] = TA(z * z * c_w[tm + i]);
+      } else {
+        reinterpret_cast<float*>(C_v)[row * ldc + nn] = acc[i][j];
+      }
     }
   }
 }
@@ -271,11 +351,13 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+template <bool RELU2>
 __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, int a_mod,
                                                            const __nv_bfloat16* __restrict__ W, int64_t expert_stride,
                                                            int64_t ldw, const int32_t* __restrict__ perm,
                                                            const int32_t* __restrict__ meta, const int32_t* __restrict__ tiles,
-                                                           int N, int K, float* __restrict__ C, int64_t ldc, int c_perm) {
+                                                           int N, int K, void* __restrict__ C_v, int64_t ldc, int c_perm,
+                                                           const float* __restrict__ wsel) {
   pdl_wait();
   const int tile = blockIdx.y;
   if (tile >= meta[0]) return;
@@ -285,11 +367,13 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
   ATile As = reinterpret_cast<ATile>(mma_smem);                                           // [kStages][64][40]
   BTile Bs = reinterpret_cast<BTile>(mma_smem + (size_t)kStages * kTile * kLds * sizeof(__nv_bfloat16));   // [kStages][128][40]
   __shared__ int32_t a_row[kTile], c_row[kTile];
+  __shared__ float c_w[kTile];
   const int e = tiles[3 * tile], s0 = tiles[3 * tile + 1], M = tiles[3 * tile + 2];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid < kTile) {
     const int s = s0 + min(tid, M - 1);
     const int p = perm[s];
+    if constexpr (RELU2) c_w[tid] = wsel[p];
     a_row[tid] = a_mod > 0 ? p % a_mod : s;
     c_row[tid] = c_perm ? p : s;
   }
@@ -348,7 +432,20 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
     for (int half = 0; half < 2; ++half) {
       const int m = wm + 16 * i + (lane >> 2) + 8 * half;
       if (m >= M) continue;
-      float* crow = C + (int64_t)c_row[m] * ldc;
+      const int64_t at = (int64_t)c_row[m] * ldc;
+      if constexpr (RELU2) {
+        __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(C_v) + at;
+        const float w = c_w[m];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int nn = n0 + wn + 8 * j + (lane & 3) * 2;
+          const float z0 = fmaxf(acc[i][j][2 * half], 0.f), z1 = fmaxf(acc[i][j][2 * half + 1], 0.f);
+          if (nn < N) crow[nn] = __float2bfloat16_rn(z0 * z0 * w);
+          if (nn + 1 < N) crow[nn + 1] = __float2bfloat16_rn(z1 * z1 * w);
+        }
+        continue;
+      }
+      float* crow = reinterpret_cast<float*>(C_v) + at;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int nn = n0 + wn + 8 * j + (lane & 3) * 2;
@@ -437,11 +534,31 @@ extern "C" int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, i
   return PRL_OK;
 }
 
-extern "C" int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
-                            int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
-                            const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, float* C, int64_t ldc,
-                            int32_t c_perm, prl_stream_t st) {
-  PRL_CHECK_ARG(A && W && perm && meta && tiles && C, "prl_moe_gemm: NULL argument");
+// Choice among outputs whose logits are already there (columns of a projection buffer), and the grouping of the pairs by expert:
+// `outputs` = experts + identity outputs; see moe_choose_kernel.  keep == groups (e.g. 1, 1): every output is open.
+extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
+                              int32_t top, int32_t groups, int32_t keep, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta,
+                              int32_t* tiles, prl_stream_t st) {
+  PRL_CHECK_ARG(logits && sel && wsel && perm && meta && tiles, "prl_moe_choose: NULL argument");
+  PRL_CHECK_ARG(n >= 1 && experts >= 1 && outputs >= experts && outputs <= 1024 && ld >= outputs && groups >= 1 &&
+                outputs % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= outputs / groups * keep,
+                "prl_moe_choose: bad shape (experts=%d outputs=%d top=%d groups=%d keep=%d)", experts, outputs, top, groups, keep);
+  cudaStream_t s = (cudaStream_t)st;
+  PRL_CUDA(launch_pdl(moe_choose_kernel, dim3((n + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32),
+                      (size_t)kChooseWarps * (outputs + groups) * sizeof(float), s, logits, ld, correction, n, outputs, top, groups,
+                      keep, sel, wsel));
+  PRL_LAUNCH_CHECK();
+  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, perm, meta, tiles));
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+template <bool RELU2>
+static int moe_gemm_impl(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                         int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
+                         int64_t max_tiles, int64_t N, int64_t K, void* C, int64_t ldc, int32_t c_perm, const float* wsel,
+                         prl_stream_t st) {
+  PRL_CHECK_ARG(A && W && perm && meta && tiles && C && (!RELU2 || wsel), "prl_moe_gemm: NULL argument");
   PRL_CHECK_ARG(max_tiles >= 1 && max_tiles <= 65535 && N >= 1 && K >= 1 && lda >= K && ldw >= K && ldc >= N && a_mod >= 0,
                 "prl_moe_gemm: bad shape (tiles=%lld N=%lld K=%lld)", (long long)max_tiles, (long long)N, (long long)K);
   cudaStream_t s = (cudaStream_t)st;
@@ -449,15 +566,15 @@ extern "C" int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_
       ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
     dim3 grid_tc((unsigned)((N + kBN - 1) / kBN), (unsigned)max_tiles);
     static SmemAttr attr = {};
-    PRL_CUDA(ensure_smem(moe_gemm_mma_kernel, (int)kMmaSmem, attr));
-    PRL_CUDA(launch_pdl(moe_gemm_mma_kernel, grid_tc, dim3(256), kMmaSmem, s, (const bf16*)A, lda, a_mod, (const bf16*)W,
-                        expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm));
+    PRL_CUDA(ensure_smem(moe_gemm_mma_kernel<RELU2>, (int)kMmaSmem, attr));
+    PRL_CUDA(launch_pdl(moe_gemm_mma_kernel<RELU2>, grid_tc, dim3(256), kMmaSmem, s, (const bf16*)A, lda, a_mod, (const bf16*)W,
+                        expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm, wsel));
     PRL_LAUNCH_CHECK();
     return PRL_OK;
   }
   dim3 grid((unsigned)((N + kTile - 1) / kTile), (unsigned)max_tiles);
-#define PRL_MG(TA, TW) PRL_CUDA(launch_pdl((moe_gemm_kernel<TA, TW>), grid, dim3(256), (size_t)0, s, (const TA*)A, lda, a_mod, (const TW*)W, \
-                                           expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm))
+#define PRL_MG(TA, TW) PRL_CUDA(launch_pdl((moe_gemm_kernel<TA, TW, RELU2>), grid, dim3(256), (size_t)0, s, (const TA*)A, lda, a_mod, (const TW*)W, \
+                                           expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm, wsel))
   if (a_is_f32 && w_is_f32) PRL_MG(float, float);
   else if (a_is_f32) PRL_MG(float, bf16);
   else if (w_is_f32) PRL_MG(bf16, float);
@@ -465,6 +582,24 @@ extern "C" int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_
 #undef PRL_MG
   PRL_LAUNCH_CHECK();
   return PRL_OK;
+}
+
+extern "C" int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                            int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
+                            const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, float* C, int64_t ldc,
+                            int32_t c_perm, prl_stream_t st) {
+  return moe_gemm_impl<false>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles, N, K, C, ldc,
+                              c_perm, nullptr, st);
+}
+
+// First product of squared-ReLU experts: act[s] = relu(A[row of s] W_e^T)^2 * wsel[pair of s], in the operand type of A and in
+// sorted order, i.e. the second product's operand (its weight on the expert's OUTPUT: that product is linear).
+extern "C" int prl_moe_gemm_relu2(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                                  int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
+                                  const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, const float* wsel, void* act,
+                                  int64_t ld_act, prl_stream_t st) {
+  return moe_gemm_impl<true>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles, N, K, act,
+                             ld_act, 0, wsel, st);
 }
 
 extern "C" int prl_moe_glu(const float* gate_up, int64_t ld, int64_t pairs, int32_t F, const int32_t* perm,

@@ -16,7 +16,12 @@ heads expanded from one cached low-rank latent, a rotated key part shared by the
 softmax denominator), a delta-rule matrix memory with per-channel decay and removal rate, a residual kept as several
 parallel streams that every sublayer reads and writes through learned weights, a statistics-free tanh norm, per-channel
 layer scale and a sigmoid gate on every sublayer's result, routed experts weighted by a softmax over all experts, and a
-hashed token-pair table added to the embedding (the previous token is per-sequence state).
+hashed token-pair table added to the embedding (the previous token is per-sequence state).  "Futetar" (`.from_futetar`)
+adds the "one norm" block: mixer and feed-forward of a layer read the same normed input and are both added to the residual,
+so a layer is one input projection, one output product over both branches and one closing kernel; softmax attention whose
+keys and values may be another layer's, rotary frequencies scaled in bands, a gated feed-forward with a tanh-form gelu,
+squared-ReLU experts chosen by corrected softmax shares inside the best expert groups, outputs of the router that hand the
+input through, and a gated shared expert.
 
 Numerics: the residual stream, every norm, softmax, router-like gate, decay, step size and recurrent state are fp32.
 GEMM operands and the KV cache are bf16, or fp32 when the arena is fp32 (the true-fp32 mode: CUDA-core GEMMs with fp32
@@ -58,7 +63,9 @@ class AttnSpec:
     v_bias: bool = False        # the value projection has a bias
     o_bias: bool = False        # the output projection has a bias
     rot_half: bool = False      # rotated pairs are (i, i + rot_dims / 2) instead of (2i, 2i + 1)
-    rot_scaling: tuple | None = None   # YaRN: (factor, original length, fast turns, slow turns)
+    rot_scaling: tuple | None = None   # YaRN: (factor, original length, fast turns, slow turns); "bands": see rotary_table
+    rot_scaling_kind: str = "yarn"     # "yarn" | "bands"
+    kv_from: int = -1           # >= 0: the run whose cache this layer reads; it has no keys and values of its own
     v_norm: bool = False        # every value head divided by its root mean square (no gain) before it is cached
     v_mix: int = 0              # 1: this layer's values are kept for later layers; 2: v <- (1 - l) v + l v_first, l = `vmix`
     v_mix_tensor: bool = False  # the checkpoint has a `vmix` scalar for this layer (used only when v_mix == 2)
@@ -151,6 +158,16 @@ class MoeSpec:
     router_bias: bool = False   # the router logits get a bias per expert (`router.b`) before the choice
     weight_on: str = "input"    # the score scales the expert's "input" (clamped unit) or its "output" (plain SiLU unit)
     weight_scale: float = 1.0   # constant factor on the scores
+    # what follows belongs to the routed feed-forwards of the "one_norm" block (squared-ReLU experts, score "softmax_all")
+    identity: int = 0           # router outputs behind the experts that hand the input through
+    groups: int = 1             # the outputs form this many equal groups of neighbours, ranked by their best choice score;
+    keep_groups: int = 1        # only outputs of the best `keep_groups` of them can be chosen
+    correction: bool = False    # a learned offset per output joins the scores for the choice, not for the weights
+    shared_gate: bool = False   # the shared expert's output times the sigmoid of one logit per token
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
 
 
 @dataclass(frozen=True)
@@ -190,6 +207,7 @@ class MlpSpec:
     limit: float
     beta: float = 1.702  # g * sigmoid(beta * g)
     kind: str = "glu"    # "glu": clamped gated unit | "relu2": W_down relu(W_up h)^2 | "moe": routed experts (+ a shared one)
+                         # | "geglu": W_down (gelu(W_gate h) * (W_up h)), gelu in its tanh form
     moe: MoeSpec | None = None
 
 
@@ -198,7 +216,8 @@ class LayerSpec:
     kind: str                       # "gla" | "parallel" (attention || state space) | "parallel_lin" (attention || lightning) | "mlstm"
                                     # | "latent" (latent attention) | "delta" (delta-rule memory): the multi-stream program
                                     # | "attention" | "latent_attention" | "sigmoid_delta" (attention without a softmax ||
-                                    #   gated delta rule): the layers normed after the sum
+                                    #   gated delta rule): the layers normed after the sum ("post_ln")
+                                    # | "mlstm" and "attention" are also the mixers of the "one_norm" block
     weights_of: int                 # index of the layer whose tensors this layer uses (its own index if it has its own)
     gla: GlaSpec | None = None
     attn: AttnSpec | None = None
@@ -219,6 +238,16 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
+class JointRows:
+    """Columns of the projection buffer of a 'one_norm' layer: [mixer | gate, up  or  shared up, shared gate, router]."""
+    mix: int        # rows of the mixer's part (a multiple of eight)
+    ff: int         # first row of the feed-forward's part: gate | up, or the shared expert's up projection
+    shared_gate: int
+    router: int
+    total: int      # a multiple of eight
+
+
+@dataclass(frozen=True)
 class HybridConfig:
     vocab_size: int
     width: int
@@ -233,6 +262,7 @@ class HybridConfig:
     streams: int = 1                # parallel copies of the residual ("tanh" program only)
     pair_embed: tuple | None = None  # (buckets, mul_prev, mul_cur): hashed (previous, current) token table `bigram`
     block: str = "out_norm"         # "post_ln": x <- norm(skip_scale * x + f(x)) for every sublayer, f reads x itself
+                                    # "one_norm": x <- x + (mixer(h) + ff(h)), h = norm(x)
     skip_scale: float = 1.0
     tied_head: bool = False         # logits = embed . x: no separate `head` tensor
 
@@ -467,7 +497,85 @@ class HybridConfig:
         cfg.validate()
         return cfg
 
+    # ---- the "Futetar" reading of config.json ---------------------------------------------------------------------
+    @staticmethod
+    def from_futetar(d: dict, tensor_shapes: dict | None = None) -> "HybridConfig":
+        """config.json of a Futetar checkpoint: the "one norm" block around matrix-memory LSTM and attention mixers in any
+        order, with a gated dense, a routed or no feed-forward.  `kv_from` names the layer whose cache an attention layer
+        reads.  Whether a router has a correction and a shared expert a gate is read off the tensor names when a file is
+        at hand."""
+        shapes = tensor_shapes or {}
+        layers = []
+        for i, L in enumerate(d["layers"]):
+            m, f, mlp = L["mixer"], L.get("mlp"), None
+            has = (lambda name: f"l{i}.{name}" in shapes) if shapes else (lambda name: True)
+            if f is not None:
+                kind = f.get("kind", "dense")
+                if kind == "dense":
+                    mlp = MlpSpec(ff=int(f["ff"]), limit=0.0, kind="geglu")
+                elif kind == "moe":
+                    r, sh, g = f["router"], f.get("shared"), f["router"].get("groups") or {}
+                    moe = MoeSpec(int(r["experts"]), int(r["top"]), int(f["expert"]["ff"]), 0.0, int(sh["ff"]) if sh else 0,
+                                  score="softmax_all", weight_on="output", identity=int(r.get("identity") or 0),
+                                  groups=int(g.get("count", 1)), keep_groups=int(g.get("keep", g.get("count", 1))),
+                                  correction=has("mlp.correction"), shared_gate=bool(sh) and has("mlp.shared.sg"))
+                    mlp = MlpSpec(ff=moe.shared_ff, limit=0.0, kind="moe", moe=moe)
+                else:
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
+            if L["type"] == "mlstm":
+                layers.append(LayerSpec("mlstm", i, mlp=mlp, mlstm=MlstmSpec(
+                    int(m["heads"]), int(m["dim"]), int(m.get("vdim", m["dim"])), float(m.get("gate_cap") or 0.0))))
+            elif L["type"] == "attention":
+                rot = m.get("rot") or {}
+                sc = rot.get("scaling")
+                src = m.get("kv_from")
+                attn = AttnSpec(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m.get("vdim", m["dim"])),
+                                int(rot.get("dims", 0)), float(rot.get("base", 10000.0)), float(m["scale"]), head_norm=True,
+                                head_gain=True, gate=False, rot_half=True, rot_scaling_kind="bands",
+                                rot_scaling=(float(sc["factor"]), float(sc["low"]), float(sc["high"]), float(sc["original"])) if sc else None,
+                                kv_from=-1 if src is None else int(src))
+                layers.append(LayerSpec("attention", i, attn=attn, mlp=mlp))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+        cfg = HybridConfig(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), 1.0, tuple(layers), block="one_norm",
+                           norm_offset=1.0)
+        cfg.validate()
+        return cfg
+
+    def _validate_one_norm(self) -> None:
+        for i, L in enumerate(self.layers):
+            if L.kind not in ("mlstm", "attention"):
+                raise ValueError(f"layer run {i}: the 'one_norm' block has matrix-memory and attention mixers")
+            if L.kind == "mlstm":
+                c = L.mlstm
+                if c.dim > 256 or c.gate_cap < 0 or min(c.heads, c.dim, c.vdim) < 1:
+                    raise ValueError(f"layer run {i}: bad matrix-memory geometry {c}")
+            else:
+                a = L.attn
+                if (min(a.heads, a.kv_heads, a.dim, a.vdim) < 1 or a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim
+                        or a.dim > 1024 or a.vdim > 512):
+                    raise ValueError(f"layer run {i}: bad attention geometry {a}")
+                if a.kv_from >= 0:
+                    b = self.layers[a.kv_from].attn if a.kv_from < i else None
+                    if b is None or self.layers[a.kv_from].kind != "attention" or b.kv_from >= 0:
+                        raise ValueError(f"layer run {i}: kv_from names run {a.kv_from}, which has no keys of its own before it")
+                    if (a.kv_heads, a.dim, a.vdim, a.rot_dims, a.rot_base, a.rot_scaling) != (b.kv_heads, b.dim, b.vdim, b.rot_dims,
+                                                                                              b.rot_base, b.rot_scaling):
+                        raise ValueError(f"layer run {i}: key / value geometry differs from run {a.kv_from}, whose cache it reads")
+            f = L.mlp
+            if f is None:
+                continue
+            if f.kind == "moe":
+                e = f.moe
+                if (e.experts < 1 or e.ff < 1 or e.identity < 0 or e.outputs > 1024 or e.groups < 1 or e.outputs % e.groups
+                        or not 1 <= e.keep_groups <= e.groups or not 1 <= e.top <= e.outputs // e.groups * e.keep_groups):
+                    raise ValueError(f"layer run {i}: bad router {e}")
+            elif f.kind != "geglu" or f.ff < 1:
+                raise ValueError(f"layer run {i}: bad feed-forward {f}")
+
     def validate(self) -> None:
+        if self.block == "one_norm":
+            return self._validate_one_norm()
         if self.norm_kind == "tanh":
             if not 1 <= self.streams <= 8 or any(L.kind not in ("latent", "delta") for L in self.layers):
                 raise ValueError("the multi-stream program runs latent-attention and delta-rule layers over 1 to 8 streams")
@@ -552,8 +660,8 @@ class HybridConfig:
             if L.kind in ("latent", "delta"):
                 out += [(name, shape) for name, shape, _ in self._stream_layer_tensors(i, L)]
                 continue
-            if self.block == "post_ln":
-                out += [(name, shape) for name, shape, _ in self._postln_layer_tensors(i, L)]
+            if self.block in ("post_ln", "one_norm"):
+                out += [(name, shape) for name, shape, _ in self._layer_tensors(i, L)]
                 continue
             if L.kind == "gla":
                 g = L.gla
@@ -711,6 +819,77 @@ class HybridConfig:
             one("norm2", (W,))
         return out
 
+    def joint_rows(self, L: LayerSpec) -> "JointRows":
+        """Row layout of the fused input projection of a 'one_norm' layer."""
+        if L.kind == "mlstm":
+            c = L.mlstm
+            mix = 2 * c.heads * (c.dim + c.vdim) + 2 * c.heads
+        else:
+            a = L.attn
+            mix = a.heads * a.dim + (a.kv_heads * (a.dim + a.vdim) if a.kv_from < 0 else 0)
+        mix = (mix + 7) // 8 * 8
+        f, at = L.mlp, mix
+        sg = router = -1
+        if f is not None and f.kind == "geglu":
+            at += 2 * f.ff
+        elif f is not None:
+            at += f.ff
+            if f.moe.shared_gate:
+                sg, at = at, at + 1
+            router, at = at, at + f.moe.outputs
+        return JointRows(mix, mix, sg, router, (at + 7) // 8 * 8)
+
+    def _layer_tensors(self, i: int, L: LayerSpec) -> list:
+        return self._postln_layer_tensors(i, L) if self.block == "post_ln" else self._joint_layer_tensors(i, L)
+
+    def _joint_layer_tensors(self, i: int, L: LayerSpec) -> list:
+        """(fused tensor, shape, [(checkpoint tensor or None = padding, rows)] in row order) of a layer of the 'one_norm'
+        block.  Everything that reads the layer's normed input is ONE fused tensor `in`: the mixer's projections, then the
+        dense feed-forward's gate and up, or the shared expert's up projection, its gate and the router.  The mixer's and
+        the whole tensor's rows are padded to multiples of eight (aligned rows of the projection buffer)."""
+        W, p, out = self.width, f"l{i}.", []
+        one = lambda name, shape: out.append((p + name, shape, [(p + name, shape[0])]))
+        J, f = self.joint_rows(L), L.mlp
+        if L.kind == "mlstm":
+            c = L.mlstm
+            nq, nv = c.heads * c.dim, c.heads * c.vdim
+            parts = [(p + "mix.q", nq), (p + "mix.k", nq), (p + "mix.v", nv), (p + "mix.g", nv), (p + "mix.i", c.heads),
+                     (p + "mix.f", c.heads)]
+        else:
+            a = L.attn
+            parts = [(p + "mix.q", a.heads * a.dim)]
+            if a.kv_from < 0:
+                parts += [(p + "mix.k", a.kv_heads * a.dim), (p + "mix.v", a.kv_heads * a.vdim)]
+        parts.append((None, J.mix - sum(n for _, n in parts)))
+        if f is not None and f.kind == "geglu":
+            parts += [(p + "mlp.gate", f.ff), (p + "mlp.up", f.ff)]
+        elif f is not None:
+            parts += [(p + "mlp.shared.up", f.ff)] if f.ff else []
+            parts += [(p + "mlp.shared.sg", 1)] if f.moe.shared_gate else []
+            parts += [(p + "mlp.router", f.moe.outputs)]
+        parts.append((None, J.total - sum(n for _, n in parts)))
+        out.append((p + "in", (J.total, W), parts))
+        if L.kind == "mlstm":
+            out.append((p + "mix.gate.b", (2 * c.heads,), [(p + "mix.i.b", c.heads), (p + "mix.f.b", c.heads)]))
+            one("mix.norm", (nv,)); one("mix.o", (W, nv))
+        else:
+            one("mix.q.norm", (a.dim,))
+            if a.kv_from < 0:
+                one("mix.k.norm", (a.dim,))
+            one("mix.o", (W, a.heads * a.vdim))
+        one("norm1", (W,))
+        if f is not None and f.kind == "geglu":
+            one("mlp.down", (W, f.ff))
+        elif f is not None:
+            e = f.moe
+            if e.correction:
+                one("mlp.correction", (e.outputs,))
+            out.append((p + "mlp.experts.up", (e.experts * e.ff, W), [(f"{p}mlp.e{k}.up", e.ff) for k in range(e.experts)]))
+            out.append((p + "mlp.experts.down", (e.experts * W, e.ff), [(f"{p}mlp.e{k}.down", W) for k in range(e.experts)]))
+            if f.ff:
+                out.append((p + "mlp.down", (W, f.ff), [(p + "mlp.shared.down", W)]))
+        return out
+
     def checkpoint_slices(self) -> dict[str, tuple[str, int, int]]:
         """checkpoint tensor name -> (fused tensor, first row, rows)."""
         m: dict[str, tuple[str, int, int]] = {}
@@ -718,7 +897,8 @@ class HybridConfig:
         def rows(fused, parts):
             at = 0
             for name, n in parts:
-                m[name] = (fused, at, n)
+                if name is not None:               # None: padding rows, which no checkpoint tensor fills
+                    m[name] = (fused, at, n)
                 at += n
         for i, L in self._own():
             p = f"l{i}."
@@ -726,8 +906,8 @@ class HybridConfig:
                 for fused, _, parts in self._stream_layer_tensors(i, L):
                     rows(fused, parts)
                 continue
-            if self.block == "post_ln":
-                for fused, _, parts in self._postln_layer_tensors(i, L):
+            if self.block in ("post_ln", "one_norm"):
+                for fused, _, parts in self._layer_tensors(i, L):
                     rows(fused, parts)
                 continue
             if L.kind == "gla":
@@ -826,6 +1006,8 @@ class HybridConfig:
             view.copy_((torch.randn(view.shape, generator=gen, device=view.device) * 0.1).to(view.dtype))
         elif leaf == "A_log":
             view.copy_(torch.log(torch.linspace(1.0, 4.0, view.numel())).to(view.dtype))
+        elif leaf == "correction":
+            view.copy_((torch.randn(view.shape, generator=gen, device=view.device) * 0.01).to(view.dtype))
         elif leaf in ("D",):
             view.fill_(1.0)
         elif leaf in ("b", "dt_bias"):
@@ -849,8 +1031,11 @@ class HybridConfig:
         return n
 
 
-def rotary_table(dims: int, base: float, scaling: tuple | None = None):
-    """(frequencies of the dims / 2 rotated pairs, factor on cos and sin).  Plain: base^(-2i/dims), factor 1.  With YaRN
+def rotary_table(dims: int, base: float, scaling: tuple | None = None, kind: str = "yarn"):
+    """(frequencies of the dims / 2 rotated pairs, factor on cos and sin).  Plain: base^(-2i/dims), factor 1.  With "bands"
+    scaling (factor, low turns, high turns, original length), as Llama 3.1's: pairs that complete more than `high` turns
+    over the original length keep their frequency, those below `low` turns are divided by `factor`, and in between the two
+    are mixed linearly in the number of turns; factor 1 on cos and sin.  With YaRN
     scaling (factor, original length, fast turns, slow turns): pairs that complete more than `fast` turns over the
     original length keep their frequency, those below `slow` turns are divided by `factor`, a linear ramp over the pair
     index in between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
@@ -858,6 +1043,14 @@ def rotary_table(dims: int, base: float, scaling: tuple | None = None):
     f = [base ** (-2.0 * i / dims) for i in range(half)]
     if not scaling or not half:
         return f, 1.0
+    if kind == "bands":
+        factor, low, high, orig = scaling
+        out = []
+        for w in f:
+            turns = orig * w / (2.0 * math.pi)
+            keep = 1.0 if turns > high else 0.0 if turns < low else (turns - low) / (high - low) if high > low else 1.0
+            out.append(keep * w + (1.0 - keep) * w / factor)
+        return out, 1.0
     factor, orig, fast, slow = scaling
     at = lambda turns: dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
     lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dims - 1)
@@ -878,6 +1071,8 @@ class _Rows:
         wide_gate, moe_pairs, moe_ff, moe_experts = 0, 0, 1, 1     # mLSTM gate heads; routed pairs per row, expert width
         wide_vfirst, wide_prep = 0, 0                               # values kept for later layers; gated-delta vectors
         for L in cfg.layers:
+            if cfg.block == "one_norm":
+                wide_p = max(wide_p, cfg.joint_rows(L).total)
             if L.kind == "attention":
                 a = L.attn
                 nq = a.heads * a.dim
@@ -940,7 +1135,7 @@ class _Rows:
                 if L.mlp.kind == "moe":
                     e = L.mlp.moe
                     wide_p = max(wide_p, e.top * 2 * e.ff)
-                    moe_pairs, moe_ff, moe_experts = max(moe_pairs, e.top), max(moe_ff, e.ff), max(moe_experts, e.experts)
+                    moe_pairs, moe_ff, moe_experts = max(moe_pairs, e.top), max(moe_ff, e.ff), max(moe_experts, e.outputs)
         f32 = dict(dtype=torch.float32, device=d)
         i32 = dict(dtype=torch.int32, device=d)
         self.n = n
@@ -955,7 +1150,8 @@ class _Rows:
         self.ob = torch.zeros(n * wide_o if any(eng.tc_attn.values()) else 1, dtype=torch.bfloat16, device=d)  # tcgen05 attention out
         self.ya = torch.zeros(n * wide_o, dtype=T, device=d)    # gated / normed input of the output projection
         self.yb = torch.zeros(n * wide_o2, dtype=T, device=d)
-        ny = max(n, 16 * min(n, 128)) * W                       # up to 16 split-K slices of a <= 128-row projection
+        # up to 16 split-K slices of a <= 128-row projection, or the two products of a joint output projection
+        ny = max(2 * n if cfg.block == "one_norm" else n, 16 * min(n, 128)) * W
         self.y0 = torch.zeros(ny, **f32)
         self.y1 = torch.zeros(ny, **f32)
         self.q = torch.zeros(n * wide_q, dtype=T, device=d)
@@ -1037,10 +1233,18 @@ class HybridEngine(EngineCore):
         for i, L in enumerate(cfg.layers):               # one cache / state per layer RUN, also where weights are shared
             if L.kind in ("attention", "sigmoid_delta"):
                 a = L.attn
-                self.k_pool[i] = torch.zeros(self.n_pages, a.kv_heads, PAGE_SIZE, a.dim, dtype=self.op_dtype, device=d)
-                self.v_pool[i] = torch.zeros(self.n_pages, a.kv_heads, PAGE_SIZE, a.vdim, dtype=self.op_dtype, device=d)
-                self.tc_attn[i] = False
-                f, self.rot_mag[i] = rotary_table(a.rot_dims, a.rot_base, a.rot_scaling)
+                # head size 128 in bf16 without window, sink or cap: the tcgen05 prompt kernel and the TMA decode kernel
+                self.tc_attn[i] = (cfg.block == "one_norm" and not self.f32 and a.dim == 128 and a.vdim == 128
+                                   and a.heads // a.kv_heads in (1, 2, 4, 8, 16))
+                if a.kv_from >= 0:                       # another run's cache: nothing of its own
+                    self.k_pool[i], self.v_pool[i] = self.k_pool[a.kv_from], self.v_pool[a.kv_from]
+                elif self.tc_attn[i]:                    # K and V pools adjacent
+                    pair = torch.zeros(2, self.n_pages, a.kv_heads, PAGE_SIZE, a.dim, dtype=self.op_dtype, device=d)
+                    self.k_pool[i], self.v_pool[i] = pair[0], pair[1]
+                else:
+                    self.k_pool[i] = torch.zeros(self.n_pages, a.kv_heads, PAGE_SIZE, a.dim, dtype=self.op_dtype, device=d)
+                    self.v_pool[i] = torch.zeros(self.n_pages, a.kv_heads, PAGE_SIZE, a.vdim, dtype=self.op_dtype, device=d)
+                f, self.rot_mag[i] = rotary_table(a.rot_dims, a.rot_base, a.rot_scaling, a.rot_scaling_kind)
                 self.rot_freq[i] = torch.tensor(f or [0.0], dtype=torch.float64, device=d)
                 if L.kind == "sigmoid_delta":
                     g = L.gdelta
@@ -1172,7 +1376,8 @@ class HybridEngine(EngineCore):
 
     def kv_bytes_per_token(self) -> int:
         e = 4 if self.f32 else 2
-        return (sum(L.attn.kv_heads * (L.attn.dim + L.attn.vdim) * e for L in self.cfg.layers if L.attn is not None)
+        return (sum(L.attn.kv_heads * (L.attn.dim + L.attn.vdim) * e for L in self.cfg.layers
+                    if L.attn is not None and L.attn.kv_from < 0)
                 + sum((L.latent.kv_rank + L.latent.rot_dim) * e for L in self.cfg.layers if L.latent is not None))
 
     # ---- GEMM dispatch ------------------------------------------------------------------------------------------------
@@ -1201,6 +1406,8 @@ class HybridEngine(EngineCore):
             return self._stream_layers(R, n, ns, max_q, row_pos, seg_pos0, trace)
         if cfg.block == "post_ln":
             return self._postln_layers(R, n, ns, max_q, row_pos, seg_pos0, trace)
+        if cfg.block == "one_norm":
+            return self._joint_layers(R, n, ns, max_q, row_pos, seg_pos0, trace, decode)
         W, eps, vec = cfg.width, cfg.eps, self.vec
         seg_start, seg_len, seg_slot = R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr()
         P, x, xa = R.P.data_ptr(), R.x.data_ptr(), R.xa.data_ptr()
@@ -1398,11 +1605,19 @@ class HybridEngine(EngineCore):
         """Matrix-memory LSTM: one projection [q | k | v | g | i | f]; the gates' running maximum is walked first (fp32),
         which turns the cell into S <- keep S + take k v^T, the recurrence prl_decay_scan runs; the normaliser rides along
         as one more value column (v with a one appended)."""
-        c, lib, st, vec, f32, W = L.mlstm, self.lib, self._st, self.vec, int(self.f32), self.cfg.width
-        H, nq, nv = c.heads, c.heads * c.dim, c.heads * c.vdim
-        ld, P = 2 * nq + 2 * nv + 2 * H, R.P.data_ptr()
-        seg_start, seg_len, seg_slot, ns = segs
+        c, vec, W = L.mlstm, self.vec, self.cfg.width
+        nv, ld = c.heads * c.vdim, 2 * c.heads * (c.dim + c.vdim + 1)
         self._mm(R.xa, W, w + "mix.in", ld, R.P, n)
+        self._mlstm_cell(R, n, i, c, w, segs, pieces, ld)
+        k0 = self._mm(R.ya, nv, w + "mix.o", W, R.y0, n, split=True)
+        self._close(R, n, R.y0, k0, post_gain=vec[w + "norm1b"] if L.sandwich else vec[w + "norm1"],
+                    next_gain=self._next_gain(i, True))
+
+    def _mlstm_cell(self, R, n, i, c, w, segs, pieces, ld) -> None:
+        """From the projections [q | k | v | g | i | f] (R.P, rows ld apart) to the cell's normed and gated output R.ya."""
+        lib, st, vec, f32 = self.lib, self._st, self.vec, int(self.f32)
+        H, nq, nv, P = c.heads, c.heads * c.dim, c.heads * c.vdim, R.P.data_ptr()
+        seg_start, seg_len, seg_slot, ns = segs
         gb = vec[w + "mix.gate.b"].data_ptr()
         _lib.check(lib.prl_mlstm_gates(P, ld, 2 * nq + 2 * nv, 2 * nq + 2 * nv + H, gb, gb + 4 * H, c.gate_cap, H, seg_start,
                                        seg_len, seg_slot, ns, self.mlstm_m[i].data_ptr(), R.gates.data_ptr(),
@@ -1418,9 +1633,6 @@ class HybridEngine(EngineCore):
                                           R.o.data_ptr(), H * dv, st))
         _lib.check(lib.prl_mlstm_out(R.o.data_ptr(), n, H, c.vdim, R.minv.data_ptr(), c.den_eps, P + 4 * (2 * nq + nv), ld,
                                      vec[w + "mix.norm"].data_ptr(), self.cfg.eps, R.ya.data_ptr(), f32, st))
-        k0 = self._mm(R.ya, nv, w + "mix.o", W, R.y0, n, split=True)
-        self._close(R, n, R.y0, k0, post_gain=vec[w + "norm1b"] if L.sandwich else vec[w + "norm1"],
-                    next_gain=self._next_gain(i, True))
 
     def _attn_lightning_mixer(self, R, n, i, L, w, segs, pieces, max_q, row_pos, seg_pos0) -> None:
         """Softmax attention (values = keys, per-head unit norms, capped scores, window + kept first tokens) beside
@@ -1519,6 +1731,114 @@ class HybridEngine(EngineCore):
             _lib.check(lib.prl_gate_heads(R.o.data_ptr(), 1, no, P + 4 * (nq + nk + nv), ld, n, a.heads, a.vdim, R.ya.data_ptr(),
                                           f32, st))
         return self._mm(R.ya, no, w + "mix.o", W, R.y0, n, split=True)
+
+    # ---- the 'one_norm' block: x <- x + (mixer(h) + ff(h)), h = norm(x) --------------------------------------------------
+    def _joint_layers(self, R, n, ns, max_q, row_pos, seg_pos0, trace=None, decode=False) -> None:
+        """Layer program of the 'one_norm' block.  On entry R.x holds the embedding; R.xa always holds the next layer's
+        normed input.  Per layer: ONE input projection for the mixer, the (shared) feed-forward and the router; the mixer
+        and the feed-forward's activation from its columns; the routed experts; ONE product that adds both branches'
+        output projections in its accumulator; the closing kernel (routed slices, residual, next norm)."""
+        cfg, lib, st, vec, f32, W = self.cfg, self.lib, self._st, self.vec, int(self.f32), self.cfg.width
+        segs = (R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr(), ns)
+        n_sub = 0 if decode else R.n_sub
+        pieces = (R.seg_sub[0].data_ptr(), R.seg_sub[1].data_ptr(), R.sub[0].data_ptr(), R.sub[1].data_ptr(), n_sub,
+                  R.scratch.data_ptr(), R.cdec.data_ptr()) if n_sub else None
+        x, xa = R.x.data_ptr(), R.xa.data_ptr()
+        if cfg.layers:
+            _lib.check(lib.prl_rmsnorm_rows(x, None, vec[f"l{cfg.layers[0].weights_of}.norm1"].data_ptr(), cfg.eps, n, W, xa, f32, st))
+        for i, L in enumerate(cfg.layers):
+            w, f, J = f"l{L.weights_of}.", L.mlp, cfg.joint_rows(L)
+            # gate and up through the activation epilogue of their own GEMM when the batch is compute-bound; a decode step
+            # streams all rows of the input projection in one launch that fills the SMs
+            fused = (f is not None and f.kind == "geglu" and n > 128 and f.ff % 128 == 0 and W % 8 == 0 and W >= 64
+                     and not (self.f32 or self.force_plain_gemm or self.unfused_glu))
+            ld = J.mix if fused else J.total
+            self._mm(R.xa, W, w + "in", ld, R.P, n)
+            if fused:
+                up = self.arena.ptr(w + "in") + J.ff * W * 2
+                _lib.check(lib.prl_gemm_geglu_f32(xa, W, up, W, n, f.ff, W, R.act.data_ptr(), f.ff, st))
+            elif f is not None and f.ff:
+                _lib.check(lib.prl_ff_act(R.P.data_ptr(), ld, J.ff, n, f.ff, int(f.kind == "geglu"), J.shared_gate,
+                                          R.act.data_ptr(), f32, st))
+            routed, top, experts = None, 1, 1
+            if f is not None and f.kind == "moe":
+                routed, top, experts = self._choose_and_run_experts(R, n, w, f.moe, ld, J.router), f.moe.top, f.moe.experts
+            if L.kind == "mlstm":
+                self._mlstm_cell(R, n, i, L.mlstm, w, segs, pieces, ld)
+                y, no = R.ya, L.mlstm.heads * L.mlstm.vdim
+            else:
+                y = self._attn_core(R, n, i, L, w, segs, max_q, row_pos, seg_pos0, ld, decode)
+                no = L.attn.heads * L.attn.vdim
+            if f is not None and f.ff:
+                k0 = self._mm_dual(y, no, w + "mix.o", R.act, f.ff, w + "mlp.down", W, R.y0, n)
+            else:
+                k0 = self._mm(y, no, w + "mix.o", W, R.y0, n, split=True)
+            nxt = vec[f"l{cfg.layers[i + 1].weights_of}.norm1"].data_ptr() if i + 1 < len(cfg.layers) else None
+            _lib.check(lib.prl_joint_close(R.y0.data_ptr(), k0, None if routed is None else routed.data_ptr(), top,
+                                           *((R.sel.data_ptr(), R.wsel.data_ptr()) if routed is not None else (None, None)),
+                                           experts, nxt, cfg.eps, n, W, x, xa, f32, st))
+            if trace is not None:
+                trace.append(R.x[:n * W].view(n, W).clone())
+
+    def _mm_dual(self, src1, K1, w1, src2, K2, w2, N, out, n) -> int:
+        """out [slices][n][N] (fp32) whose sum is src1[n, K1] @ W1[N, K1]^T + src2[n, K2] @ W2[N, K2]^T: one tcgen05 GEMM
+        that accumulates both products, or the two CUDA-core products as two slices.  Returns the number of slices."""
+        lib, st, p1, p2 = self.lib, self._st, self.arena.ptr(w1), self.arena.ptr(w2)
+        if self.f32 or self.force_plain_gemm or K1 % 8 or K2 % 8 or min(K1, K2) < 64:
+            for src, K, wp, o in ((src1, K1, p1, 0), (src2, K2, p2, n * N)):
+                _lib.check(lib.prl_gemm_any(src.data_ptr(), int(self.f32), K, wp, int(self.f32), K, n, N, K,
+                                            out.data_ptr() + 4 * o, N, st))
+            return 2
+        if n <= 128:
+            k = int(lib.prl_gemm_dual_split_k(n, N, K1, K2))
+            _lib.check(lib.prl_gemm_bf16_dual(p1, src1.data_ptr(), K1, p2, src2.data_ptr(), K2, n, N, k, out.data_ptr(), st))
+            return k
+        _lib.check(lib.prl_gemm_tn_dual(src1.data_ptr(), p1, K1, src2.data_ptr(), p2, K2, n, N, out.data_ptr(), N, st))
+        return 1
+
+    def _choose_and_run_experts(self, R, n, w, e, ld, off_router) -> torch.Tensor:
+        """Squared-ReLU experts chosen from the router's columns of R.P; returns [top][n][W] fp32 (R.moe_out), in which the
+        slices of choices that hand the input through (R.sel >= experts) are not written."""
+        lib, st, W, f32 = self.lib, self._st, self.cfg.width, int(self.f32)
+        corr = self.vec[w + "mlp.correction"].data_ptr() if e.correction else None
+        _lib.check(lib.prl_moe_choose(R.P.data_ptr() + 4 * off_router, ld, corr, n, e.experts, e.outputs, e.top, e.groups,
+                                      e.keep_groups, R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(),
+                                      R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), st))
+        table = (R.perm.data_ptr(), R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), int(lib.prl_moe_max_tiles(n * e.top, e.experts)))
+        _lib.check(lib.prl_moe_gemm_relu2(R.xa.data_ptr(), f32, W, n, self.arena.ptr(w + "mlp.experts.up"), f32, e.ff * W, W,
+                                          *table, e.ff, W, R.wsel.data_ptr(), R.moe_act.data_ptr(), e.ff, st))
+        _lib.check(lib.prl_moe_gemm(R.moe_act.data_ptr(), f32, e.ff, 0, self.arena.ptr(w + "mlp.experts.down"), f32, W * e.ff,
+                                    e.ff, *table, W, e.ff, R.moe_out.data_ptr(), W, 1, st))
+        return R.moe_out
+
+    def _attn_core(self, R, n, i, L, w, segs, max_q, row_pos, seg_pos0, ld, decode) -> torch.Tensor:
+        """Softmax attention from the projections [q | k | v] (R.P, rows ld apart; [q] alone for a layer that reads another
+        run's cache) to the concatenated heads in the operand type.  Returns the buffer that holds them."""
+        a, lib, st, vec, f32 = L.attn, self.lib, self._st, self.vec, int(self.f32)
+        seg_start, seg_len, seg_slot, ns = segs
+        own = a.kv_from < 0
+        nq, nk = a.heads * a.dim, a.kv_heads * a.dim
+        kv = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr())
+        bt = (self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE)
+        _lib.check(lib.prl_attn_front(R.P.data_ptr(), ld, 0, nq, nq + nk, n, a.heads, a.kv_heads if own else 0, a.dim, a.vdim, None,
+                                      None, None, int(a.head_norm), vec[w + "mix.q.norm"].data_ptr(),
+                                      vec[w + "mix.k.norm"].data_ptr() if own else None, a.dim, self.cfg.eps, a.rot_dims,
+                                      self.rot_freq[i].data_ptr(), self.rot_mag[i], 0, 0, None, None, row_pos.data_ptr(),
+                                      R.row_slot.data_ptr(), *bt, R.q.data_ptr(), *(kv if own else (None, None)), f32, st))
+        if self.tc_attn[i] and not self.force_plain_attn:
+            if decode:
+                _lib.check(lib.prl_paged_attn_decode(R.q.data_ptr(), kv[0], self.n_pages, 1, 0, *bt[:2], self.seq_lens.data_ptr(),
+                                                     n, a.heads, a.kv_heads, a.dim, PAGE_SIZE, self.attn_splits[i], a.scale,
+                                                     R.ob.data_ptr(), self.attn_ws.data_ptr(), self.attn_ws.numel(), st))
+            else:
+                _lib.check(lib.prl_paged_attn_prefill_tc(R.q.data_ptr(), n, kv[0], self.n_pages, 1, 0, *bt[:2], seg_start, seg_len,
+                                                         seg_pos0.data_ptr(), seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim,
+                                                         PAGE_SIZE, a.scale, R.ob.data_ptr(), st))
+            return R.ob
+        _lib.check(lib.prl_attn_any_sink(R.q.data_ptr(), *kv, a.vdim, f32, *bt, seg_start, seg_len, seg_pos0.data_ptr(), seg_slot, ns,
+                                         max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.keep_first, a.softcap,
+                                         None, 1, R.ya.data_ptr(), st))
+        return R.ya
 
     def _latent_direct_mixer(self, R, n, i, L, w, segs, max_q, row_pos, seg_pos0) -> int:
         """Latent attention whose query comes straight from the layer's input: ONE projection [q | dkv | g].  As in

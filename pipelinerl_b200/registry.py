@@ -118,6 +118,11 @@ def _kolotar_config(config: dict, shapes: dict):
     return HybridConfig.from_kolotar(config, shapes)
 
 
+def _futetar_config(config: dict, shapes: dict):
+    from .hybrid import HybridConfig
+    return HybridConfig.from_futetar(config, shapes)
+
+
 def _hybrid_engine():
     from .hybrid import HybridEngine
     return HybridEngine
@@ -128,6 +133,7 @@ register(Family("Povurax", _povurax_config, _hybrid_engine, (torch.bfloat16, tor
 register(Family("Belelorn", _belelorn_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 register(Family("Pametar", _pametar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 register(Family("Kolotar", _kolotar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
+register(Family("Futetar", _futetar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 
 
 def parse_dtype(name: str) -> torch.dtype:
