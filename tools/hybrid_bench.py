@@ -104,6 +104,23 @@ def kolotar_config(s):
                 layers=[[att, att, lat, par][i % 4] for i in range(s["layers"])])
 
 
+def futetar_config(s):
+    """Eight layers: a matrix-memory cell with a dense feed-forward, attention with a routed one, a cell with a routed one,
+    attention that reads the second layer's cache with a dense one, twice.  Cells and attention heads as in the Belelorn
+    model (heads of 128, cells 128 x 256), dense ff equal, routed ones of the same active width (four of sixteen experts of
+    ff / 8, four identity outputs, a shared expert of ff / 2)."""
+    W, ff = s["width"], s["ff"]
+    cell = dict(type="mlstm", mixer=dict(heads=W // 256, dim=128, vdim=256, gate_cap=15.0))
+    att = dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5,
+               rot=dict(base=5e5, dims=128, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
+    dense = dict(kind="dense", ff=ff)
+    routed = dict(kind="moe", router=dict(experts=16, top=4, identity=4, groups=dict(count=4, keep=3)), expert=dict(ff=ff // 8),
+                  shared=dict(ff=ff // 2))
+    block = [dict(cell, mlp=dense), dict(type="attention", mixer=att, mlp=routed), dict(cell, mlp=routed),
+             dict(type="attention", mixer=dict(att, kv_from=1), mlp=dense)]
+    return dict(architecture="Futetar", vocab=s["vocab"], width=W, norm=dict(eps=1e-5), layers=[block[i % 4] for i in range(s["layers"])])
+
+
 def peaks():
     try:
         p = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())
@@ -612,6 +629,138 @@ def run_kolotar(sizes, prompt, context, batch, steps, warm, kernels=True, e2e=Tr
     return res
 
 
+def run_futetar(sizes, prompt, context, batch, steps, warm, kernels=True, e2e=True, others=True):
+    """Futetar beside Belelorn (the closest design: the same memory cell, attention heads of the same size, dense and routed
+    feed-forwards with a shared expert) and the Qwen2 engine at equal width / depth / active ff / attention heads."""
+    from pipelinerl_b200.engine import DecodeEngine
+    from pipelinerl_b200.hybrid import HybridConfig, HybridEngine
+    from pipelinerl_b200.model import ModelConfig, ParamArena
+    dev = torch.device("cuda:0")
+    timer = Timer()
+    res = {}
+    for name in sizes:
+        s = SIZES[name]
+        kw = dict(max_batch=batch, max_seq_len=max(prompt, context) + 256, max_new_tokens=warm + steps + 8, device=dev,
+                  prefill_chunk=1024)
+        entry = {}
+        models = {"futetar": (HybridEngine, HybridConfig.from_futetar(futetar_config(s)))}
+        if others:
+            models = {"qwen2": (DecodeEngine, ModelConfig(vocab_size=s["vocab"], hidden_size=s["width"], intermediate_size=s["ff"],
+                                                          num_layers=s["layers"], num_q_heads=s["heads"], num_kv_heads=s["kv"])),
+                      "belelorn": (HybridEngine, HybridConfig.from_belelorn(belelorn_config(s))), **models}
+        for model, (cls, cfg) in models.items():
+            eng = cls(cfg, ParamArena(cfg, dev).init_random(seed=1), **kw)
+            if e2e:
+                entry[model] = end_to_end(eng, s["vocab"], prompt, context, batch, steps, warm)
+                entry[model]["params_M"] = round(cfg.num_params() / 1e6)
+            if kernels and model in ("futetar", "belelorn"):
+                table = kernel_table_futetar if model == "futetar" else kernel_table_belelorn
+                entry[f"kernels_{model}" if model != "futetar" else "kernels"] = table(eng, s, batch, 1024, timer)
+            del eng
+            torch.cuda.empty_cache()
+        if e2e and others:
+            for other in ("qwen2", "belelorn"):
+                entry[f"futetar_over_{other}"] = {k: round(entry["futetar"][f"{k}_tokens_per_s"] / entry[other][f"{k}_tokens_per_s"], 3)
+                                                  for k in ("prefill", "decode")}
+        res[name] = entry
+    return res
+
+
+def kernel_table_futetar(eng, s, batch, chunk, timer):
+    """The parts of the Futetar layers alone, at the decode shape (`batch` one-token segments at position 2047) and the
+    prefill shape (one segment of `chunk` rows whose sequence already holds `chunk` tokens): the engine's own methods on its
+    buffers; weight streams and row kernels against the measured copy bandwidth, products of many rows and attention
+    against the measured bf16 GEMM rate, the recurrence against the SMs' fp32 FMA rate."""
+    from pipelinerl_b200 import _lib
+    from pipelinerl_b200.cache import PAGE_SIZE
+    from pipelinerl_b200.hybrid import _Rows
+    lib, cfg = eng.lib, eng.cfg
+    hbm, tflops, how = peaks()
+    fma_tflops = 148 * 128 * 2 * 1.965e9 / 1e12
+    W = cfg.width
+    kinds = {(L.kind, L.mlp.kind): i for i, L in reversed(list(enumerate(cfg.layers)))}
+    ci, ai, di = kinds["mlstm", "geglu"], kinds["attention", "moe"], kinds["attention", "geglu"]
+    LC, LA, LD = cfg.layers[ci], cfg.layers[ai], cfg.layers[di]
+    c, a, e, F, Fs = LC.mlstm, LA.attn, LA.mlp.moe, LC.mlp.ff, LA.mlp.ff
+    JC, JA = cfg.joint_rows(LC), cfg.joint_rows(LA)
+    wc, wa = f"l{LC.weights_of}.", f"l{LA.weights_of}."
+    nv, no = c.heads * c.vdim, a.heads * a.vdim
+    out = {"peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "fp32_fma_tflops": round(fma_tflops, 1), "source": how}}
+    i32 = dict(dtype=torch.int32, device=eng.dev)
+    ctx = 2047
+    pages_per = (ctx + PAGE_SIZE) // PAGE_SIZE
+    for b in range(batch):
+        eng.block_table[b, :pages_per].copy_(torch.arange(1 + b * pages_per, 1 + (b + 1) * pages_per, **i32))
+    for pools in (eng.k_pool, eng.v_pool):
+        for pool in pools.values():
+            pool.normal_(0, 0.5)
+    eng.seq_lens.fill_(ctx + 1)
+    for shape, n, ns in (("decode", batch, batch), ("prefill", chunk, 1)):
+        decode = shape == "decode"
+        R = _Rows(eng, n, pieces=not decode)
+        R.P.normal_(0, 0.5); R.xa.normal_(0, 0.5); R.x.normal_(0, 0.5); R.ya.normal_(0, 0.5); R.act.normal_(0, 0.5)
+        pos0 = ctx if decode else chunk
+        pieces = None
+        if decode:
+            R.seg.copy_(torch.stack([torch.arange(n, **i32), torch.ones(n, **i32), torch.full((n,), ctx, **i32), torch.arange(n, **i32)]))
+            R.row_slot.copy_(torch.arange(n, **i32)); R.row_pos.fill_(ctx)
+        else:
+            R.seg[:, :1].copy_(torch.tensor([[0], [n], [pos0], [0]], **i32))
+            R.row_slot.zero_(); R.row_pos.copy_(torch.arange(pos0, pos0 + n, **i32)); R.row_back.copy_(torch.arange(n, **i32))
+            step = eng.piece_tokens
+            n_sub = (n + step - 1) // step
+            R.sub[0, :n_sub].copy_(torch.arange(0, n, step, **i32))
+            R.sub[1, :n_sub].copy_(torch.tensor([min(step, n - k) for k in range(0, n, step)], **i32))
+            R.seg_sub[:, :1].copy_(torch.tensor([[0], [n_sub]], **i32))
+            pieces = (R.seg_sub[0].data_ptr(), R.seg_sub[1].data_ptr(), R.sub[0].data_ptr(), R.sub[1].data_ptr(), n_sub,
+                      R.scratch.data_ptr(), R.cdec.data_ptr())
+        eng._st = st = _lib.stream_ptr()
+        segs = (R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr(), ns)
+        max_q = 1 if decode else n
+        keys = (ctx + 1) * n if decode else n * pos0 + n * (n + 1) // 2
+        t, hb, fl = {}, {}, {}
+        ldc = JC.total if decode else JC.mix
+        t["in_product"] = timer.events(lambda: eng._mm(R.xa, W, wc + "in", ldc, R.P, n))
+        hb["in_product"], fl["in_product"] = (ldc + n) * W * 2 + n * ldc * 4, 2.0 * n * ldc * W
+        if not decode:
+            up = eng.arena.ptr(wc + "in") + JC.ff * W * 2
+            t["geglu_product"] = timer.events(lambda: _lib.check(lib.prl_gemm_geglu_f32(R.xa.data_ptr(), W, up, W, n, F, W, R.act.data_ptr(), F, st)))
+            fl["geglu_product"] = 4.0 * n * F * W
+        t["ff_act"] = timer.events(lambda: _lib.check(lib.prl_ff_act(R.P.data_ptr(), JA.total, JA.ff, n, Fs, 0, JA.shared_gate, R.act.data_ptr(), 0, st)))
+        hb["ff_act"] = n * Fs * 6
+        t["cell"] = timer.events(lambda: eng._mlstm_cell(R, n, ci, c, wc, segs, pieces, ldc))
+        hb["cell"] = 2 * ns * c.heads * c.dim * (c.vdim + 1) * 4 + n * (2 * c.heads * (c.dim + c.vdim) * 4 + nv * 2)
+        t["attention"] = timer.events(lambda: eng._attn_core(R, n, ai, LA, wa, segs, max_q, R.row_pos, R.seg[2], JA.total, decode))
+        hb["attention"], fl["attention"] = (ns * (ctx + 1) if decode else pos0 + n) * a.kv_heads * (a.dim + a.vdim) * 2, 2.0 * keys * a.heads * (a.dim + a.vdim)
+        wd = f"l{LD.weights_of}."
+        t["attention_other_cache"] = timer.events(lambda: eng._attn_core(R, n, di, LD, wd, segs, max_q, R.row_pos, R.seg[2], JA.total, decode))
+        hb["attention_other_cache"], fl["attention_other_cache"] = hb["attention"], fl["attention"]
+        t["dual_product"] = timer.events(lambda: eng._mm_dual(R.ya, nv, wc + "mix.o", R.act, F, wc + "mlp.down", W, R.y0, n))
+        hb["dual_product"], fl["dual_product"] = (nv + F) * (W + n) * 2 + n * W * 4, 2.0 * n * (nv + F) * W
+        t["routed_experts"] = timer.events(lambda: eng._choose_and_run_experts(R, n, wa, e, JA.total, JA.router))
+        live = int((R.sel[:n * e.top] < e.experts).sum())
+        used = len(torch.unique(R.sel[:n * e.top][R.sel[:n * e.top] < e.experts]))
+        hb["routed_experts"], fl["routed_experts"] = used * 2 * e.ff * W * 2 + live * (W * 6 + e.ff * 4), 4.0 * live * e.ff * W
+        nxt = eng.vec["final.norm"].data_ptr()
+        t["joint_close"] = timer.events(lambda: _lib.check(lib.prl_joint_close(R.y0.data_ptr(), 1, R.moe_out.data_ptr(), e.top, R.sel.data_ptr(),
+                                                                               R.wsel.data_ptr(), e.experts, nxt, cfg.eps, n, W, R.x.data_ptr(),
+                                                                               R.xa.data_ptr(), 0, st)))
+        hb["joint_close"] = n * W * (4 * 3 + 2) + live * W * 4
+        row = {k: {"us": round(v * 1e3, 1)} for k, v in t.items()}
+        for k in t:
+            if decode or k in ("ff_act", "joint_close"):
+                row[k]["of_hbm"] = round(hb[k] / t[k] / 1e6 / hbm, 3)
+            elif k in fl:
+                row[k]["of_bf16_peak"] = round(fl[k] / t[k] / 1e9 / tflops, 3)
+        row["cell"]["of_fp32_fma"] = round(5.0 * n * c.heads * c.dim * (c.vdim + 1) / t["cell"] / 1e9 / fma_tflops, 3)
+        out[shape] = row
+        del R
+    eng.block_table.zero_()
+    for b in range(batch):
+        eng.states.reset(b)
+    return out
+
+
 def kernel_table_kolotar(eng, s, batch, chunk, timer):
     """The parts of the three Kolotar layer kinds alone, at the decode shape (`batch` one-token segments at position 2047)
     and the prefill shape (one segment of `chunk` rows whose sequence already holds `chunk` tokens): the engine's own
@@ -850,12 +999,15 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--only-kernels", action="store_true", help="skip the end-to-end runs (a small case for a profiler)")
-    ap.add_argument("--design", default="povurax", choices=["povurax", "belelorn", "pametar", "kolotar"], help="which hybrid design is measured")
+    ap.add_argument("--design", default="povurax", choices=["povurax", "belelorn", "pametar", "kolotar", "futetar"], help="which hybrid design is measured")
     ap.add_argument("--alone", action="store_true", help="--design belelorn: skip the Qwen2 and Povurax runs beside it")
     a = ap.parse_args()
     from pipelinerl_b200 import _lib
     before = _lib.launch_count()
-    if a.design == "kolotar":
+    if a.design == "futetar":
+        res = run_futetar(a.sizes.split(","), a.prompt, a.context, a.batch, a.steps, a.warmup, kernels=not a.no_kernels,
+                          e2e=not a.only_kernels, others=not a.alone)
+    elif a.design == "kolotar":
         res = run_kolotar(a.sizes.split(","), a.prompt, a.context, a.batch, a.steps, a.warmup, kernels=not a.no_kernels,
                           e2e=not a.only_kernels, others=not a.alone)
     elif a.design == "pametar":
