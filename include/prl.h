@@ -692,7 +692,8 @@ int prl_ff_act(const float* P, int64_t ld, int32_t off, int32_t n, int32_t F, in
                int32_t f32, prl_stream_t stream);
 /* C = A1 B1^T + A2 B2^T in one accumulation (two branches of one residual): many rows, and the token step's split-K form */
 int prl_gemm_tn_dual(const void* A1_bf16, const void* B1_bf16, int64_t K1, const void* A2_bf16, const void* B2_bf16, int64_t K2,
-                     int64_t M, int64_t N, float* C, int64_t ldc, prl_stream_t stream);
+                     int64_t M, int64_t N, int32_t split_k, float* C /* [split_k][M][N] */, prl_stream_t stream);
+int prl_gemm_tn_dual_split_k(int64_t M, int64_t N, int64_t K1, int64_t K2, int32_t most);
 int prl_gemm_dual_split_k(int64_t M, int64_t N, int64_t K1, int64_t K2);
 int prl_gemm_bf16_dual(const void* W1, const void* X1, int64_t K1, const void* W2, const void* X2, int64_t K2, int64_t M,
                        int64_t N, int32_t split_k, float* partials, prl_stream_t stream);
@@ -727,14 +728,24 @@ int prl_decay_scan(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, fl
                    const float* const_decay, int32_t heads, int32_t dk, int32_t dv, const int32_t* seg_start,
                    const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg, float* state, float* out,
                    int64_t ld_out, prl_stream_t stream);
+/* (pieces: ones = 1 makes the last of the dv value columns constant one, not stored in xval) */
 int prl_decay_scan_split(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, float q_scale, const float* xval,
-                         int64_t ld_x, int32_t off_x, const float* gates, int64_t ld_g, int32_t off_g,
+                         int64_t ld_x, int32_t off_x, int32_t ones, const float* gates, int64_t ld_g, int32_t off_g,
                          const float* const_decay, int32_t heads, int32_t dk, int32_t dv, const int32_t* seg_slot,
                          int32_t n_seg, const int32_t* seg_sub0, const int32_t* seg_nsub, const int32_t* sub_start,
                          const int32_t* sub_len, int32_t n_sub, float* scratch, float* piece_decay, float* state,
                          float* out, int64_t ld_out, prl_stream_t stream);
 /* matrix-memory LSTM: stabilised exponential gates (keep, take) per head and token with the running maximum m carried
  * in m_state[slot][head]; values with a one appended per head; output normaliser, head norm, gain and sigmoid gate */
+int prl_mlstm_gates_scan(const float* P, int64_t ldp, int32_t off_i, int32_t off_f, const float* bias_i, const float* bias_f,
+                         float cap, int32_t H, const int32_t* seg_start, const int32_t* seg_len, const int32_t* seg_slot,
+                         int32_t n_seg, float* m_state, float* gates, float* minv, prl_stream_t stream);
+/* one token of the whole cell (gates, state, normaliser, head norm, output gate) for segments of one row */
+int prl_mlstm_step(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, int32_t off_v, int32_t off_g, int32_t off_i,
+                   int32_t off_f, const float* bias_i, const float* bias_f, float cap, float q_scale, float den_eps,
+                   const float* gain, float eps, int32_t heads, int32_t dk, int32_t vdim, const int32_t* seg_start,
+                   const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg, float* m_state, float* state, void* out,
+                   int32_t f32, prl_stream_t stream);
 int prl_mlstm_gates(const float* P, int64_t ldp, int32_t off_i, int32_t off_f, const float* bias_i, const float* bias_f,
                     float cap, int32_t H, const int32_t* seg_start, const int32_t* seg_len, const int32_t* seg_slot,
                     int32_t n_seg, float* m_state, float* gates, float* minv, prl_stream_t stream);

@@ -39,6 +39,8 @@ struct TnParams {
   int k_wrap;        // k-blocks >= k_wrap are k-blocks (kb - k_wrap) of the SECOND pair of tensor maps: C = A B^T + A2 B2^T in one
                      // accumulation (fp32-equivalent lm_head: A2 = A, B = bf16 hi part, B2 = bf16 lo residual; two branches
                      // that join the same sum: each with its own operand and weight)
+  int split;         // > 1 (fp32 output, plain epilogue): the k-blocks of a tile are shared by `split` clusters' worth of work, slice s of
+                     // C = rows s * M .. of an output [split][M][ldc] that the consumer sums
   int m_tiles, n_tiles;
   int a_mn, b_mn;    // operand stored MN-major: A as [K, M] / B as [K, N] row-major (no transposed copy needed)
   void* C;
@@ -83,7 +85,15 @@ __device__ __forceinline__ float gelu_tanh(float z) {
   return z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
+// k-blocks of work item t: all of them, or the item's share of a split tile (items of a tile are neighbours)
+__device__ __forceinline__ void k_range(int t, const TnParams& p, int& kb0, int& kb1) {
+  const int split = p.split > 1 ? p.split : 1, s = t % split;
+  kb0 = (int)((int64_t)p.kblocks * s / split);
+  kb1 = (int)((int64_t)p.kblocks * (s + 1) / split);
+}
+
 __device__ __forceinline__ void tile_coords(int t, const TnParams& p, int& tm, int& tn) {
+  if (p.split > 1) t /= p.split;
   const int per_group = kGroupM * p.n_tiles;
   const int g = t / per_group;
   const int first_m = g * kGroupM;
@@ -110,7 +120,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
   const uint32_t rank = ptx::cluster_ctarank();
   const int n_clusters = (int)gridDim.x >> 1;
   const int cluster = (int)blockIdx.x >> 1;
-  const int total_tiles = p.m_tiles * p.n_tiles;
+  const int total_tiles = p.m_tiles * p.n_tiles * (p.split > 1 ? p.split : 1);
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -144,9 +154,11 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
       for (int t = cluster; t < total_tiles; t += n_clusters) {
         int tm, tn;
         tile_coords(t, p, tm, tn);
+        int kb0, kb1;
+        k_range(t, p, kb0, kb1);
         const int a_row = tm * kTile + (int)rank * kHalf;
         const int b_row = p.swiglu_I ? tn * kHalf + (int)rank * (int)p.swiglu_I : tn * kTile + (int)rank * kHalf;
-        for (int kb = 0; kb < p.kblocks; ++kb, ++it) {
+        for (int kb = kb0; kb < kb1; ++kb, ++it) {
           const int s = it % kStages;
           const uint32_t ph = (uint32_t)((it / kStages) & 1);
           ptx::mbar_wait(empty_bar(s), ph ^ 1u);
@@ -184,7 +196,9 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
         ptx::mbar_wait(acc_empty_bar(acc), acc_ph ^ 1u);  // both CTAs' epilogues have drained this accumulator
         ptx::tc_fence_after_sync();
         const uint32_t d_tmem = tmem_base + (uint32_t)(acc * kTile);
-        for (int kb = 0; kb < p.kblocks; ++kb, ++it) {
+        int kb0, kb1;
+        k_range(t, p, kb0, kb1);
+        for (int kb = kb0; kb < kb1; ++kb, ++it) {
           const int s = it % kStages;
           const uint32_t ph = (uint32_t)((it / kStages) & 1);
           ptx::mbar_wait(full_bar(s), ph);
@@ -196,7 +210,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
 #pragma unroll
           for (int k = 0; k < kBK / 16; ++k)
             ptx::mma_bf16_ss_2sm(d_tmem, a_desc + a_step * (uint64_t)k, b_desc + b_step * (uint64_t)k, idesc,
-                                 (kb > 0 || k > 0) ? 1u : 0u);
+                                 (kb > kb0 || k > 0) ? 1u : 0u);
           ptx::tc_commit_2sm(empty_bar(s), 3);
         }
         ptx::tc_commit_2sm(acc_full_bar(acc), 3);
@@ -419,7 +433,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
           continue;
         }
         if (p.c_f32) {
-          float* cp = reinterpret_cast<float*>(p.C) + row * p.ldc + col;
+          float* cp = reinterpret_cast<float*>(p.C) + (row + (p.split > 1 ? (int64_t)(t % p.split) * p.M : 0)) * p.ldc + col;
           if (full && ((p.ldc & 3) == 0)) {
 #pragma unroll
             for (int j = 0; j < 32; j += 4) {
@@ -605,11 +619,22 @@ extern "C" int prl_gemm_ex(const void* A, int64_t lda, int32_t a_mn_major, const
 }
 
 // Two products in one accumulation, C[M, N] (fp32) = A1[M, K1] * B1[N, K1]^T + A2[M, K2] * B2[N, K2]^T: the output projections of two
-// branches that are added to the same residual.
+// branches that are added to the same residual.  split_k slices [split_k][M][N] (prl_gemm_tn_dual_split_k: as many, up to `most`,
+// as give idle clusters a share of the k-blocks, eight each at least).
+extern "C" int prl_gemm_tn_dual_split_k(int64_t M, int64_t N, int64_t K1, int64_t K2, int32_t most) {
+  const int64_t tiles = ((M + kTile - 1) / kTile) * ((N + kTile - 1) / kTile), clusters = num_sms() / 2;
+  const int64_t kb = (K1 + kBK - 1) / kBK + (K2 + kBK - 1) / kBK;
+  int64_t k = tiles > 0 ? clusters / tiles : 1;
+  k = k > most ? most : k;
+  k = k > kb / 8 ? kb / 8 : k;
+  return (int)(k < 1 ? 1 : k);
+}
+
 extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, const void* A2, const void* B2, int64_t K2, int64_t M,
-                                int64_t N, float* C, int64_t ldc, prl_stream_t stream_) {
+                                int64_t N, int32_t split_k, float* C, prl_stream_t stream_) {
   PRL_CHECK_ARG(A1 && B1 && A2 && B2 && C, "prl_gemm_tn_dual: NULL argument");
-  PRL_CHECK_ARG(M >= 1 && N >= 1 && K1 >= 8 && K2 >= 8 && K1 % 8 == 0 && K2 % 8 == 0 && ldc >= N,
+  PRL_CHECK_ARG(split_k >= 1 && split_k <= (K1 + kBK - 1) / kBK + (K2 + kBK - 1) / kBK, "prl_gemm_tn_dual: bad split %d", split_k);
+  PRL_CHECK_ARG(M >= 1 && N >= 1 && K1 >= 8 && K2 >= 8 && K1 % 8 == 0 && K2 % 8 == 0,
                 "prl_gemm_tn_dual: need M, N >= 1 and K1, K2 multiples of 8 (M=%lld N=%lld K1=%lld K2=%lld)", (long long)M, (long long)N,
                 (long long)K1, (long long)K2);
   TnParams p = {};
@@ -618,7 +643,7 @@ extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, cons
   p.kblocks = p.k_wrap + (int)((K2 + kBK - 1) / kBK);
   p.m_tiles = (int)((M + kTile - 1) / kTile);
   p.n_tiles = (int)((N + kTile - 1) / kTile);
-  p.C = C; p.ldc = ldc; p.c_f32 = 1; p.alpha = 1.f;
+  p.C = C; p.ldc = N; p.c_f32 = 1; p.alpha = 1.f; p.split = split_k;
   CUtensorMap ta, tb, ta2, tb2;
   int rc = make_tmap_2d_bf16(&ta, A1, (uint64_t)K1, (uint64_t)M, (uint64_t)K1 * 2, kBK, kHalf);
   if (rc) return rc;
@@ -631,7 +656,7 @@ extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, cons
   const int smem = kStages * kStageBytes + 1024 + 8 * (2 * kStages + 4) + 16;
   static SmemAttr smem_attr = {};
   PRL_CUDA(ensure_smem(gemm_tn_kernel<false>, smem, smem_attr));
-  const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles;
+  const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles * split_k;
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
   gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta2, tb2, p);

@@ -413,6 +413,99 @@ __global__ void sublayer_close_kernel(const float* __restrict__ y0, int64_t ld0,
   for (int c = threadIdx.x; c < W; c += blockDim.x) stf(xa, r * W + c, next_gain ? b0[c] * in * next_gain[c] : b0[c]);
 }
 
+// The close of a layer whose branches carry no norms of their own (prl_joint_close), rows of a multiple of four channels:
+// a thread keeps NC groups of four channels of the row in registers from the sum to the normed store.
+template <typename T> __device__ __forceinline__ float4 ld4(const T* p);
+template <> __device__ __forceinline__ float4 ld4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+template <typename T> __device__ __forceinline__ void st4(T* p, float4 v);
+template <> __device__ __forceinline__ void st4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  uint2 u;
+  __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+  h[0] = __floats2bfloat162_rn(v.x, v.y);
+  h[1] = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+__device__ __forceinline__ void add4(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+
+template <typename T, int NC>
+__global__ void joint_close_kernel(const float* __restrict__ y0, int ns0, int64_t stride, const float* __restrict__ y1, int top,
+                                   const int32_t* __restrict__ sel, const float* __restrict__ wsel, int experts,
+                                   const float* __restrict__ next_gain, float eps, int W, float* __restrict__ x, T* __restrict__ xa) {
+  pdl_wait();
+  __shared__ float red[32];
+  const int64_t r = blockIdx.x, at = r * W;
+  const int n4 = W / 4;
+  uint32_t live = 0;                   // choices that are experts; the others hand the input through
+  float w_pass = 0.f;
+  if (y1)
+    for (int k = 0; k < top; ++k) {
+      if (sel[(int64_t)k * gridDim.x + r] < experts) live |= 1u << k;
+      else w_pass += wsel[(int64_t)k * gridDim.x + r];
+    }
+  float4 v[NC];
+#pragma unroll
+  for (int u = 0; u < NC; ++u) v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int k = 0; k < ns0; ++k)
+#pragma unroll
+    for (int u = 0; u < NC; ++u) {
+      const int c = threadIdx.x + u * blockDim.x;
+      if (c < n4) add4(v[u], ld4(y0 + k * stride + at + 4 * c));
+    }
+  if (y1) {
+    float4 b[NC];
+#pragma unroll
+    for (int u = 0; u < NC; ++u) b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) {
+      if (!(live >> k & 1u)) continue;
+#pragma unroll
+      for (int u = 0; u < NC; ++u) {
+        const int c = threadIdx.x + u * blockDim.x;
+        if (c < n4) add4(b[u], ld4(y1 + k * stride + at + 4 * c));
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < NC; ++u) {
+      const int c = threadIdx.x + u * blockDim.x;
+      if (c < n4 && w_pass != 0.f) {
+        const float4 h = ld4(xa + at + 4 * c);
+        b[u].x = fmaf(w_pass, h.x, b[u].x); b[u].y = fmaf(w_pass, h.y, b[u].y);
+        b[u].z = fmaf(w_pass, h.z, b[u].z); b[u].w = fmaf(w_pass, h.w, b[u].w);
+      }
+      add4(v[u], b[u]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c < n4) {
+      add4(v[u], ld4(x + at + 4 * c));
+      st4(x + at + 4 * c, v[u]);
+      ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    }
+  }
+  float inv = 1.f;
+  if (next_gain) inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c >= n4) continue;
+    float4 o = v[u];
+    if (next_gain) {
+      const float4 g = ld4(next_gain + 4 * c);
+      o = make_float4(o.x * inv * g.x, o.y * inv * g.y, o.z * inv * g.z, o.w * inv * g.w);
+    }
+    st4(xa + at + 4 * c, o);
+  }
+}
+
 // Attention front end with PER-HEAD unit norms: q and k get their biases (NULL: none), every head of q and of k is
 // divided by its own root mean square over `dim` and multiplied by a gain (NULL: none; indexed head * dim + channel);
 // q goes to the query buffer, k into the paged cache.  The value written beside it is either the key as projected
@@ -557,6 +650,60 @@ __global__ void mlstm_gates_kernel(const float* __restrict__ P, int64_t ldp, int
     }
     if (lane == 0) m_state[(int64_t)slot * H + h] = m;
   }
+}
+
+// The same for long segments: one CTA per (head, segment), a thread per token.  A stretch of tokens acts on the running
+// maximum as m -> max(m + F, I), and two stretches compose to (F1 + F2, max(I1 + F2, I2)), so the walk is a scan over the
+// CTA's tokens (shuffles inside a warp, then over the warps' totals).  Equal to the token-by-token walk up to rounding.
+__global__ void __launch_bounds__(1024) mlstm_gates_scan_kernel(const float* __restrict__ P, int64_t ldp, int off_i, int off_f,
+                                                                const float* __restrict__ bias_i, const float* __restrict__ bias_f,
+                                                                float cap, int H, const int32_t* __restrict__ seg_start,
+                                                                const int32_t* __restrict__ seg_len, const int32_t* __restrict__ seg_slot,
+                                                                float* __restrict__ m_state, float* __restrict__ gates,
+                                                                float* __restrict__ minv) {
+  pdl_wait();
+  __shared__ float wF[32], wI[32], last;
+  const int h = blockIdx.x, seg = blockIdx.y;
+  const int len = seg_len[seg];
+  if (len <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
+  const int64_t row0 = seg_start[seg];
+  float* ms = m_state + (int64_t)seg_slot[seg] * H + h;
+  float m0 = *ms;
+  for (int t0 = 0; t0 < len; t0 += blockDim.x) {
+    const int t = t0 + tid;
+    float gi = -INFINITY, gf = 0.f;              // past the end: leaves the maximum as it is
+    if (t < len) {
+      const float* pr = P + (row0 + t) * ldp;
+      const float zi = pr[off_i + h] + bias_i[h], zf = pr[off_f + h] + bias_f[h];
+      gi = cap > 0.f ? cap * tanhf(zi / cap) : zi;
+      gf = logsigmoid_g(cap > 0.f ? cap * tanhf(zf / cap) : zf);
+    }
+    float F = gf, I = gi;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pF = __shfl_up_sync(0xffffffffu, F, o), pI = __shfl_up_sync(0xffffffffu, I, o);
+      if (lane >= o) { I = fmaxf(pI + F, I); F = pF + F; }
+    }
+    __syncthreads();                             // the previous round is done with wF, wI and last
+    if (lane == 31) { wF[warp] = F; wI[warp] = I; }
+    __syncthreads();
+    float m_in = m0;                             // the maximum in front of this warp's tokens
+    for (int w = 0; w < warp; ++w) m_in = fmaxf(m_in + wF[w], wI[w]);
+    const float m = fmaxf(m_in + F, I);
+    float m_prev = __shfl_up_sync(0xffffffffu, m, 1);
+    if (lane == 0) m_prev = m_in;
+    if (t < len) {
+      const int64_t o = (row0 + t) * H + h;
+      gates[2 * o] = expf(gf + m_prev - m);
+      gates[2 * o + 1] = expf(gi - m);
+      minv[o] = expf(-m);
+    }
+    if (tid == (nw << 5) - 1) last = m;
+    __syncthreads();
+    m0 = last;
+  }
+  if (tid == 0) *ms = m0;
 }
 
 // Values of the scan with a ONE appended per head: [row][head][dv + 1], so that the recurrence also carries the
@@ -925,6 +1072,20 @@ extern "C" int prl_joint_close(const float* y0, int32_t n_split0, const float* y
                                int32_t experts, const float* next_gain, float eps, int32_t n, int32_t W, float* x, void* xa,
                                int32_t f32, prl_stream_t st) {
   PRL_CHECK_ARG(!y1 || (sel && wsel && experts >= 1), "prl_joint_close: routed slices need their choices and weights");
+  PRL_CHECK_ARG(y0 && x && xa && n >= 1 && W >= 1 && n_split0 >= 1 && (!y1 || top >= 1), "prl_joint_close: bad argument");
+  const uintptr_t bits = (uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)x | (uintptr_t)xa | (uintptr_t)next_gain;
+  if (W % 4 == 0 && W <= 16384 && (bits & 15) == 0 && (!y1 || top <= 32)) {
+    const int n4 = W / 4, nc = n > 256 ? (n4 <= 256 ? 1 : n4 <= 1024 ? 2 : 4) : (n4 <= 1024 ? 1 : 4);
+    const int th = ((n4 + nc - 1) / nc + 31) / 32 * 32;
+    const int64_t stride = (int64_t)n * W;
+#define PRL_JC(T, NC) PRL_CUDA(launch_pdl((joint_close_kernel<T, NC>), dim3(n), dim3(th), (size_t)0, (cudaStream_t)st, y0, n_split0, stride, y1, top, sel, wsel, experts, \
+                                          next_gain, eps, W, x, (T*)xa))
+    if (f32) { if (nc == 1) PRL_JC(float, 1); else if (nc == 2) PRL_JC(float, 2); else PRL_JC(float, 4); }
+    else { if (nc == 1) PRL_JC(bf16, 1); else if (nc == 2) PRL_JC(bf16, 2); else PRL_JC(bf16, 4); }
+#undef PRL_JC
+    PRL_LAUNCH_CHECK();
+    return PRL_OK;
+  }
   return sublayer_close_impl(y0, W, n_split0, nullptr, 1.f, y1, W, y1 ? top : 1, nullptr, 1.f, nullptr, nullptr, 1, next_gain, eps,
                              n, W, y1 ? sel : nullptr, wsel, experts, x, xa, f32, st);
 }
@@ -988,6 +1149,18 @@ extern "C" int prl_mlstm_gates(const float* P, int64_t ldp, int32_t off_i, int32
   int th = 32 * H;
   th = th > 256 ? 256 : th;
   PRL_CUDA(launch_pdl(mlstm_gates_kernel, dim3(n_seg), dim3(th), (size_t)0, (cudaStream_t)st, P, ldp, off_i, off_f, bias_i, bias_f, cap, H, seg_start, seg_len, seg_slot, m_state, gates, minv));
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+// prl_mlstm_gates for batches with long segments (prompt portions): a scan over the tokens instead of a walk, equal up to rounding
+extern "C" int prl_mlstm_gates_scan(const float* P, int64_t ldp, int32_t off_i, int32_t off_f, const float* bias_i,
+                                    const float* bias_f, float cap, int32_t H, const int32_t* seg_start, const int32_t* seg_len,
+                                    const int32_t* seg_slot, int32_t n_seg, float* m_state, float* gates, float* minv,
+                                    prl_stream_t st) {
+  PRL_CHECK_ARG(P && bias_i && bias_f && seg_start && seg_len && seg_slot && m_state && gates && minv && H >= 1 && n_seg >= 1 &&
+                n_seg <= 65535 && cap >= 0.f, "prl_mlstm_gates_scan: bad argument");
+  PRL_CUDA(launch_pdl(mlstm_gates_scan_kernel, dim3(H, n_seg), dim3(1024), (size_t)0, (cudaStream_t)st, P, ldp, off_i, off_f, bias_i, bias_f, cap, H, seg_start, seg_len, seg_slot, m_state, gates, minv));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }

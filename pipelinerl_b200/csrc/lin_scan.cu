@@ -356,6 +356,202 @@ struct SplitArgs {
   int r;                                                 // key channels per key lane in the state layout
 };
 
+// ---- 1. for SCALAR recurrences: a piece as three products ---------------------------------------------------------------
+// With one decay a_t and one input scale b_t per token, let w_tj = b_j prod_(j < s <= t) a_s (j <= t).  Then, inside a piece,
+//   o_t^local = sum_j w_tj (q_t . k_j) v_j        and        L = sum_j w_Tj k_j v_j^T     (T: the piece's last token),
+// i.e. two products over tokens and one over the piece's outer products, register-blocked on the CUDA cores in fp32
+// (everything that enters the recurrence stays fp32), instead of a dependent walk over the tokens.  w is formed column by
+// column as running products, so nothing is divided and no logarithms are summed.  CTA = (piece, head, 128 value columns).
+// `ones` = 1: value column dv - 1 is constant one and not stored in xval; where the others are a multiple of four, its two
+// results are row sums that the first column tile forms on the side.
+// Also writes the piece's total decay (piece_decay_kernel's table).
+constexpr int kCC = 128;                 // value columns per CTA
+constexpr int kCD = 32;                  // key channels per round of the q . k product
+constexpr int kTS = kPiece + 4;          // padded stride of token-minor tiles
+constexpr int kVS = kCC + 4;
+constexpr int kChunkSmem = (2 * kPiece * kTS + kPiece * kVS + 2 * kPiece) * (int)sizeof(float);
+
+__global__ void __launch_bounds__(256) chunk_kernel(ScanArgs a, SplitArgs p, int ones, int vec4) {
+  pdl_wait();
+  extern __shared__ __align__(16) float csm[];
+  float* As = csm;                        // [token j][token t]: w_tj, then w_tj (q_t . k_j)
+  float* Qs = As + kPiece * kTS;          // [channel][token] (kCD rows), with Ks behind it; later [token][channel], 64 channels
+  float* Ks = Qs + kCD * kTS;
+  float* Vs = Qs + kPiece * kTS;          // [token][column]
+  float* keep = Vs + kPiece * kVS;        // [kPiece] decays, later the weights w_Tj
+  float* take = keep + kPiece;
+  const int sub = blockIdx.x, h = blockIdx.y, vt = blockIdx.z, tid = threadIdx.x;
+  const int len = p.sub_len[sub], dk = a.dk, dv = a.dv, r = p.r;
+  const int64_t row0 = p.sub_start[sub];
+  const int nx = dv - (ones ? 1 : 0);                       // columns stored in xval
+  const bool side = ones && nx % 4 == 0 && vt == 0;         // this CTA forms the constant column's results as row sums
+  const float* qb = a.qvec + a.off_q + h * dk;
+  const float* kb = a.kvec + a.off_k + h * dk;
+  const float* xb = a.xval + a.off_x + h * nx;
+  if (tid < kPiece) {
+    const bool in = tid < len;
+    const float* gp = a.dt_raw ? a.dt_raw + (row0 + (in ? tid : 0)) * a.ld_dt + a.off_dt + 2 * h : nullptr;
+    keep[tid] = in ? (gp ? gp[0] : a.a_log[h]) : 1.f;       // past the end: the state stays as it is
+    take[tid] = in ? (gp ? gp[1] : 1.f) : 0.f;
+  }
+  // values: columns vt * 128 .. of every token (zero past the piece's end and past the last column)
+  for (int e = tid; e < kPiece * (kCC / 4); e += 256) {
+    const int t = e / (kCC / 4), c = (e % (kCC / 4)) * 4, col = vt * kCC + c;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t < len) {
+      const float* src = xb + (row0 + t) * a.ld_x + col;
+      if (vec4 && col + 4 <= nx) {
+        v = *reinterpret_cast<const float4*>(src);
+      } else {
+        float u[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) u[j] = col + j < nx ? src[j] : ((ones && col + j == nx) ? 1.f : 0.f);
+        v = make_float4(u[0], u[1], u[2], u[3]);
+      }
+    }
+    *reinterpret_cast<float4*>(Vs + t * kVS + c) = v;
+  }
+  __syncthreads();
+  if (tid < kPiece) {                      // column j of w: zero above the diagonal, then a running product
+    float w = take[tid];
+    for (int t = 0; t < kPiece; ++t) {
+      if (t > tid) w *= keep[t];
+      As[tid * kTS + t] = t >= tid ? w : 0.f;
+    }
+  }
+  if (vt == 0 && tid >= 64) {              // the piece's total decay
+    float d = 1.f;
+    for (int t = 0; t < len; ++t) d *= keep[t];
+    for (int i = tid - 64; i < kKeyLanes * r; i += 192) p.cdec[((int64_t)sub * a.heads + h) * kKeyLanes * r + i] = d;
+  }
+  // ---- q . k: 4 x 4 (t, j) pairs per thread
+  const int tx = tid % 16, ty = tid / 16;
+  float qk[4][4] = {};                     // [t][j]
+  for (int d0 = 0; d0 < dk; d0 += kCD) {
+    __syncthreads();
+    for (int e = tid; e < kPiece * (kCD / 4); e += 256) {
+      const int t = e / (kCD / 4), d = (e % (kCD / 4)) * 4;
+      float q4[4] = {0.f, 0.f, 0.f, 0.f}, k4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (t < len) {
+        const float* qs = qb + (row0 + t) * a.ld_q + d0 + d;
+        const float* ks = kb + (row0 + t) * a.ld_k + d0 + d;
+        if (vec4 && d0 + d + 4 <= dk) {
+          *reinterpret_cast<float4*>(q4) = *reinterpret_cast<const float4*>(qs);
+          *reinterpret_cast<float4*>(k4) = *reinterpret_cast<const float4*>(ks);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (d0 + d + j < dk) { q4[j] = qs[j]; k4[j] = ks[j]; }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { Qs[(d + j) * kTS + t] = q4[j]; Ks[(d + j) * kTS + t] = k4[j]; }
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int d = 0; d < kCD; ++d) {
+      const float4 qv = *reinterpret_cast<const float4*>(Qs + d * kTS + ty * 4);
+      const float4 kv = *reinterpret_cast<const float4*>(Ks + d * kTS + tx * 4);
+      const float qq[4] = {qv.x, qv.y, qv.z, qv.w}, kk[4] = {kv.x, kv.y, kv.z, kv.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) qk[i][j] = fmaf(qq[i], kk[j], qk[i][j]);
+    }
+  }
+  __syncthreads();
+  if (tid < kPiece) keep[tid] = As[tid * kTS + kPiece - 1];       // w_Tj (tokens past the end do not decay it)
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    float4* ap = reinterpret_cast<float4*>(As + (tx * 4 + j) * kTS + ty * 4);
+    float4 w = *ap;
+    *ap = make_float4(w.x * qk[0][j], w.y * qk[1][j], w.z * qk[2][j], w.w * qk[3][j]);
+  }
+  __syncthreads();
+  // ---- o^local: 4 tokens x 8 columns per thread (columns 4 tx .. and 64 + 4 tx ..)
+  auto product = [&](const float* left, float (&acc)[4][8]) {     // left: [token j][kTS], four rows 4 ty .. of the result
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < kPiece; ++j) {
+      const float4 l4 = *reinterpret_cast<const float4*>(left + j * kTS + ty * 4);
+      const float4 v0 = *reinterpret_cast<const float4*>(Vs + j * kVS + tx * 4);
+      const float4 v1 = *reinterpret_cast<const float4*>(Vs + j * kVS + 64 + tx * 4);
+      const float ll[4] = {l4.x, l4.y, l4.z, l4.w}, vv[8] = {v0.x, v0.y, v0.z, v0.w, v1.x, v1.y, v1.z, v1.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(ll[i], vv[e], acc[i][e]);
+    }
+  };
+  float acc[4][8];
+  product(As, acc);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = ty * 4 + i;
+    if (t >= len) continue;
+    float* o = a.out + (row0 + t) * a.ld_out + h * dv;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int col = vt * kCC + (e < 4 ? 0 : 64) + tx * 4 + (e & 3);
+      if (col < (side || (ones && nx % 4 == 0) ? nx : dv)) o[col] = acc[i][e] * a.q_scale;
+    }
+  }
+  if (side && tid < len) {
+    float s = 0.f;
+    for (int j = 0; j < kPiece; ++j) s += As[j * kTS + tid];
+    a.out[(row0 + tid) * a.ld_out + h * dv + nx] = s * a.q_scale;
+  }
+  // ---- L: key channels in blocks of 64 (the state's padding channels and columns are written as zeros)
+  const int nv4 = (dv + 3) / 4;
+  float* st = p.scratch + (int64_t)sub * a.state_slot_stride + (int64_t)h * r * nv4 * 32;
+  for (int d0 = 0; d0 < kKeyLanes * r; d0 += 64) {
+    __syncthreads();
+    for (int e = tid; e < kPiece * 16; e += 256) {
+      const int t = e / 16, d = (e % 16) * 4;
+      float k4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (t < len) {
+        const float* ks = kb + (row0 + t) * a.ld_k + d0 + d;
+        const float w = keep[t];
+        if (vec4 && d0 + d + 4 <= dk) {
+          *reinterpret_cast<float4*>(k4) = *reinterpret_cast<const float4*>(ks);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) k4[j] *= w;
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (d0 + d + j < dk) k4[j] = w * ks[j];
+        }
+      }
+      *reinterpret_cast<float4*>(Qs + t * kTS + d) = make_float4(k4[0], k4[1], k4[2], k4[3]);
+    }
+    __syncthreads();
+    product(Qs, acc);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = d0 + ty * 4 + i;
+      if (d >= kKeyLanes * r) continue;
+      const int dg = d / r, ri = d % r;
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        const int c4 = vt * (kCC / 4) + g * 16 + tx;
+        if (c4 < ((ones && nx % 4 == 0) ? nx / 4 : nv4))
+          *reinterpret_cast<float4*>(st + (((int64_t)ri * nv4 + c4) * kKeyLanes + dg) * 4) =
+              make_float4(acc[i][4 * g], acc[i][4 * g + 1], acc[i][4 * g + 2], acc[i][4 * g + 3]);
+      }
+    }
+    if (side && tid < 64 && d0 + tid < kKeyLanes * r) {
+      float s = 0.f;
+      for (int j = 0; j < kPiece; ++j) s += Qs[j * kTS + tid];
+      const int d = d0 + tid;
+      *reinterpret_cast<float4*>(st + (((int64_t)(d % r) * nv4 + nx / 4) * kKeyLanes + d / r) * 4) = make_float4(s, 0.f, 0.f, 0.f);
+    }
+  }
+}
+
 template <int MODE>
 __global__ void __launch_bounds__(256) piece_decay_kernel(ScanArgs a, SplitArgs p) {
   constexpr bool SSD = MODE == kSsd, SCL = MODE == kScalar;
@@ -502,15 +698,26 @@ __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
 }
 
 template <int SSD>
-int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st) {
+int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st, int ones = 0) {
   p.r = plan_r(a.dk);
-  ScanArgs pieces = a;                 // 1. every piece from a zero state into its scratch slot
-  pieces.seg_start = p.sub_start; pieces.seg_len = p.sub_len; pieces.seg_slot = nullptr;
-  pieces.state = p.scratch; pieces.zero_init = 1;
-  const int rc = launch_scan<SSD>(pieces, n_sub, st);
-  if (rc != PRL_OK) return rc;
-  PRL_CUDA(launch_pdl(piece_decay_kernel<SSD>, dim3(n_sub, a.heads), dim3(256), (size_t)0, st, a, p));
-  PRL_LAUNCH_CHECK();
+  if (SSD == kScalar) {
+    const int nx = a.dv - ones;
+    const int vec4 = a.dk % 4 == 0 && nx % 4 == 0 && a.ld_k % 4 == 0 && a.ld_q % 4 == 0 && a.ld_x % 4 == 0 && a.off_k % 4 == 0 &&
+                     a.off_q % 4 == 0 && a.off_x % 4 == 0 && aligned16(a.kvec) && aligned16(a.qvec) && aligned16(a.xval);
+    const int cols = (ones && nx % 4 == 0 && nx > 0) ? nx : a.dv;
+    static SmemAttr attr = {};
+    PRL_CUDA(ensure_smem(chunk_kernel, kChunkSmem, attr));
+    PRL_CUDA(launch_pdl(chunk_kernel, dim3(n_sub, a.heads, (cols + kCC - 1) / kCC), dim3(256), (size_t)kChunkSmem, st, a, p, ones, vec4));
+    PRL_LAUNCH_CHECK();
+  } else {
+    ScanArgs pieces = a;               // 1. every piece from a zero state into its scratch slot
+    pieces.seg_start = p.sub_start; pieces.seg_len = p.sub_len; pieces.seg_slot = nullptr;
+    pieces.state = p.scratch; pieces.zero_init = 1;
+    const int rc = launch_scan<SSD>(pieces, n_sub, st);
+    if (rc != PRL_OK) return rc;
+    PRL_CUDA(launch_pdl(piece_decay_kernel<SSD>, dim3(n_sub, a.heads), dim3(256), (size_t)0, st, a, p));
+    PRL_LAUNCH_CHECK();
+  }
   const int nv4 = (a.dv + 3) / 4, per_head = p.r * nv4 * 32;
   PRL_CUDA(launch_pdl(carry_kernel, dim3((per_head + 1023) / 1024, a.heads, n_seg), dim3(256), (size_t)0, st, a, p));
   PRL_LAUNCH_CHECK();
@@ -650,7 +857,7 @@ static int decay_scan_impl(const float* P, int64_t ldp, int32_t off_q, int32_t o
                            int64_t ld_x, int32_t off_x, const float* gates, int64_t ld_g, int32_t off_g,
                            const float* const_decay, int32_t heads, int32_t dk, int32_t dv, const int32_t* seg_start,
                            const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg, float* state, float* out,
-                           int64_t ld_out, const SplitArgs* split, int32_t n_sub, prl_stream_t st) {
+                           int64_t ld_out, const SplitArgs* split, int32_t n_sub, prl_stream_t st, int32_t ones = 0) {
   PRL_CHECK_ARG(P && xval && (gates || const_decay) && seg_start && seg_len && seg_slot && state && out,
                 "prl_decay_scan: NULL argument");
   PRL_CHECK_ARG(heads >= 1 && dk >= 1 && dk <= 256 && dv >= 1 && n_seg >= 1 && n_seg <= 65535,
@@ -666,7 +873,7 @@ static int decay_scan_impl(const float* P, int64_t ldp, int32_t off_q, int32_t o
   a.q_scale = q_scale;
   a.dt_raw = gates; a.ld_dt = ld_g; a.off_dt = off_g; a.groups = heads;
   a.a_log = const_decay;
-  if (split) return launch_split<kScalar>(a, n_seg, *split, n_sub, (cudaStream_t)st);
+  if (split) return launch_split<kScalar>(a, n_seg, *split, n_sub, (cudaStream_t)st, ones);
   return launch_scan<kScalar>(a, n_seg, (cudaStream_t)st);
 }
 
@@ -679,16 +886,165 @@ extern "C" int prl_decay_scan(const float* P, int64_t ldp, int32_t off_q, int32_
                          seg_start, seg_len, seg_slot, n_seg, state, out, ld_out, nullptr, 0, st);
 }
 
-// The same with every segment cut into side-by-side pieces (see prl_gla_scan_split for the tables).
+// The same with every segment cut into side-by-side pieces (see prl_gla_scan_split for the tables).  ones = 1: the last of the
+// dv value columns is constant one and not stored (xval has heads * (dv - 1) columns).
 extern "C" int prl_decay_scan_split(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, float q_scale,
-                                    const float* xval, int64_t ld_x, int32_t off_x, const float* gates, int64_t ld_g,
+                                    const float* xval, int64_t ld_x, int32_t off_x, int32_t ones, const float* gates, int64_t ld_g,
                                     int32_t off_g, const float* const_decay, int32_t heads, int32_t dk, int32_t dv,
                                     const int32_t* seg_slot, int32_t n_seg, const int32_t* seg_sub0,
                                     const int32_t* seg_nsub, const int32_t* sub_start, const int32_t* sub_len,
                                     int32_t n_sub, float* scratch, float* cdec, float* state, float* out, int64_t ld_out,
                                     prl_stream_t st) {
   SplitArgs p;
+  PRL_CHECK_ARG(ones == 0 || (ones == 1 && dv >= 2), "prl_decay_scan_split: a constant column beside at least one stored one");
   PRL_CHECK_ARG(split_args(p, seg_sub0, seg_nsub, sub_start, sub_len, n_sub, scratch, cdec), "prl_decay_scan_split: bad piece tables");
   return decay_scan_impl(P, ldp, off_q, off_k, q_scale, xval, ld_x, off_x, gates, ld_g, off_g, const_decay, heads, dk, dv,
-                         sub_start, sub_len, seg_slot, n_seg, state, out, ld_out, &p, n_sub, st);
+                         sub_start, sub_len, seg_slot, n_seg, state, out, ld_out, &p, n_sub, st, ones);
+}
+
+// ---- one token of the matrix-memory LSTM cell -----------------------------------------------------------------------------
+// A decode step of the whole cell in one kernel: gates and running maximum, S <- keep S + take k [v; 1]^T, o = S^T q over the
+// normaliser, the head's RMS norm, gain and output gate, written in the operand type.  CTA = (head, segment): thread (column
+// group, key lane) as in the scan, so that the state streams through registers as whole lines; the sums are those of the scan
+// kernel and prl_mlstm_out in the same order.  Segments that are not exactly one row long are skipped.
+namespace prl {
+namespace {
+struct CellArgs {
+  const float* P; int64_t ldp; int off_q, off_k, off_v, off_g, off_i, off_f;
+  const float* bias_i; const float* bias_f; float cap, q_scale, den_eps;
+  const float* gain; float eps;
+  int heads, dk, vdim;
+  const int32_t* seg_start; const int32_t* seg_len; const int32_t* seg_slot;
+  float* m_state; float* state; int64_t state_slot_stride;
+};
+
+constexpr int kStepThreads = 320;
+template <typename T, int R>
+__global__ void __launch_bounds__(kStepThreads, 2) mlstm_step_kernel(CellArgs a, T* __restrict__ out) {
+  pdl_wait();
+  extern __shared__ float sm[];
+  constexpr int QS = R + 1;                       // padded stride of one key lane's channels
+  float* qs = sm;                                 // [8][QS]
+  float* ks = qs + kKeyLanes * QS;
+  float* os = ks + kKeyLanes * QS;                // [nv4 * 4]
+  __shared__ float red[32];
+  const int h = blockIdx.x, seg = blockIdx.y, tid = threadIdx.x;
+  if (a.seg_len[seg] != 1) return;
+  const int64_t row = a.seg_start[seg];
+  const int slot = a.seg_slot[seg], dv = a.vdim + 1, nv4 = (dv + 3) / 4, groups = nv4 * kKeyLanes;
+  const float* pr = a.P + row * a.ldp;
+  float* st = a.state + (int64_t)slot * a.state_slot_stride + (int64_t)h * R * nv4 * 32;
+  for (int d = tid; d < kKeyLanes * R; d += blockDim.x) {
+    const int o = (d / R) * QS + d % R;
+    qs[o] = d < a.dk ? pr[a.off_q + h * a.dk + d] : 0.f;
+    ks[o] = d < a.dk ? pr[a.off_k + h * a.dk + d] : 0.f;
+  }
+  const float zi = pr[a.off_i + h] + a.bias_i[h], zf = pr[a.off_f + h] + a.bias_f[h];
+  const float gi = a.cap > 0.f ? a.cap * tanhf(zi / a.cap) : zi;
+  const float gf = logsigmoid_f(a.cap > 0.f ? a.cap * tanhf(zf / a.cap) : zf);
+  const float m_prev = a.m_state[(int64_t)slot * a.heads + h];
+  const float m_new = fmaxf(gf + m_prev, gi);
+  const float keep = expf(gf + m_prev - m_new), take = expf(gi - m_new);
+  __syncthreads();
+  constexpr int RB = R < 8 ? R : 8;               // state rows in flight per thread
+  for (int g0 = 0; g0 < groups; g0 += blockDim.x) {
+    const int g = g0 + tid, c4 = g / kKeyLanes, dg = g % kKeyLanes;
+    const bool on = g < groups;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (on) {
+      float xin[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int c = 4 * c4 + j;
+        xin[j] = (c < a.vdim ? pr[a.off_v + h * a.vdim + c] : (c == a.vdim ? 1.f : 0.f)) * take;
+      }
+      float4* sp = reinterpret_cast<float4*>(st) + g;           // row i of the state: + i * groups
+#pragma unroll
+      for (int i0 = 0; i0 < R; i0 += RB) {
+        float4 s4[RB];
+#pragma unroll
+        for (int i = 0; i < RB; ++i) s4[i] = sp[(int64_t)(i0 + i) * groups];
+#pragma unroll
+        for (int i = 0; i < RB; ++i) {
+          const float k = ks[dg * QS + i0 + i], q = qs[dg * QS + i0 + i];
+          s4[i].x = fmaf(keep, s4[i].x, k * xin[0]); acc[0] = fmaf(s4[i].x, q, acc[0]);
+          s4[i].y = fmaf(keep, s4[i].y, k * xin[1]); acc[1] = fmaf(s4[i].y, q, acc[1]);
+          s4[i].z = fmaf(keep, s4[i].z, k * xin[2]); acc[2] = fmaf(s4[i].z, q, acc[2]);
+          s4[i].w = fmaf(keep, s4[i].w, k * xin[3]); acc[3] = fmaf(s4[i].w, q, acc[3]);
+          sp[(int64_t)(i0 + i) * groups] = s4[i];
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], 1);
+      acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], 2);
+      acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], 4);
+    }
+    if (on && dg == 0) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) os[4 * c4 + j] = acc[j] * a.q_scale;
+    }
+  }
+  __syncthreads();
+  const float den = fmaxf(fabsf(os[a.vdim]), expf(-m_new)) + a.den_eps;
+  const int th = min((a.vdim + 31) / 32 * 32, 256);             // threads that sum: prl_mlstm_out's block
+  float ss = 0.f;
+  if (tid < th)
+    for (int c = tid; c < a.vdim; c += th) {
+      const float v = os[c] / den;
+      ss += v * v;
+    }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < th / 32; ++w) tot += red[w];
+  const float inv = 1.f / sqrtf(tot / (float)a.vdim + a.eps);
+  for (int c = tid; c < a.vdim; c += blockDim.x) {
+    const int ch = h * a.vdim + c;
+    const float gate = 1.f / (1.f + expf(-pr[a.off_g + ch]));
+    out[row * a.heads * a.vdim + ch] = T(os[c] / den * inv * a.gain[ch] * gate);
+  }
+  if (tid == 0) a.m_state[(int64_t)slot * a.heads + h] = m_new;
+}
+
+template <int R>
+int launch_step(const CellArgs& a, int n_seg, void* out, int f32, cudaStream_t st) {
+  const int nv4 = (a.vdim + 4) / 4;
+  // several CTAs per SM: at most kStepThreads threads, each with a few column groups one after the other
+  const int groups = nv4 * kKeyLanes, rounds = (groups + kStepThreads - 1) / kStepThreads;
+  int th = ((groups + rounds - 1) / rounds + 31) / 32 * 32;
+  const int sum_th = (a.vdim + 31) / 32 * 32 < 256 ? (a.vdim + 31) / 32 * 32 : 256;
+  th = th < sum_th ? sum_th : th;
+  const size_t smem = (size_t)(2 * kKeyLanes * (R + 1) + nv4 * 4) * sizeof(float);
+  if (f32) PRL_CUDA(launch_pdl((mlstm_step_kernel<float, R>), dim3(a.heads, n_seg), dim3(th), smem, st, a, (float*)out));
+  else PRL_CUDA(launch_pdl((mlstm_step_kernel<__nv_bfloat16, R>), dim3(a.heads, n_seg), dim3(th), smem, st, a, (__nv_bfloat16*)out));
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+}  // namespace
+}  // namespace prl
+
+extern "C" int prl_mlstm_step(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, int32_t off_v, int32_t off_g, int32_t off_i,
+                              int32_t off_f, const float* bias_i, const float* bias_f, float cap, float q_scale, float den_eps,
+                              const float* gain, float eps, int32_t heads, int32_t dk, int32_t vdim, const int32_t* seg_start,
+                              const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg, float* m_state, float* state, void* out,
+                              int32_t f32, prl_stream_t st) {
+  PRL_CHECK_ARG(P && bias_i && bias_f && gain && seg_start && seg_len && seg_slot && m_state && state && out, "prl_mlstm_step: NULL argument");
+  PRL_CHECK_ARG(heads >= 1 && dk >= 1 && dk <= 256 && vdim >= 1 && vdim <= 8192 && n_seg >= 1 && n_seg <= 65535 && cap >= 0.f &&
+                ((uintptr_t)state & 15) == 0, "prl_mlstm_step: bad shape (heads=%d dk=%d vdim=%d, dk at most 256)", heads, dk, vdim);
+  CellArgs a = {};
+  a.P = P; a.ldp = ldp; a.off_q = off_q; a.off_k = off_k; a.off_v = off_v; a.off_g = off_g; a.off_i = off_i; a.off_f = off_f;
+  a.bias_i = bias_i; a.bias_f = bias_f; a.cap = cap; a.q_scale = q_scale; a.den_eps = den_eps; a.gain = gain; a.eps = eps;
+  a.heads = heads; a.dk = dk; a.vdim = vdim; a.seg_start = seg_start; a.seg_len = seg_len; a.seg_slot = seg_slot;
+  a.m_state = m_state; a.state = state; a.state_slot_stride = prl_lin_scan_state_floats(heads, dk, vdim + 1);
+  switch (plan_r(dk)) {
+    case 1: return launch_step<1>(a, n_seg, out, f32, (cudaStream_t)st);
+    case 2: return launch_step<2>(a, n_seg, out, f32, (cudaStream_t)st);
+    case 4: return launch_step<4>(a, n_seg, out, f32, (cudaStream_t)st);
+    case 8: return launch_step<8>(a, n_seg, out, f32, (cudaStream_t)st);
+    case 16: return launch_step<16>(a, n_seg, out, f32, (cudaStream_t)st);
+    default: return launch_step<32>(a, n_seg, out, f32, (cudaStream_t)st);
+  }
 }

@@ -1150,8 +1150,8 @@ class _Rows:
         self.ob = torch.zeros(n * wide_o if any(eng.tc_attn.values()) else 1, dtype=torch.bfloat16, device=d)  # tcgen05 attention out
         self.ya = torch.zeros(n * wide_o, dtype=T, device=d)    # gated / normed input of the output projection
         self.yb = torch.zeros(n * wide_o2, dtype=T, device=d)
-        # up to 16 split-K slices of a <= 128-row projection, or the two products of a joint output projection
-        ny = max(2 * n if cfg.block == "one_norm" else n, 16 * min(n, 128)) * W
+        # up to 16 split-K slices of a <= 128-row projection, or up to four of a joint output projection
+        ny = max(4 * n if cfg.block == "one_norm" else n, 16 * min(n, 128)) * W
         self.y0 = torch.zeros(ny, **f32)
         self.y1 = torch.zeros(ny, **f32)
         self.q = torch.zeros(n * wide_q, dtype=T, device=d)
@@ -1209,6 +1209,7 @@ class HybridEngine(EngineCore):
         self.force_plain_gemm = False      # tests: route every GEMM through the CUDA-core kernel
         self.unfused_glu = False           # tests: gate_up GEMM + activation kernel instead of the GEMM's gated epilogue
         self.force_plain_attn = False      # tests: the any-geometry attention kernel also where the tcgen05 ones fit
+        self.unfused_cell = False          # tests: the matrix-memory cell's token step as separate kernels
         self.unfused_router = False        # tests: router logits through the GEMM and a separate choice kernel
         # Long prompt portions run their recurrences as side-by-side pieces (prl_*_scan_split): same values up to fp32
         # rounding, many times the parallelism.  Off in the true-fp32 mode, whose results do not depend on the cut of
@@ -1619,18 +1620,29 @@ class HybridEngine(EngineCore):
         H, nq, nv, P = c.heads, c.heads * c.dim, c.heads * c.vdim, R.P.data_ptr()
         seg_start, seg_len, seg_slot, ns = segs
         gb = vec[w + "mix.gate.b"].data_ptr()
+        off_g, off_i, norm = 2 * nq + nv, 2 * nq + 2 * nv, vec[w + "mix.norm"].data_ptr()
+        if n == ns and not self.unfused_cell:       # every segment is one token (or idle): the whole cell in one kernel
+            _lib.check(lib.prl_mlstm_step(P, ld, 0, nq, 2 * nq, off_g, off_i, off_i + H, gb, gb + 4 * H, c.gate_cap, c.dim ** -0.5,
+                                          c.den_eps, norm, self.cfg.eps, H, c.dim, c.vdim, seg_start, seg_len, seg_slot, ns,
+                                          self.mlstm_m[i].data_ptr(), self.mlstm_state[i].data_ptr(), R.ya.data_ptr(), f32, st))
+            return
+        if pieces is not None:                      # side-by-side pieces: the normaliser's column of ones is implied
+            _lib.check(lib.prl_mlstm_gates_scan(P, ld, off_i, off_i + H, gb, gb + 4 * H, c.gate_cap, H, seg_start, seg_len, seg_slot,
+                                                ns, self.mlstm_m[i].data_ptr(), R.gates.data_ptr(), R.minv.data_ptr(), st))
+            _lib.check(lib.prl_decay_scan_split(P, ld, 0, nq, c.dim ** -0.5, P, ld, 2 * nq, 1, R.gates.data_ptr(), 2 * H, 0, None, H,
+                                                c.dim, c.vdim + 1, seg_slot, ns, *pieces, self.mlstm_state[i].data_ptr(),
+                                                R.o.data_ptr(), H * (c.vdim + 1), st))
+            _lib.check(lib.prl_mlstm_out(R.o.data_ptr(), n, H, c.vdim, R.minv.data_ptr(), c.den_eps, P + 4 * off_g, ld, norm,
+                                         self.cfg.eps, R.ya.data_ptr(), f32, st))
+            return
         _lib.check(lib.prl_mlstm_gates(P, ld, 2 * nq + 2 * nv, 2 * nq + 2 * nv + H, gb, gb + 4 * H, c.gate_cap, H, seg_start,
                                        seg_len, seg_slot, ns, self.mlstm_m[i].data_ptr(), R.gates.data_ptr(),
                                        R.minv.data_ptr(), st))
         _lib.check(lib.prl_append_one(P, ld, 2 * nq, n, H, c.vdim, R.aux.data_ptr(), st))
         dv = c.vdim + 1
         head = (P, ld, 0, nq, c.dim ** -0.5, R.aux.data_ptr(), H * dv, 0, R.gates.data_ptr(), 2 * H, 0, None, H, c.dim, dv)
-        if pieces is not None:
-            _lib.check(lib.prl_decay_scan_split(*head, seg_slot, ns, *pieces, self.mlstm_state[i].data_ptr(), R.o.data_ptr(),
-                                                H * dv, st))
-        else:
-            _lib.check(lib.prl_decay_scan(*head, seg_start, seg_len, seg_slot, ns, self.mlstm_state[i].data_ptr(),
-                                          R.o.data_ptr(), H * dv, st))
+        _lib.check(lib.prl_decay_scan(*head, seg_start, seg_len, seg_slot, ns, self.mlstm_state[i].data_ptr(), R.o.data_ptr(), H * dv,
+                                      st))
         _lib.check(lib.prl_mlstm_out(R.o.data_ptr(), n, H, c.vdim, R.minv.data_ptr(), c.den_eps, P + 4 * (2 * nq + nv), ld,
                                      vec[w + "mix.norm"].data_ptr(), self.cfg.eps, R.ya.data_ptr(), f32, st))
 
@@ -1661,7 +1673,7 @@ class HybridEngine(EngineCore):
         _lib.check(lib.prl_act_cols(P, ld, off, n, 2 * rq + rv, 0, st))            # SiLU on q, k, v
         head = (P, ld, off, off + rq, 1.0, P, ld, off + 2 * rq, None, 0, 0, self.lin_decay[i].data_ptr(), r.heads, r.dim, r.vdim)
         if pieces is not None:
-            _lib.check(lib.prl_decay_scan_split(*head, seg_slot, ns, *pieces, self.lin_state[i].data_ptr(), R.o2.data_ptr(),
+            _lib.check(lib.prl_decay_scan_split(*head[:8], 0, *head[8:], seg_slot, ns, *pieces, self.lin_state[i].data_ptr(), R.o2.data_ptr(),
                                                 rv, st))
         else:
             _lib.check(lib.prl_decay_scan(*head, seg_start, seg_len, seg_slot, ns, self.lin_state[i].data_ptr(),
@@ -1793,8 +1805,9 @@ class HybridEngine(EngineCore):
             k = int(lib.prl_gemm_dual_split_k(n, N, K1, K2))
             _lib.check(lib.prl_gemm_bf16_dual(p1, src1.data_ptr(), K1, p2, src2.data_ptr(), K2, n, N, k, out.data_ptr(), st))
             return k
-        _lib.check(lib.prl_gemm_tn_dual(src1.data_ptr(), p1, K1, src2.data_ptr(), p2, K2, n, N, out.data_ptr(), N, st))
-        return 1
+        k = int(lib.prl_gemm_tn_dual_split_k(n, N, K1, K2, 4))
+        _lib.check(lib.prl_gemm_tn_dual(src1.data_ptr(), p1, K1, src2.data_ptr(), p2, K2, n, N, k, out.data_ptr(), st))
+        return k
 
     def _choose_and_run_experts(self, R, n, w, e, ld, off_router) -> torch.Tensor:
         """Squared-ReLU experts chosen from the router's columns of R.P; returns [top][n][W] fp32 (R.moe_out), in which the

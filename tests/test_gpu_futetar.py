@@ -377,9 +377,10 @@ def test_dual_product_gemm(cuda_device, M_, N, K1, K2):
             _lib.check(lib.prl_gemm_bf16_dual(B1.data_ptr(), A1.data_ptr(), K1, B2.data_ptr(), A2.data_ptr(), K2, M_, N, k, out.data_ptr(), st))
             assert (out.sum(0).double() - ref).abs().max().item() < 1e-4
     else:
-        out = torch.full((M_, N), float("nan"), device=cuda_device)
-        _lib.check(lib.prl_gemm_tn_dual(A1.data_ptr(), B1.data_ptr(), K1, A2.data_ptr(), B2.data_ptr(), K2, M_, N, out.data_ptr(), N, st))
-        assert (out.double() - ref).abs().max().item() < 1e-4
+        for k in (1, int(lib.prl_gemm_tn_dual_split_k(M_, N, K1, K2, 4)), 3):
+            out = torch.full((k, M_, N), float("nan"), device=cuda_device)
+            _lib.check(lib.prl_gemm_tn_dual(A1.data_ptr(), B1.data_ptr(), K1, A2.data_ptr(), B2.data_ptr(), K2, M_, N, k, out.data_ptr(), st))
+            assert (out.sum(0).double() - ref).abs().max().item() < 1e-4
 
 
 def test_long_decoding(cuda_device):

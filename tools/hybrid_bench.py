@@ -410,7 +410,7 @@ def kernel_table_belelorn(eng, s, batch, chunk, timer):
                                               fp32_fma_frac=round(flops / ms / 1e9 / fma_tflops, 3))
         if shape == "prefill":
             def lin_split():
-                _lib.check(lib.prl_decay_scan_split(*head, seg[3], ns, *pieces, eng.lin_state[pi].data_ptr(), R.o2.data_ptr(), rv, st))
+                _lib.check(lib.prl_decay_scan_split(*head[:8], 0, *head[8:], seg[3], ns, *pieces, eng.lin_state[pi].data_ptr(), R.o2.data_ptr(), rv, st))
             ms = timer.events(lin_split)
             out["lightning_scan_split/prefill"] = dict(ms=round(ms, 4), fp32_fma_frac=round(1.4 * flops / ms / 1e9 / fma_tflops, 3))
         # -- matrix-memory LSTM
@@ -441,7 +441,7 @@ def kernel_table_belelorn(eng, s, batch, chunk, timer):
                                           fp32_fma_frac=round(flops / ms / 1e9 / fma_tflops, 3))
         if shape == "prefill":
             def cell_split():
-                _lib.check(lib.prl_decay_scan_split(*mhead, seg[3], ns, *pieces, eng.mlstm_state[mi].data_ptr(), R.o.data_ptr(), H * dv, st))
+                _lib.check(lib.prl_decay_scan_split(*mhead[:5], R.P.data_ptr(), ldm, 2 * mq, 1, *mhead[8:], seg[3], ns, *pieces, eng.mlstm_state[mi].data_ptr(), R.o.data_ptr(), H * dv, st))
             ms = timer.events(cell_split)
             out["mlstm_scan_split/prefill"] = dict(ms=round(ms, 4), fp32_fma_frac=round(1.4 * flops / ms / 1e9 / fma_tflops, 3))
 
