@@ -769,8 +769,15 @@ int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, co
 /* choice from ready logits: outputs ranked by softmax share + correction (nullable) inside the `keep` best of `groups`
  * equal groups, weighted by the share alone; outputs experts .. outputs - 1 hand the input through (no rows) */
 int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
-                   int32_t top, int32_t groups, int32_t keep, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta,
-                   int32_t* tiles, prl_stream_t stream);
+                   int32_t top, int32_t groups, int32_t keep, int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm,
+                   int32_t* meta, int32_t* tiles, prl_stream_t stream);
+/* many rows per expert: rows gathered into sorted order, then a persistent tcgen05 grouped GEMM over row tiles of 256; wsel
+ * NULL: fp32 rows perm[s] of out, else bf16 rows s = relu(.)^2 * wsel[perm[s]] */
+int prl_moe_gather(const void* x_bf16, const int32_t* perm, const int32_t* meta, int32_t n, int32_t pairs, int32_t W, void* out,
+                   prl_stream_t stream);
+int prl_moe_gemm_tc(const void* A_bf16, int64_t rows_cap, const void* W_bf16, int32_t experts, int64_t N, int64_t K,
+                    const int32_t* perm, const int32_t* meta, const int32_t* tiles, const float* wsel, void* out, int64_t ldc,
+                    prl_stream_t stream);
 /* prl_moe_gemm with act[s] = relu(product)^2 * wsel[pair] written in sorted order in A's type (the second product's operand) */
 int prl_moe_gemm_relu2(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
                        int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,

@@ -62,6 +62,13 @@ struct TnParams {
   // g = min(gate, limit), u = clamp(up, +-limit), act = g * sigmoid(glu_beta * g) * (u + 1)
   float glu_limit, glu_beta;
   int glu_gelu;            // 1 (with swiglu_fp32): gelu(gate) * up, the tanh form of gelu
+  // grouped rows (g_tiles != NULL): work item t is row tile t / n_tiles of a device table [expert, first row, rows <= 256] (g_meta[0]
+  // entries) against columns (t % n_tiles) * 256 .. of the expert's rows of B (stacked, N rows each).  Row s of the sorted A
+  // goes to C row g_perm[s] (fp32) or, with g_w, to act row s as bf16 relu(.)^2 * g_w[g_perm[s]]
+  const int32_t* g_tiles;
+  const int32_t* g_meta;
+  const int32_t* g_perm;
+  const float* g_w;
   // head epilogue (kHead): logits never leave TMEM/registers
   const int64_t* targets;  // [M] or NULL
   float4* head_part;       // [n_tiles, M]: (max, sum exp, sum exp*z, target logit or -inf) of one 256-column vocabulary tile
@@ -93,6 +100,11 @@ __device__ __forceinline__ void k_range(int t, const TnParams& p, int& kb0, int&
 }
 
 __device__ __forceinline__ void tile_coords(int t, const TnParams& p, int& tm, int& tn) {
+  if (p.g_tiles) {
+    tm = t / p.n_tiles;
+    tn = t - tm * p.n_tiles;
+    return;
+  }
   if (p.split > 1) t /= p.split;
   const int per_group = kGroupM * p.n_tiles;
   const int g = t / per_group;
@@ -120,7 +132,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
   const uint32_t rank = ptx::cluster_ctarank();
   const int n_clusters = (int)gridDim.x >> 1;
   const int cluster = (int)blockIdx.x >> 1;
-  const int total_tiles = p.m_tiles * p.n_tiles * (p.split > 1 ? p.split : 1);
+  const int total_tiles = p.g_tiles ? p.g_meta[0] * p.n_tiles : p.m_tiles * p.n_tiles * (p.split > 1 ? p.split : 1);
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -156,8 +168,8 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
         tile_coords(t, p, tm, tn);
         int kb0, kb1;
         k_range(t, p, kb0, kb1);
-        const int a_row = tm * kTile + (int)rank * kHalf;
-        const int b_row = p.swiglu_I ? tn * kHalf + (int)rank * (int)p.swiglu_I : tn * kTile + (int)rank * kHalf;
+        const int a_row = (p.g_tiles ? p.g_tiles[3 * tm + 1] : tm * kTile) + (int)rank * kHalf;
+        const int b_row = p.g_tiles ? p.g_tiles[3 * tm] * (int)p.N + tn * kTile + (int)rank * kHalf : p.swiglu_I ? tn * kHalf + (int)rank * (int)p.swiglu_I : tn * kTile + (int)rank * kHalf;
         for (int kb = kb0; kb < kb1; ++kb, ++it) {
           const int s = it % kStages;
           const uint32_t ph = (uint32_t)((it / kStages) & 1);
@@ -228,9 +240,20 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
       const uint32_t acc_ph = (uint32_t)((local >> 1) & 1);
       ptx::mbar_wait(acc_full_bar(acc), acc_ph);
       ptx::tc_fence_after_sync();
-      const int64_t row = (int64_t)tm * kTile + (int64_t)rank * kHalf + q * 32 + lane;
+      int64_t row = (int64_t)tm * kTile + (int64_t)rank * kHalf + q * 32 + lane;
       const int64_t col0 = (int64_t)tn * kTile;
-      const bool row_ok = row < p.M;
+      bool row_ok = row < p.M;
+      float row_w = 0.f;
+      if (!kHead && p.g_tiles) {
+        const int local_row = (int)rank * kHalf + q * 32 + lane;
+        row_ok = local_row < p.g_tiles[3 * tm + 2];
+        row = p.g_tiles[3 * tm + 1] + local_row;
+        if (row_ok) {
+          const int pair = p.g_perm[row];
+          if (p.g_w) row_w = p.g_w[pair];
+          else row = pair;
+        }
+      }
       if constexpr (kHead) {
         // thread = one token; online softmax statistics over this tile's 256 vocabulary columns, all thread-local
         constexpr float kLog2e = 1.4426950408889634f;
@@ -403,6 +426,29 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
             for (int j = 0; j < 32; ++j)
               if (col + j < p.N) v[j] += __bfloat162float(rp[j]);
           }
+        }
+        if (p.g_w) {
+          __nv_bfloat16* ap = p.act + row * p.ld_act + col;
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float z = fmaxf(v[j], 0.f);
+            v[j] = z * z * row_w;
+          }
+          if (full && ((p.ld_act & 7) == 0)) {
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              uint4 u;
+              __nv_bfloat162* hb = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) hb[e] = __floats2bfloat162_rn(v[j + 2 * e], v[j + 2 * e + 1]);
+              *reinterpret_cast<uint4*>(ap + j) = u;
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (col + j < p.N) ap[j] = __float2bfloat16_rn(v[j]);
+          }
+          continue;
         }
         if (p.dgu != nullptr) {
           // d act tile -> (d gate, d up): same rounding points as the two-kernel path (d act rounded to bf16, then
@@ -660,6 +706,41 @@ extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, cons
   int clusters = num_sms() / 2;
   if (tiles < clusters) clusters = (int)tiles;
   gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta2, tb2, p);
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+// Grouped GEMM over rows sorted by expert (csrc/moe_ops.cu tables with row tiles of at most 256): A [rows_cap, K] bf16 holds the sorted
+// rows, W the experts' matrices stacked ([experts * N, K]).  wsel NULL: C[perm[s]] (fp32, row stride ldc) = A[s] W_e^T;
+// otherwise out[s] (bf16, row stride ldc) = relu(A[s] W_e^T)^2 * wsel[perm[s]].  The number of tiles stays on the device: the
+// persistent clusters walk meta[0] * ceil(N / 256) items.
+extern "C" int prl_moe_gemm_tc(const void* A, int64_t rows_cap, const void* W, int32_t experts, int64_t N, int64_t K, const int32_t* perm,
+                               const int32_t* meta, const int32_t* tiles, const float* wsel, void* out, int64_t ldc,
+                               prl_stream_t stream_) {
+  PRL_CHECK_ARG(A && W && perm && meta && tiles && out, "prl_moe_gemm_tc: NULL argument");
+  PRL_CHECK_ARG(rows_cap >= 1 && experts >= 1 && N >= 1 && K >= 8 && K % 8 == 0 && ldc >= N && experts * N < (1ll << 31),
+                "prl_moe_gemm_tc: bad shape (rows=%lld experts=%d N=%lld K=%lld)", (long long)rows_cap, experts, (long long)N, (long long)K);
+  TnParams p = {};
+  p.M = rows_cap; p.N = N; p.K = K;
+  p.kblocks = p.k_wrap = (int)((K + kBK - 1) / kBK);
+  p.m_tiles = 1;
+  p.n_tiles = (int)((N + kTile - 1) / kTile);
+  p.alpha = 1.f;
+  p.g_tiles = tiles; p.g_meta = meta; p.g_perm = perm; p.g_w = wsel;
+  if (wsel) { p.act = (__nv_bfloat16*)out; p.ld_act = ldc; }
+  else { p.C = out; p.ldc = ldc; p.c_f32 = 1; }
+  CUtensorMap ta, tb;
+  int rc = make_tmap_2d_bf16(&ta, A, (uint64_t)K, (uint64_t)rows_cap, (uint64_t)K * 2, kBK, kHalf);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tb, W, (uint64_t)K, (uint64_t)(experts * N), (uint64_t)K * 2, kBK, kHalf);
+  if (rc) return rc;
+  const int smem = kStages * kStageBytes + 1024 + 8 * (2 * kStages + 4) + 16;
+  static SmemAttr smem_attr = {};
+  PRL_CUDA(ensure_smem(gemm_tn_kernel<false>, smem, smem_attr));
+  const int64_t items = ((rows_cap + kTile - 1) / kTile + experts) * p.n_tiles;
+  int clusters = num_sms() / 2;
+  if (items < clusters) clusters = (int)items;
+  gemm_tn_kernel<false><<<dim3((unsigned)(2 * clusters)), dim3(kThreadsTN), (size_t)smem, (cudaStream_t)stream_>>>(ta, tb, ta, tb, p);
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }

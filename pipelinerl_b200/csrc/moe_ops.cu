@@ -12,6 +12,8 @@
 //   3. grouped GEMM (twice):  C[row] = A[row'] * W_e^T for every tile, W_e = W + e * expert_stride.  The first product
 //              reads the token's row (perm[s] % n) and writes sorted rows; the second reads sorted rows and writes
 //              pair rows, i.e. `top` slices [top][n][width] that the sublayer's closing kernel adds up.
+//      Batches with many rows per expert (bf16) gather the tokens' rows into sorted order first and run both products on
+//      the tcgen05 CTA-pair kernel (prl_moe_gather, prl_moe_gemm_tc in gemm_tn.cu) with row tiles of 256.
 //   4. gated activation of an expert with the pair's weight folded in: the weight multiplies the expert's INPUT, and
 //              the two first projections are linear, so gate and up are scaled after the product (in fp32).
 //
@@ -213,8 +215,8 @@ __global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const flo
   }
 }
 
-// meta[0] = number of tiles; tiles[3 * i + {0, 1, 2}] = expert, first sorted place, rows
-__global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restrict__ sel, int pairs, int E,
+// meta[0] = number of tiles, meta[1] = sorted pairs; tiles[3 * i + {0, 1, 2}] = expert, first sorted place, rows (<= tile_rows)
+__global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restrict__ sel, int pairs, int E, int tile_rows,
                                                          int32_t* __restrict__ perm, int32_t* __restrict__ meta,
                                                          int32_t* __restrict__ tiles) {
   pdl_wait();
@@ -230,15 +232,16 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
     int at = 0, nt = 0;
     for (int e = 0; e < E; ++e) {
       off[e] = at;
-      for (int r0 = 0; r0 < cnt[e]; r0 += kTile) {
+      for (int r0 = 0; r0 < cnt[e]; r0 += tile_rows) {
         tiles[3 * nt] = e;
         tiles[3 * nt + 1] = at + r0;
-        tiles[3 * nt + 2] = min(kTile, cnt[e] - r0);
+        tiles[3 * nt + 2] = min(tile_rows, cnt[e] - r0);
         ++nt;
       }
       at += cnt[e];
     }
     meta[0] = nt;
+    meta[1] = at;
   }
   __syncthreads();
   for (int e = warp; e < E; e += nw) {     // stable: pairs of an expert keep their order
@@ -251,6 +254,18 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
       at += __popc(mask);
     }
   }
+}
+
+// out[s] = x[perm[s] % n]: the tokens' rows (16-byte units) in sorted order, the A operand of the tcgen05 grouped GEMM
+__global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict__ x, const int32_t* __restrict__ perm,
+                                                         const int32_t* __restrict__ meta, int n, int units, uint4* __restrict__ out) {
+  pdl_wait();
+  const int s = blockIdx.x;
+  if (s >= meta[1]) return;
+  const uint4* src = x + (int64_t)(perm[s] % n) * units;
+  uint4* dst = out + (int64_t)s * units;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < units; i += 128) dst[i] = src[i];
 }
 
 // RELU2: C is the next product's operand (type TA), C[row] = relu(product)^2 * wsel[pair]
@@ -331,8 +346,8 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
 }
 
 // ---- bf16 tensor-core variant ------------------------------------------------------------------------------------------
-constexpr int kBN = 128, kBK = 32, kPad = 8;      // tile N, K step, padding (halves) that keeps ldmatrix conflict-free
-constexpr int kLds = kBK + kPad;                  // 40 halves = 80 bytes per staged row
+constexpr int kBN = 128, kBK = 64, kPad = 8;      // tile N, K step, padding (halves) that keeps ldmatrix conflict-free
+constexpr int kLds = kBK + kPad;                  // 72 halves = 144 bytes per staged row
 constexpr int kStages = 4;                        // cp.async stages in flight: a few-row tile is a pure weight stream
 constexpr size_t kMmaSmem = (size_t)kStages * (kTile + kBN) * kLds * sizeof(__nv_bfloat16);
 
@@ -364,8 +379,8 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
   extern __shared__ __align__(16) unsigned char mma_smem[];
   typedef __nv_bfloat16 (*ATile)[kTile][kLds];
   typedef __nv_bfloat16 (*BTile)[kBN][kLds];
-  ATile As = reinterpret_cast<ATile>(mma_smem);                                           // [kStages][64][40]
-  BTile Bs = reinterpret_cast<BTile>(mma_smem + (size_t)kStages * kTile * kLds * sizeof(__nv_bfloat16));   // [kStages][128][40]
+  ATile As = reinterpret_cast<ATile>(mma_smem);                                           // [kStages][64][72]
+  BTile Bs = reinterpret_cast<BTile>(mma_smem + (size_t)kStages * kTile * kLds * sizeof(__nv_bfloat16));   // [kStages][128][72]
   __shared__ int32_t a_row[kTile], c_row[kTile];
   __shared__ float c_w[kTile];
   const int e = tiles[3 * tile], s0 = tiles[3 * tile + 1], M = tiles[3 * tile + 2];
@@ -388,16 +403,19 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
     for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int q = 0; q < 4; ++q) acc[i][j][q] = 0.f;
-  // loaders: A 64 rows x 4 chunks of 8 halves (one per thread), B 128 rows x 4 chunks (two per thread)
-  const int lr = tid >> 2, lc = (tid & 3) * 8;
-  const int64_t a_off = (int64_t)a_row[lr] * lda;
+  // loaders: A 64 rows x 8 chunks of 8 halves (two per thread), B 128 rows x 8 chunks (four per thread)
+  const int lr = tid >> 3, lc = (tid & 7) * 8;
+  const int64_t a_off[2] = {(int64_t)a_row[lr] * lda, (int64_t)a_row[lr + 32] * lda};
   auto stage = [&](int k0, int buf) {
     const int k = k0 + lc;
     const bool kin = k < K;
-    cp_async16_zfill(&As[buf][lr][lc], A + a_off + (kin ? k : 0), (kin && lr < M) ? 16 : 0);
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int r = lr + 64 * h, nn = n0 + r;
+    for (int h = 0; h < 2; ++h)
+      if (32 * h < M)         // uniform: the upper half of a short tile is not staged, and the warps that own it do nothing
+        cp_async16_zfill(&As[buf][lr + 32 * h][lc], A + a_off[h] + (kin ? k : 0), (kin && lr + 32 * h < M) ? 16 : 0);
+#pragma unroll
+    for (int h = 0; h < 4; ++h) {
+      const int r = lr + 32 * h, nn = n0 + r;
       const bool ok = kin && nn < N;
       cp_async16_zfill(&Bs[buf][r][lc], We + (int64_t)(ok ? nn : 0) * ldw + (kin ? k : 0), ok ? 16 : 0);
     }
@@ -412,6 +430,7 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
     asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
     __syncthreads();            // step k0 has landed for every thread, and every warp is done with the buffer refilled next
     stage(k0 + (kStages - 1) * kBK, (buf + kStages - 1) % kStages);
+    if (wm < M)                 // warp-uniform
 #pragma unroll
     for (int kk = 0; kk < kBK; kk += 16) {
       uint32_t af[2][4], bf[2][4];
@@ -500,7 +519,7 @@ extern "C" int prl_moe_route(const float* logits, int64_t ld, const float* bias,
   cudaStream_t s = (cudaStream_t)st;
   PRL_CUDA(launch_pdl(moe_route_kernel, dim3((n + 7) / 8), dim3(256), (size_t)0, s, logits, ld, bias, n, experts, top, softmax_weights, sel, wsel));
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, perm, meta, tiles));
+  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, kTile, perm, meta, tiles));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -529,16 +548,17 @@ extern "C" int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, i
   else PRL_RT(bf16, bf16, 3);
 #undef PRL_RT
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, perm, meta, tiles));
+  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, kTile, perm, meta, tiles));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
 
 // Choice among outputs whose logits are already there (columns of a projection buffer), and the grouping of the pairs by expert:
-// `outputs` = experts + identity outputs; see moe_choose_kernel.  keep == groups (e.g. 1, 1): every output is open.
+// `outputs` = experts + identity outputs; see moe_choose_kernel.  tile_rows: 64 for prl_moe_gemm, 256 for prl_moe_gemm_tc.  keep == groups (e.g. 1, 1): every output is open.
 extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
-                              int32_t top, int32_t groups, int32_t keep, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta,
-                              int32_t* tiles, prl_stream_t st) {
+                              int32_t top, int32_t groups, int32_t keep, int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm,
+                              int32_t* meta, int32_t* tiles, prl_stream_t st) {
+  PRL_CHECK_ARG(tile_rows == kTile || tile_rows == 256, "prl_moe_choose: row tiles of 64 or 256");
   PRL_CHECK_ARG(logits && sel && wsel && perm && meta && tiles, "prl_moe_choose: NULL argument");
   PRL_CHECK_ARG(n >= 1 && experts >= 1 && outputs >= experts && outputs <= 1024 && ld >= outputs && groups >= 1 &&
                 outputs % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= outputs / groups * keep,
@@ -548,7 +568,16 @@ extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* corr
                       (size_t)kChooseWarps * (outputs + groups) * sizeof(float), s, logits, ld, correction, n, outputs, top, groups,
                       keep, sel, wsel));
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, perm, meta, tiles));
+  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, tile_rows, perm, meta, tiles));
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+extern "C" int prl_moe_gather(const void* x_bf16, const int32_t* perm, const int32_t* meta, int32_t n, int32_t pairs, int32_t W, void* out,
+                              prl_stream_t st) {
+  PRL_CHECK_ARG(x_bf16 && perm && meta && out && n >= 1 && pairs >= 1 && W >= 8 && W % 8 == 0 && (((uintptr_t)x_bf16 | (uintptr_t)out) & 15) == 0,
+                "prl_moe_gather: bad argument (rows of a multiple of eight bf16)");
+  PRL_CUDA(launch_pdl(moe_gather_kernel, dim3(pairs), dim3(128), (size_t)0, (cudaStream_t)st, (const uint4*)x_bf16, perm, meta, n, W / 8, (uint4*)out));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }

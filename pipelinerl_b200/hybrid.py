@@ -1210,6 +1210,7 @@ class HybridEngine(EngineCore):
         self.unfused_glu = False           # tests: gate_up GEMM + activation kernel instead of the GEMM's gated epilogue
         self.force_plain_attn = False      # tests: the any-geometry attention kernel also where the tcgen05 ones fit
         self.unfused_cell = False          # tests: the matrix-memory cell's token step as separate kernels
+        self.moe_tc_rows = 48              # routed pairs per expert from which the tcgen05 grouped GEMM runs (tests lower it)
         self.unfused_router = False        # tests: router logits through the GEMM and a separate choice kernel
         # Long prompt portions run their recurrences as side-by-side pieces (prl_*_scan_split): same values up to fp32
         # rounding, many times the parallelism.  Off in the true-fp32 mode, whose results do not depend on the cut of
@@ -1814,14 +1815,24 @@ class HybridEngine(EngineCore):
         slices of choices that hand the input through (R.sel >= experts) are not written."""
         lib, st, W, f32 = self.lib, self._st, self.cfg.width, int(self.f32)
         corr = self.vec[w + "mlp.correction"].data_ptr() if e.correction else None
+        pairs, up, down = n * e.top, self.arena.ptr(w + "mlp.experts.up"), self.arena.ptr(w + "mlp.experts.down")
+        # enough rows per expert for 256-row tiles: the tcgen05 grouped GEMM over gathered rows
+        tc = (pairs >= self.moe_tc_rows * e.experts and n > 128 and W % 8 == 0 and e.ff % 8 == 0 and min(W, e.ff) >= 64
+              and not (self.f32 or self.force_plain_gemm))
         _lib.check(lib.prl_moe_choose(R.P.data_ptr() + 4 * off_router, ld, corr, n, e.experts, e.outputs, e.top, e.groups,
-                                      e.keep_groups, R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(),
+                                      e.keep_groups, 256 if tc else 64, R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(),
                                       R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), st))
-        table = (R.perm.data_ptr(), R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), int(lib.prl_moe_max_tiles(n * e.top, e.experts)))
-        _lib.check(lib.prl_moe_gemm_relu2(R.xa.data_ptr(), f32, W, n, self.arena.ptr(w + "mlp.experts.up"), f32, e.ff * W, W,
-                                          *table, e.ff, W, R.wsel.data_ptr(), R.moe_act.data_ptr(), e.ff, st))
-        _lib.check(lib.prl_moe_gemm(R.moe_act.data_ptr(), f32, e.ff, 0, self.arena.ptr(w + "mlp.experts.down"), f32, W * e.ff,
-                                    e.ff, *table, W, e.ff, R.moe_out.data_ptr(), W, 1, st))
+        table = (R.perm.data_ptr(), R.moe_meta.data_ptr(), R.moe_tiles.data_ptr())
+        act, out = R.moe_act.data_ptr(), R.moe_out.data_ptr()
+        if tc:      # the gathered rows live where the second product's output goes: they are consumed before it is written
+            _lib.check(lib.prl_moe_gather(R.xa.data_ptr(), *table[:2], n, pairs, W, out, st))
+            _lib.check(lib.prl_moe_gemm_tc(out, pairs, up, e.experts, e.ff, W, *table, R.wsel.data_ptr(), act, e.ff, st))
+            _lib.check(lib.prl_moe_gemm_tc(act, pairs, down, e.experts, W, e.ff, *table, None, out, W, st))
+            return R.moe_out
+        table += (int(lib.prl_moe_max_tiles(pairs, e.experts)),)
+        _lib.check(lib.prl_moe_gemm_relu2(R.xa.data_ptr(), f32, W, n, up, f32, e.ff * W, W, *table, e.ff, W, R.wsel.data_ptr(), act,
+                                          e.ff, st))
+        _lib.check(lib.prl_moe_gemm(act, f32, e.ff, 0, down, f32, W * e.ff, e.ff, *table, W, e.ff, out, W, 1, st))
         return R.moe_out
 
     def _attn_core(self, R, n, i, L, w, segs, max_q, row_pos, seg_pos0, ld, decode) -> torch.Tensor:

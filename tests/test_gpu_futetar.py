@@ -277,7 +277,7 @@ def test_choice_kernel_against_the_oracle(cuda_device, n):
         wsel, meta = torch.zeros(top, n, device=cuda_device), torch.zeros(4, **i32)
         tiles = torch.zeros(3 * int(lib.prl_moe_max_tiles(top * n, experts)), **i32)
         zd, cd = z.to(cuda_device), corr.to(cuda_device)
-        _lib.check(lib.prl_moe_choose(zd.data_ptr(), E + 3, cd.data_ptr(), n, experts, E, top, groups, keep, sel.data_ptr(), wsel.data_ptr(),
+        _lib.check(lib.prl_moe_choose(zd.data_ptr(), E + 3, cd.data_ptr(), n, experts, E, top, groups, keep, 64, sel.data_ptr(), wsel.data_ptr(),
                                       perm.data_ptr(), meta.data_ptr(), tiles.data_ptr(), _lib.stream_ptr()))
         torch.cuda.synchronize()
         score = torch.softmax(z[:, :E].double(), -1)
@@ -331,6 +331,8 @@ def test_bf16_serving_mode(cuda_device, mode):
     assert fc.rel_err(whole[clear], ref[clear]) < BF16_TOL
     assert fc.rel_err(fc.stream_logits(eng, toks, [100, 2, 30])[clear], ref[clear]) < BF16_TOL
     assert fc.rel_err(fc.stream_logits(eng, toks, [130, 129])[clear], ref[clear]) < BF16_TOL
+    eng.moe_tc_rows = 1 << 20                                # the routed products of the prompt on the few-row kernel
+    assert fc.rel_err(fc.stream_logits(eng, toks, [300])[clear], ref[clear]) < BF16_TOL
     # the bf16 engine is about as close to the oracle as the oracle with only its matrix products' inputs rounded
     least = fc.rel_err(fc.oracle_logits(BIG, wt, toks, round_in=fc.bf16_round)[clear], ref[clear])
     assert fc.rel_err(whole[clear], ref[clear]) < 3 * least + 1e-3
@@ -381,6 +383,42 @@ def test_dual_product_gemm(cuda_device, M_, N, K1, K2):
             out = torch.full((k, M_, N), float("nan"), device=cuda_device)
             _lib.check(lib.prl_gemm_tn_dual(A1.data_ptr(), B1.data_ptr(), K1, A2.data_ptr(), B2.data_ptr(), K2, M_, N, k, out.data_ptr(), st))
             assert (out.sum(0).double() - ref).abs().max().item() < 1e-4
+
+
+@pytest.mark.parametrize("n,W,ff,experts,identity,top", [(300, 64, 64, 3, 1, 2), (700, 136, 200, 5, 3, 3), (129, 256, 520, 2, 0, 1), (1024, 64, 72, 40, 8, 6)])
+def test_grouped_gemm_of_many_rows(cuda_device, n, W, ff, experts, identity, top):
+    """The tcgen05 grouped GEMM over gathered rows (row tiles of 256, expert sizes that are no multiple of a tile, choices
+    that belong to no expert) against fp32 torch, for both products."""
+    from pipelinerl_b200 import _lib
+    lib = _lib.load()
+    g = torch.Generator().manual_seed(n)
+    bf = lambda *s: (torch.randn(*s, generator=g) / s[-1] ** 0.5).to(torch.bfloat16).to(cuda_device)
+    x, up, down = bf(n, W) * 4, bf(experts * ff, W), bf(experts * W, ff)
+    E = experts + identity
+    z = torch.randn(n, E, generator=g).to(cuda_device)
+    i32 = dict(dtype=torch.int32, device=cuda_device)
+    sel, perm, meta = torch.zeros(top, n, **i32), torch.zeros(top * n, **i32), torch.zeros(4, **i32)
+    wsel, tiles = torch.zeros(top, n, device=cuda_device), torch.zeros(3 * int(lib.prl_moe_max_tiles(top * n, experts)), **i32)
+    st = _lib.stream_ptr()
+    table = (perm.data_ptr(), meta.data_ptr(), tiles.data_ptr())
+    _lib.check(lib.prl_moe_choose(z.data_ptr(), E, None, n, experts, E, top, 1, 1, 256, sel.data_ptr(), wsel.data_ptr(), *table, st))
+    xs, act = torch.zeros(top * n, W, dtype=torch.bfloat16, device=cuda_device), torch.zeros(top * n, ff, dtype=torch.bfloat16, device=cuda_device)
+    out = torch.full((top * n, W), float("nan"), device=cuda_device)
+    _lib.check(lib.prl_moe_gather(x.data_ptr(), *table[:2], n, top * n, W, xs.data_ptr(), st))
+    _lib.check(lib.prl_moe_gemm_tc(xs.data_ptr(), top * n, up.data_ptr(), experts, ff, W, *table, wsel.data_ptr(), act.data_ptr(), ff, st))
+    _lib.check(lib.prl_moe_gemm_tc(act.data_ptr(), top * n, down.data_ptr(), experts, W, ff, *table, None, out.data_ptr(), W, st))
+    torch.cuda.synchronize()
+    assert int(meta[1]) == int((sel < experts).sum())
+    for k in range(top):
+        for e in range(E):
+            rows = (sel[k] == e).nonzero().view(-1)
+            got = out[k * n + rows]
+            if e >= experts:
+                assert torch.isnan(got).all()                        # handed through elsewhere, not written here
+                continue
+            a = torch.relu(x[rows].float() @ up[e * ff:(e + 1) * ff].float().T) ** 2 * wsel[k, rows, None]
+            want = a.to(torch.bfloat16).float() @ down[e * W:(e + 1) * W].float().T
+            assert (got - want).abs().max().item() < 2e-2 * max(1.0, want.abs().max().item()) if len(rows) else True
 
 
 def test_long_decoding(cuda_device):
