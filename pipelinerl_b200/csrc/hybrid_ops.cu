@@ -743,6 +743,41 @@ __global__ void mlstm_out_kernel(const float* __restrict__ o_aug, int H, int dv,
   }
 }
 
+// The same for many rows, one warp per (row, head) with the head's values in registers (dv <= 32 * NV)
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) mlstm_out_warp_kernel(const float* __restrict__ o_aug, int n, int H, int dv,
+                                                             const float* __restrict__ minv, float den_eps,
+                                                             const float* __restrict__ g, int64_t ldg,
+                                                             const float* __restrict__ gain, float eps, T* __restrict__ out) {
+  pdl_wait();
+  const int64_t id = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (id >= (int64_t)n * H) return;
+  const int64_t r = id / H;
+  const int h = (int)(id - r * H);
+  const float* o = o_aug + id * (dv + 1);
+  const float* gr = g + r * ldg + h * dv;
+  const float den = fmaxf(fabsf(o[dv]), minv[id]) + den_eps;
+  float v[NV], z[NV], ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int c = lane + 32 * u;
+    v[u] = c < dv ? o[c] : 0.f;
+    z[u] = c < dv ? gr[c] : 0.f;
+  }
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    v[u] /= den;
+    ss += v[u] * v[u];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int c = lane + 32 * u;
+    if (c < dv) stf(out, id * dv + c, v[u] * inv * gain[h * dv + c] * sigmoid_f(z[u]));
+  }
+}
+
 // Norm AFTER the sum ("post-LN" with a weighted skip):  v = alpha * x + s0 * y0 + s1 * y1 + bias;
 // x <- v / sqrt(mean(v^2) + eps) * gain;  xa = T(x).  y0 / y1 may be split-K slices of a projection or the choices of a
 // routed feed-forward ([slices][n][ld]), summed here in slice order; y1 and bias may be NULL.
@@ -813,10 +848,13 @@ __global__ void attn_front_kernel(const float* __restrict__ P, int64_t ldp, int 
   const int pos = row_pos[r];
   const int half = rot / 2;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    double sn, cs;
-    sincos((double)pos * freq[i], &sn, &cs);
-    trig[i] = (float)cs * mag;
-    trig[half + i] = (float)sn * mag;
+    // angle and its reduction to [-pi, pi] in double, then the fp32 sincos of a small argument (see qk_norm_rope_cache_kernel)
+    const double ang = (double)pos * freq[i];
+    const double turns = rint(ang * 0.15915494309189535);
+    float sn, cs;
+    sincosf((float)fma(-turns, 6.283185307179586, ang), &sn, &cs);
+    trig[i] = cs * mag;
+    trig[half + i] = sn * mag;
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -1179,6 +1217,14 @@ extern "C" int prl_mlstm_out(const float* o_aug, int32_t n, int32_t H, int32_t d
   PRL_CHECK_ARG(o_aug && minv && g && gain && out && n >= 1 && H >= 1 && H <= 65535 && dv >= 1, "prl_mlstm_out: bad argument");
   dim3 grid(n, H);
   const int th = row_threads(dv);
+  if (!f32 && (int64_t)n * H >= 1024 && dv <= 512) {      // the fp32 mode keeps one order of summation for every batch size
+    const dim3 wgrid((unsigned)(((int64_t)n * H + 7) / 8));
+#define PRL_MW(NV) PRL_CUDA(launch_pdl((mlstm_out_warp_kernel<bf16, NV>), wgrid, dim3(256), (size_t)0, (cudaStream_t)st, o_aug, n, H, dv, minv, den_eps, g, ldg, gain, eps, (bf16*)out))
+    if (dv <= 64) PRL_MW(2); else if (dv <= 128) PRL_MW(4); else if (dv <= 256) PRL_MW(8); else PRL_MW(16);
+#undef PRL_MW
+    PRL_LAUNCH_CHECK();
+    return PRL_OK;
+  }
   if (f32) PRL_CUDA(launch_pdl(mlstm_out_kernel<float>, grid, dim3(th), (size_t)0, (cudaStream_t)st, o_aug, H, dv, minv, den_eps, g, ldg, gain, eps, (float*)out));
   else PRL_CUDA(launch_pdl(mlstm_out_kernel<bf16>, grid, dim3(th), (size_t)0, (cudaStream_t)st, o_aug, H, dv, minv, den_eps, g, ldg, gain, eps, (bf16*)out));
   PRL_LAUNCH_CHECK();

@@ -697,6 +697,83 @@ __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
   }
 }
 
+// ---- 4. for SCALAR recurrences: 64 tokens x 128 columns per CTA, 4 x 8 results per thread, key channels in rounds of eight per
+// key lane (whole lines of the state).  `ones` as in chunk_kernel.
+constexpr int kApplySmem = (kPiece * kTS + kPiece * kVS + 2 * kPiece) * (int)sizeof(float);
+
+__global__ void __launch_bounds__(256) apply_scalar_kernel(ScanArgs a, SplitArgs p, int ones) {
+  pdl_wait();
+  extern __shared__ __align__(16) float psm[];
+  float* wT = psm;                         // [channel of the round][token]: q_t times the decay from the piece's start through t
+  float* S = wT + kPiece * kTS;            // [channel of the round][column]
+  float* Sn = S + kPiece * kVS;            // [channel of the round]: the constant column's state
+  float* cum = Sn + kPiece;                // [token]
+  const int sub = blockIdx.x, h = blockIdx.y, vt = blockIdx.z, tid = threadIdx.x;
+  const int len = p.sub_len[sub], dk = a.dk, dv = a.dv, r = p.r, nv4 = (dv + 3) / 4;
+  const int64_t row0 = p.sub_start[sub];
+  const int nx = dv - (ones ? 1 : 0);
+  const bool apart = ones && nx % 4 == 0, side = apart && vt == 0;
+  const int cols = apart ? nx : dv;
+  const float* qb = a.qvec + a.off_q + h * dk;
+  const float* sc = p.scratch + (int64_t)sub * a.state_slot_stride + (int64_t)h * r * nv4 * 32;
+  if (tid < kPiece) cum[tid] = tid < len ? (a.dt_raw ? a.dt_raw[(row0 + tid) * a.ld_dt + a.off_dt + 2 * h] : a.a_log[h]) : 1.f;
+  __syncthreads();
+  if (tid == 0) {
+    float c = 1.f;
+#pragma unroll 8
+    for (int t = 0; t < kPiece; ++t) { c *= cum[t]; cum[t] = c; }
+  }
+  const int tx = tid % 16, ty = tid / 16;
+  float acc[4][8] = {}, extra = 0.f;
+  for (int i0 = 0; i0 < r; i0 += 8) {
+    const int ni = min(8, r - i0);
+    __syncthreads();
+    for (int e = tid; e < kPiece * kKeyLanes; e += 256) {          // tokens fastest
+      const int t = e % kPiece, dg = e / kPiece, d0 = dg * r + i0;
+      const float* qs = qb + (row0 + (t < len ? t : 0)) * a.ld_q + d0;
+      const float c = t < len ? cum[t] * a.q_scale : 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < ni) wT[(i * kKeyLanes + dg) * kTS + t] = (t < len && d0 + i < dk) ? qs[i] * c : 0.f;
+    }
+    for (int e = tid; e < ni * (kCC / 4) * kKeyLanes; e += 256) {  // key lanes fastest: whole 128-byte lines
+      const int dg = e % kKeyLanes, c4 = (e / kKeyLanes) % (kCC / 4), i = e / (kKeyLanes * (kCC / 4));
+      const int col4 = vt * (kCC / 4) + c4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (col4 * 4 < cols) v = *reinterpret_cast<const float4*>(sc + (((int64_t)(i0 + i) * nv4 + col4) * kKeyLanes + dg) * 4);
+      *reinterpret_cast<float4*>(S + (i * kKeyLanes + dg) * kVS + c4 * 4) = v;
+    }
+    if (side && tid < ni * kKeyLanes)
+      Sn[tid] = sc[(((int64_t)(i0 + tid / kKeyLanes) * nv4 + nx / 4) * kKeyLanes + tid % kKeyLanes) * 4];
+    __syncthreads();
+#pragma unroll 4
+    for (int d = 0; d < ni * kKeyLanes; ++d) {
+      const float4 w4 = *reinterpret_cast<const float4*>(wT + d * kTS + ty * 4);
+      const float4 s0 = *reinterpret_cast<const float4*>(S + d * kVS + tx * 4);
+      const float4 s1 = *reinterpret_cast<const float4*>(S + d * kVS + 64 + tx * 4);
+      const float ww[4] = {w4.x, w4.y, w4.z, w4.w}, ss[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(ww[i], ss[j], acc[i][j]);
+    }
+    if (side && tid < kPiece)
+      for (int d = 0; d < ni * kKeyLanes; ++d) extra = fmaf(wT[d * kTS + tid], Sn[d], extra);
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = ty * 4 + i;
+    if (t >= len) continue;
+    float* o = a.out + (row0 + t) * a.ld_out + h * dv;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int col = vt * kCC + (j < 4 ? 0 : 64) + tx * 4 + (j & 3);
+      if (col < cols) o[col] += acc[i][j];
+    }
+  }
+  if (side && tid < len) a.out[(row0 + tid) * a.ld_out + h * dv + nx] += extra;
+}
+
 template <int SSD>
 int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st, int ones = 0) {
   p.r = plan_r(a.dk);
@@ -721,6 +798,14 @@ int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st,
   const int nv4 = (a.dv + 3) / 4, per_head = p.r * nv4 * 32;
   PRL_CUDA(launch_pdl(carry_kernel, dim3((per_head + 1023) / 1024, a.heads, n_seg), dim3(256), (size_t)0, st, a, p));
   PRL_LAUNCH_CHECK();
+  if (SSD == kScalar) {
+    const int cols = (ones && (a.dv - ones) % 4 == 0) ? a.dv - ones : a.dv;
+    static SmemAttr attr = {};
+    PRL_CUDA(ensure_smem(apply_scalar_kernel, kApplySmem, attr));
+    PRL_CUDA(launch_pdl(apply_scalar_kernel, dim3(n_sub, a.heads, (cols + kCC - 1) / kCC), dim3(256), (size_t)kApplySmem, st, a, p, ones));
+    PRL_LAUNCH_CHECK();
+    return PRL_OK;
+  }
   PRL_CUDA(launch_pdl(apply_kernel<SSD>, dim3(n_sub, a.heads, (a.dv + kApplyCols - 1) / kApplyCols), dim3(256), (size_t)0, st, a, p));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
