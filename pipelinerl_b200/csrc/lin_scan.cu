@@ -342,6 +342,8 @@ __global__ void gla_decay_kernel(float* __restrict__ z, int64_t ldz, const float
 //      c), S <- D_c * S + L_c; the last S is the sequence's new state;
 //   4. apply_kernel adds what the incoming state contributes: o_t += (q_t * prod_{s <= t in piece} a_s)^T S_before(c),
 //      a [tokens x dk] x [dk x dv] product per piece and head from shared memory.
+// SCALAR recurrences (one decay and one input scale per head and token) run steps 1, 2 and 4 as register-blocked products
+// instead (chunk_kernel, apply_scalar_kernel).
 // All of it is fp32; the result differs from the token-by-token walk by the rounding of a different summation order.
 constexpr int kPiece = 64;          // tokens per piece at most (the token tile of apply_kernel)
 constexpr int kApplyCols = 64;      // value columns per CTA of apply_kernel
@@ -554,7 +556,7 @@ __global__ void __launch_bounds__(256) chunk_kernel(ScanArgs a, SplitArgs p, int
 
 template <int MODE>
 __global__ void __launch_bounds__(256) piece_decay_kernel(ScanArgs a, SplitArgs p) {
-  constexpr bool SSD = MODE == kSsd, SCL = MODE == kScalar;
+  constexpr bool SSD = MODE == kSsd;
   pdl_wait();
   const int sub = blockIdx.x, h = blockIdx.y, d = threadIdx.x, dpad = kKeyLanes * p.r;
   if (d >= dpad) return;
@@ -562,15 +564,13 @@ __global__ void __launch_bounds__(256) piece_decay_kernel(ScanArgs a, SplitArgs 
   const int64_t row0 = p.sub_start[sub];
   float prod = 1.f;                    // eight loads in flight at a time; the product keeps the order of the tokens
   const float neg_a = SSD ? -expf(a.a_log[h]) : 0.f, dtb = SSD ? a.dt_bias[h] : 0.f;
-  const float cdec = (SCL && !a.dt_raw) ? a.a_log[h] : 1.f;
-  if (SSD || SCL || d < a.dk) {
+  if (SSD || d < a.dk) {
     for (int t0 = 0; t0 < len; t0 += 8) {
       float v[8];
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int t = min(t0 + j, len - 1);
-        if (SCL) v[j] = a.dt_raw ? a.dt_raw[(row0 + t) * a.ld_dt + a.off_dt + 2 * h] : cdec;
-        else v[j] = SSD ? a.dt_raw[(row0 + t) * a.ld_dt + a.off_dt + h] : a.avec[(row0 + t) * a.ld_a + h * a.dk + d];
+        v[j] = SSD ? a.dt_raw[(row0 + t) * a.ld_dt + a.off_dt + h] : a.avec[(row0 + t) * a.ld_a + h * a.dk + d];
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j)
@@ -614,7 +614,7 @@ __global__ void __launch_bounds__(256) carry_kernel(ScanArgs a, SplitArgs p) {
 
 template <int MODE>
 __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
-  constexpr bool SSD = MODE == kSsd, SCL = MODE == kScalar, ONE = SSD || SCL;
+  constexpr bool SSD = MODE == kSsd;
   pdl_wait();
   __shared__ __align__(16) float wT[kApplyKeys * kWStride];     // [key channel][token]: q_t[d] * (decay from the piece's start through t)
   __shared__ __align__(16) float S[kApplyKeys * kApplyCols];    // [key channel][column]: the state before this piece
@@ -628,10 +628,9 @@ __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
   const float* sc = p.scratch + (int64_t)sub * a.state_slot_stride + (int64_t)h * r * nv4 * 32;
   const int tx = tid % 16, ty = tid / 16;      // columns 4 tx .., tokens 4 ty ..
   float acc[4][4] = {};
-  if (ONE) {
+  if (SSD) {
     if (tid < kPiece) {
-      if (SSD) dec[tid] = tid < len ? expf(-expf(a.a_log[h]) * softplus_f(a.dt_raw[(row0 + tid) * a.ld_dt + a.off_dt + h] + a.dt_bias[h])) : 1.f;
-      else dec[tid] = tid < len ? (a.dt_raw ? a.dt_raw[(row0 + tid) * a.ld_dt + a.off_dt + 2 * h] : a.a_log[h]) : 1.f;
+      dec[tid] = tid < len ? expf(-expf(a.a_log[h]) * softplus_f(a.dt_raw[(row0 + tid) * a.ld_dt + a.off_dt + h] + a.dt_bias[h])) : 1.f;
     }
     __syncthreads();
     if (tid == 0) {
@@ -645,7 +644,7 @@ __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
   // wait for each load in turn) -- then the state rows of these channels, then the product.
   for (int d0 = 0; d0 < dk; d0 += kApplyKeys) {
     const int nd = min(kApplyKeys, dk - d0);
-    if (!ONE) {
+    if (!SSD) {
       for (int e = tid; e < kPiece * nd; e += 256) {
         const int t = e / nd, d = e - t * nd;
         wT[d * kWStride + t] = t < len ? a.avec[(row0 + t) * a.ld_a + h * dk + d0 + d] : 1.f;
@@ -660,7 +659,7 @@ __global__ void __launch_bounds__(256) apply_kernel(ScanArgs a, SplitArgs p) {
     }
     for (int e = tid; e < kPiece * nd; e += 256) {
       const int t = e / nd, d = e - t * nd;
-      const float cum = ONE ? dec[t] : wT[d * kWStride + t];
+      const float cum = SSD ? dec[t] : wT[d * kWStride + t];
       wT[d * kWStride + t] = t < len ? cum * qbase[(row0 + t) * a.ld_q + d0 + d] * a.q_scale : 0.f;
     }
     for (int e = tid; e < r * (kApplyCols / 4) * kKeyLanes; e += 256) {      // key lanes fastest: whole 128-byte lines
@@ -777,7 +776,7 @@ __global__ void __launch_bounds__(256) apply_scalar_kernel(ScanArgs a, SplitArgs
 template <int SSD>
 int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st, int ones = 0) {
   p.r = plan_r(a.dk);
-  if (SSD == kScalar) {
+  if constexpr (SSD == kScalar) {
     const int nx = a.dv - ones;
     const int vec4 = a.dk % 4 == 0 && nx % 4 == 0 && a.ld_k % 4 == 0 && a.ld_q % 4 == 0 && a.ld_x % 4 == 0 && a.off_k % 4 == 0 &&
                      a.off_q % 4 == 0 && a.off_x % 4 == 0 && aligned16(a.kvec) && aligned16(a.qvec) && aligned16(a.xval);
@@ -798,16 +797,16 @@ int launch_split(ScanArgs a, int n_seg, SplitArgs p, int n_sub, cudaStream_t st,
   const int nv4 = (a.dv + 3) / 4, per_head = p.r * nv4 * 32;
   PRL_CUDA(launch_pdl(carry_kernel, dim3((per_head + 1023) / 1024, a.heads, n_seg), dim3(256), (size_t)0, st, a, p));
   PRL_LAUNCH_CHECK();
-  if (SSD == kScalar) {
+  if constexpr (SSD == kScalar) {
     const int cols = (ones && (a.dv - ones) % 4 == 0) ? a.dv - ones : a.dv;
     static SmemAttr attr = {};
     PRL_CUDA(ensure_smem(apply_scalar_kernel, kApplySmem, attr));
     PRL_CUDA(launch_pdl(apply_scalar_kernel, dim3(n_sub, a.heads, (cols + kCC - 1) / kCC), dim3(256), (size_t)kApplySmem, st, a, p, ones));
     PRL_LAUNCH_CHECK();
-    return PRL_OK;
+  } else {
+    PRL_CUDA(launch_pdl(apply_kernel<SSD>, dim3(n_sub, a.heads, (a.dv + kApplyCols - 1) / kApplyCols), dim3(256), (size_t)0, st, a, p));
+    PRL_LAUNCH_CHECK();
   }
-  PRL_CUDA(launch_pdl(apply_kernel<SSD>, dim3(n_sub, a.heads, (a.dv + kApplyCols - 1) / kApplyCols), dim3(256), (size_t)0, st, a, p));
-  PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
 

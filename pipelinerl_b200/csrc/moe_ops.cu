@@ -1,9 +1,9 @@
 // Routed feed-forward (mixture of experts) over a packed batch of n token rows, without a host round trip: the number
 // of rows each expert gets stays on the device, so the whole layer can sit in a CUDA graph.
 //
-//   1. route:  (prl_moe_route, prl_moe_router) per row, the `top` experts with the largest router logits (ties: the lower index), each with the weight
-//              sigmoid(logit) or softmax over the chosen; an optional bias per expert joins the logits first; choice c
-//              of row t is the PAIR c * n + t.  prl_moe_choose instead takes ready logits and ranks the outputs by their
+//   1. route:  (prl_moe_route, prl_moe_router) per row, the `top` experts with the largest router logits (ties: the lower
+//              index), each with the weight sigmoid(logit) or softmax over the chosen; an optional bias per expert joins
+//              the logits first; choice c of row t is the PAIR c * n + t.  prl_moe_choose instead takes ready logits and ranks the outputs by their
 //              softmax share plus a correction (which the weights do not see), inside the best groups of outputs only;
 //              outputs past the experts ("identity") hand the input through: their pairs are chosen and weighted like
 //              the others but join no expert's rows.

@@ -232,6 +232,19 @@ def test_far_tokens_in_the_memory_cell(cuda_device):
         assert fc.rel_err(fc.stream_logits(eng, toks, [140, 33, 64, 63]), ref) < F32_TOL
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(3, 10, 14), (2, 128, 256), (1, 256, 40), (4, 4, 330)])
+def test_one_kernel_token_step_equals_the_separate_kernels(cuda_device, heads, dim, vdim):
+    """The cell's token step in one kernel against gates, scan and output kernels: the same sums in the same order."""
+    config = fc.model([C(heads=heads, dim=dim, vdim=vdim)], width=48)
+    wt = fc.weights(config, 5)
+    toks = fc.tokens_for(config, 40, seed=6)
+    eng = fc.build_engine(config, wt, torch.float32, cuda_device)
+    fused = fc.stream_logits(eng, toks, [3])
+    eng.unfused_cell = True
+    assert fc.rel_err(fused, fc.stream_logits(eng, toks, [3])) < 1e-6
+    assert fc.rel_err(fused, fc.oracle_logits(config, wt, toks)) < F32_TOL
+
+
 def test_choice_of_experts(cuda_device):
     """Choice scores that are never a close call and all negative (closed groups must count as minus infinity, not zero),
     corrections large enough to change the choice: a wrong group rule, a correction inside the weights, renormalised
