@@ -766,23 +766,31 @@ int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is
 int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
                  int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
                  int64_t max_tiles, int64_t N, int64_t K, float* C, int64_t ldc, int32_t c_perm, prl_stream_t stream);
-/* choice from ready logits: outputs ranked by softmax share + correction (nullable) inside the `keep` best of `groups`
- * equal groups, weighted by the share alone; outputs experts .. outputs - 1 hand the input through (no rows) */
+/* choice from ready logits: outputs scored by softmax share (sigmoid 0) or sigmoid (1), ranked by score + correction
+ * (nullable) inside the `keep` best of `groups` equal groups (a group's rank: the sum of its group_top = 1 or 2 best), weighted
+ * by the score alone (renorm: over the chosen scores' sum) times scale; outputs experts .. outputs - 1 hand the input through
+ * (no rows).  _router_choose: the router product in the same launch */
 int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
-                   int32_t top, int32_t groups, int32_t keep, int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm,
-                   int32_t* meta, int32_t* tiles, prl_stream_t stream);
+                   int32_t top, int32_t groups, int32_t keep, int32_t group_top, int32_t sigmoid, int32_t renorm, float scale,
+                   int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta, int32_t* tiles,
+                   prl_stream_t stream);
+int prl_moe_router_choose(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is_f32, const float* correction, int32_t n,
+                          int32_t W, int32_t experts, int32_t outputs, int32_t top, int32_t groups, int32_t keep, int32_t group_top,
+                          int32_t sigmoid, int32_t renorm, float scale, int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm,
+                          int32_t* meta, int32_t* tiles, prl_stream_t stream);
 /* many rows per expert: rows gathered into sorted order, then a persistent tcgen05 grouped GEMM over row tiles of 256; wsel
- * NULL: fp32 rows perm[s] of out, else bf16 rows s = relu(.)^2 * wsel[perm[s]] */
+ * NULL: fp32 rows perm[s] of out, else bf16 rows s = act(.) * wsel[perm[s]], act 1: relu(.)^2, 2: gelu (error function) */
 int prl_moe_gather(const void* x_bf16, const int32_t* perm, const int32_t* meta, int32_t n, int32_t pairs, int32_t W, void* out,
                    prl_stream_t stream);
 int prl_moe_gemm_tc(const void* A_bf16, int64_t rows_cap, const void* W_bf16, int32_t experts, int64_t N, int64_t K,
-                    const int32_t* perm, const int32_t* meta, const int32_t* tiles, const float* wsel, void* out, int64_t ldc,
-                    prl_stream_t stream);
-/* prl_moe_gemm with act[s] = relu(product)^2 * wsel[pair] written in sorted order in A's type (the second product's operand) */
-int prl_moe_gemm_relu2(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
-                       int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
-                       int64_t max_tiles, int64_t N, int64_t K, const float* wsel, void* act, int64_t ld_act,
-                       prl_stream_t stream);
+                    const int32_t* perm, const int32_t* meta, const int32_t* tiles, const float* wsel, int32_t act, void* out,
+                    int64_t ldc, prl_stream_t stream);
+/* prl_moe_gemm with out[s] = act(product) * wsel[pair] written in sorted order in A's type (the second product's operand);
+ * act 1: relu(.)^2, 2: gelu (error function) */
+int prl_moe_gemm_act(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                     int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
+                     int64_t max_tiles, int64_t N, int64_t K, int32_t act, const float* wsel, void* out, int64_t ld_out,
+                     prl_stream_t stream);
 int prl_moe_glu(const float* gate_up, int64_t ld, int64_t pairs, int32_t F, const int32_t* perm, const float* wsel,
                 float limit, float beta, void* out, int32_t f32, prl_stream_t stream);
 
@@ -869,6 +877,8 @@ int prl_attn_front(const float* P, int64_t ldp, int32_t off_q, int32_t off_k, in
                    float mag, int32_t v_norm, int32_t v_blend, const float* v_lambda, float* v_first, const int32_t* row_pos,
                    const int32_t* row_slot, const int32_t* block_table, int32_t max_blocks, int32_t page_size, void* q_out,
                    void* k_pool, void* v_pool, int32_t f32, prl_stream_t stream);
+/* z <- cap * tanh(z / cap), `count` contiguous values in place */
+int prl_soft_cap(float* z, int64_t count, float cap, prl_stream_t stream);
 /* out[r][h * dv + j] = T(o[r][h * dv + j] * sigmoid(g[r][h])) */
 int prl_gate_heads(const void* o, int32_t o_f32, int64_t ldo, const float* g, int64_t ldg, int32_t n, int32_t H, int32_t dv,
                    void* out, int32_t f32, prl_stream_t stream);

@@ -64,11 +64,12 @@ struct TnParams {
   int glu_gelu;            // 1 (with swiglu_fp32): gelu(gate) * up, the tanh form of gelu
   // grouped rows (g_tiles != NULL): work item t is row tile t / n_tiles of a device table [expert, first row, rows <= 256] (g_meta[0]
   // entries) against columns (t % n_tiles) * 256 .. of the expert's rows of B (stacked, N rows each).  Row s of the sorted A
-  // goes to C row g_perm[s] (fp32) or, with g_w, to act row s as bf16 relu(.)^2 * g_w[g_perm[s]]
+  // goes to C row g_perm[s] (fp32) or, with g_w, to act row s as bf16 act(.) * g_w[g_perm[s]]
   const int32_t* g_tiles;
   const int32_t* g_meta;
   const int32_t* g_perm;
   const float* g_w;
+  int g_act;               // 1: relu(.)^2, 2: gelu in its error-function form
   // head epilogue (kHead): logits never leave TMEM/registers
   const int64_t* targets;  // [M] or NULL
   float4* head_part;       // [n_tiles, M]: (max, sum exp, sum exp*z, target logit or -inf) of one 256-column vocabulary tile
@@ -432,7 +433,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float z = fmaxf(v[j], 0.f);
-            v[j] = z * z * row_w;
+            v[j] = (p.g_act == 2 ? 0.5f * v[j] * (1.f + erff(v[j] * 0.70710678118654752f)) : z * z) * row_w;
           }
           if (full && ((p.ld_act & 7) == 0)) {
 #pragma unroll
@@ -712,11 +713,12 @@ extern "C" int prl_gemm_tn_dual(const void* A1, const void* B1, int64_t K1, cons
 
 // Grouped GEMM over rows sorted by expert (csrc/moe_ops.cu tables with row tiles of at most 256): A [rows_cap, K] bf16 holds the sorted
 // rows, W the experts' matrices stacked ([experts * N, K]).  wsel NULL: C[perm[s]] (fp32, row stride ldc) = A[s] W_e^T;
-// otherwise out[s] (bf16, row stride ldc) = relu(A[s] W_e^T)^2 * wsel[perm[s]].  The number of tiles stays on the device: the
+// otherwise out[s] (bf16, row stride ldc) = act(A[s] W_e^T) * wsel[perm[s]], act 1: relu(.)^2, 2: gelu (error function).  The number of tiles stays on the device: the
 // persistent clusters walk meta[0] * ceil(N / 256) items.
 extern "C" int prl_moe_gemm_tc(const void* A, int64_t rows_cap, const void* W, int32_t experts, int64_t N, int64_t K, const int32_t* perm,
-                               const int32_t* meta, const int32_t* tiles, const float* wsel, void* out, int64_t ldc,
+                               const int32_t* meta, const int32_t* tiles, const float* wsel, int32_t act, void* out, int64_t ldc,
                                prl_stream_t stream_) {
+  PRL_CHECK_ARG(!wsel || act == 1 || act == 2, "prl_moe_gemm_tc: unknown activation %d", act);
   PRL_CHECK_ARG(A && W && perm && meta && tiles && out, "prl_moe_gemm_tc: NULL argument");
   PRL_CHECK_ARG(rows_cap >= 1 && experts >= 1 && N >= 1 && K >= 8 && K % 8 == 0 && ldc >= N && experts * N < (1ll << 31),
                 "prl_moe_gemm_tc: bad shape (rows=%lld experts=%d N=%lld K=%lld)", (long long)rows_cap, experts, (long long)N, (long long)K);
@@ -726,7 +728,7 @@ extern "C" int prl_moe_gemm_tc(const void* A, int64_t rows_cap, const void* W, i
   p.m_tiles = 1;
   p.n_tiles = (int)((N + kTile - 1) / kTile);
   p.alpha = 1.f;
-  p.g_tiles = tiles; p.g_meta = meta; p.g_perm = perm; p.g_w = wsel;
+  p.g_tiles = tiles; p.g_meta = meta; p.g_perm = perm; p.g_w = wsel; p.g_act = act;
   if (wsel) { p.act = (__nv_bfloat16*)out; p.ld_act = ldc; }
   else { p.C = out; p.ldc = ldc; p.c_f32 = 1; }
   CUtensorMap ta, tb;

@@ -914,6 +914,13 @@ __global__ void attn_front_kernel(const float* __restrict__ P, int64_t ldp, int 
   }
 }
 
+// z <- cap * tanh(z / cap): the model's capped logits, in place
+__global__ void soft_cap_kernel(float* __restrict__ z, int64_t count, float cap) {
+  pdl_wait();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (int64_t)gridDim.x * blockDim.x)
+    z[i] = cap * tanhf(z[i] / cap);
+}
+
 // out[r][h * dv + j] = T(o[r][h * dv + j] * sigmoid(g[r][h])): one gate per head on an attention output
 template <typename T, typename TO>
 __global__ void gate_heads_kernel(const TO* __restrict__ o, int64_t ldo, const float* __restrict__ g, int64_t ldg, int H,
@@ -1266,6 +1273,14 @@ extern "C" int prl_attn_front(const float* P, int64_t ldp, int32_t off_q, int32_
   const size_t smem = (size_t)(rot > 0 ? rot : 1) * sizeof(float);
   if (f32) PRL_CUDA(launch_pdl(attn_front_kernel<float>, dim3(n), dim3(32 * warps), smem, (cudaStream_t)st, P, ldp, off_q, off_k, off_v, H, G, dim, vdim, q_bias, k_bias, v_bias, qk_norm, q_gain, k_gain, gain_period, eps, rot, freq, mag, v_norm, v_blend, v_lambda, v_first, row_pos, row_slot, block_table, max_blocks, page_size, (float*)q_out, (float*)k_pool, (float*)v_pool));
   else PRL_CUDA(launch_pdl(attn_front_kernel<bf16>, dim3(n), dim3(32 * warps), smem, (cudaStream_t)st, P, ldp, off_q, off_k, off_v, H, G, dim, vdim, q_bias, k_bias, v_bias, qk_norm, q_gain, k_gain, gain_period, eps, rot, freq, mag, v_norm, v_blend, v_lambda, v_first, row_pos, row_slot, block_table, max_blocks, page_size, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool));
+  PRL_LAUNCH_CHECK();
+  return PRL_OK;
+}
+
+extern "C" int prl_soft_cap(float* z, int64_t count, float cap, prl_stream_t st) {
+  PRL_CHECK_ARG(z && count >= 1 && cap > 0.f, "prl_soft_cap: bad argument");
+  const int64_t blocks = (count + 1023) / 1024;
+  PRL_CUDA(launch_pdl(soft_cap_kernel, dim3((unsigned)(blocks < 4096 ? blocks : 4096)), dim3(256), (size_t)0, (cudaStream_t)st, z, count, cap));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }

@@ -3,8 +3,9 @@
 //
 //   1. route:  (prl_moe_route, prl_moe_router) per row, the `top` experts with the largest router logits (ties: the lower
 //              index), each with the weight sigmoid(logit) or softmax over the chosen; an optional bias per expert joins
-//              the logits first; choice c of row t is the PAIR c * n + t.  prl_moe_choose instead takes ready logits and ranks the outputs by their
-//              softmax share plus a correction (which the weights do not see), inside the best groups of outputs only;
+//              the logits first; choice c of row t is the PAIR c * n + t.  prl_moe_choose (ready logits) and
+//              prl_moe_router_choose instead rank the outputs by their softmax share or sigmoid plus a correction (which the
+//              weights do not see), inside the best groups of outputs only; the weights may be divided by their sum;
 //              outputs past the experts ("identity") hand the input through: their pairs are chosen and weighted like
 //              the others but join no expert's rows.
 //   2. group:  a stable counting sort of the pairs by expert (one CTA): perm[s] = pair at sorted place s, and a table
@@ -84,16 +85,111 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
     for (int c = 0; c < top; ++c) wsel[(int64_t)c * n + t] /= denom;
 }
 
+// How a router's outputs are scored, ranked and weighted (prl_moe_choose, prl_moe_router_choose).
+struct ChoiceRule {
+  const float* correction;    // per output, joins the scores for the ranking only; NULL: none
+  int top, groups, keep;      // `groups` equal groups of neighbours of which the `keep` best are open
+  int group_top;              // a group is ranked by the sum of its `group_top` (1 or 2) best choice scores
+  int sigmoid;                // score of an output: 1 the sigmoid of its logit, 0 its softmax share over all outputs
+  int renorm;                 // 1: the chosen scores are divided by their sum (+ 1e-20)
+  float scale;                // constant factor on the weights
+};
+
+// The choice for one row by one warp: c [E] and gs [groups] are the warp's scratch in shared memory, z [E] the logits.
+// Outputs are ranked by score + correction, closed groups count as minus infinity; ties go to the lower index.
+__device__ __forceinline__ void choose_row(const float* z, int E, const ChoiceRule& r, float* c, float* gs, int n, int t,
+                                           int32_t* __restrict__ sel, float* __restrict__ wsel) {
+  const int lane = threadIdx.x & 31;
+  float zmax = 0.f, inv = 1.f;
+  if (!r.sigmoid) {
+    zmax = -INFINITY;
+    for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
+    zmax = warp_max(zmax);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
+    inv = 1.f / warp_sum(sum);
+  }
+  auto score = [&](int e) { return r.sigmoid ? sigmoid_f(z[e]) : expf(z[e] - zmax) * inv; };
+  for (int e = lane; e < E; e += 32) c[e] = score(e) + (r.correction ? r.correction[e] : 0.f);
+  __syncwarp();
+  auto best_of = [&](const float* v, int count) {          // index of the largest entry, the lowest on a tie
+    float best = -INFINITY;
+    int arg = 0x7fffffff;
+    for (int e = lane; e < count; e += 32)
+      if (v[e] > best) { best = v[e]; arg = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+    }
+    return arg;
+  };
+  if (r.keep < r.groups) {
+    const int size = E / r.groups;
+    for (int g = lane; g < r.groups; g += 32) {
+      float m = -INFINITY, m2 = -INFINITY;
+      for (int e = 0; e < size; ++e) {
+        const float v = c[g * size + e];
+        m2 = fmaxf(m2, fminf(m, v));
+        m = fmaxf(m, v);
+      }
+      gs[g] = (r.group_top > 1 && size > 1) ? m + m2 : m;
+    }
+    __syncwarp();
+    for (int k = 0; k < r.keep; ++k) {                     // an open group is marked by taking it out of the ranking
+      const int g = best_of(gs, r.groups);
+      if (lane == 0 && g < r.groups) gs[g] = -INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gs[e / size] != -INFINITY) c[e] = -INFINITY;     // still ranked: a closed group
+    __syncwarp();
+  }
+  float total = 0.f;
+  for (int k = 0; k < r.top; ++k) {
+    const int e = best_of(c, E);
+    const bool ok = e < E;                                 // always, for finite logits
+    const float w = ok ? score(e) : 0.f;
+    total += w;
+    if (lane == 0) {
+      sel[(int64_t)k * n + t] = ok ? e : 0;
+      wsel[(int64_t)k * n + t] = w * r.scale;
+      if (ok) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  if (r.renorm && lane == 0)
+    for (int k = 0; k < r.top; ++k) {
+      const float w = wsel[(int64_t)k * n + t];            // written by this lane
+      wsel[(int64_t)k * n + t] = w / (total + 1e-20f);
+    }
+}
+
+// Choice from ready logits, one warp per row.
+constexpr int kChooseWarps = 4;
+__global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const float* __restrict__ logits, int64_t ld, int n, int E,
+                                                                       ChoiceRule rule, int32_t* __restrict__ sel,
+                                                                       float* __restrict__ wsel) {
+  pdl_wait();
+  extern __shared__ float csm[];                 // per warp: [E] choice scores | [groups] group scores
+  const int warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * kChooseWarps + warp;
+  if (t >= n) return;
+  float* c = csm + (size_t)warp * (E + rule.groups);
+  choose_row(logits + (int64_t)t * ld, E, rule, c, c + E, n, t, sel, wsel);
+}
+
 // Router and choice in one kernel: logits[e] = x . Wr[e] in fp32 (block per row, the row staged in shared memory, warps
 // take experts in turn, a lane sums every 32nd channel, then the warp's shuffle tree: a fixed order), then the top-k
-// pass of moe_route_kernel over the logits in shared memory.
-template <typename TX, typename TW>
+// pass of moe_route_kernel over the logits in shared memory (RULED: choose_row instead, with scratch behind the logits).
+template <typename TX, typename TW, bool RULED>
 __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ Wr,
                                                          const float* __restrict__ bias, int n, int W, int E, int top,
-                                                         int softmax_weights, int32_t* __restrict__ sel,
+                                                         int softmax_weights, ChoiceRule rule, int32_t* __restrict__ sel,
                                                          float* __restrict__ wsel) {
   pdl_wait();
-  extern __shared__ float rsm[];       // [W] the row | [E] logits
+  extern __shared__ float rsm[];       // [W] the row | [E] logits | RULED: [E] choice scores | [groups] group scores
   float* xs = rsm;
   float* z = rsm + W;
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -110,6 +206,10 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ 
   }
   __syncthreads();
   if (warp != 0) return;
+  if constexpr (RULED) {
+    choose_row(z, E, rule, z + E, z + 2 * E, n, t, sel, wsel);
+    return;
+  }
   uint32_t taken = 0;
   float zsel_max = 0.f, denom = 0.f;
   for (int c = 0; c < top; ++c) {
@@ -147,72 +247,6 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ 
   }
   if (softmax_weights && lane == 0)
     for (int c = 0; c < top; ++c) wsel[(int64_t)c * n + t] /= denom;
-}
-
-// Choice from ready logits, one warp per row.  s = softmax(z) over all E outputs; outputs are ranked by c = s + correction.
-// The outputs form `groups` equal groups of neighbours ranked by their best c; only the `keep` best groups are open.
-// The `top` best open outputs (ties: the lower index) are chosen, each with its weight s.
-constexpr int kChooseWarps = 4;
-__global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const float* __restrict__ logits, int64_t ld,
-                                                                       const float* __restrict__ correction, int n, int E, int top,
-                                                                       int groups, int keep, int32_t* __restrict__ sel,
-                                                                       float* __restrict__ wsel) {
-  pdl_wait();
-  extern __shared__ float csm[];                 // per warp: [E] choice scores | [groups] group scores
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * kChooseWarps + warp;
-  if (t >= n) return;
-  float* c = csm + (size_t)warp * (E + groups);
-  float* gs = c + E;
-  const float* z = logits + (int64_t)t * ld;
-  float zmax = -INFINITY;
-  for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
-  zmax = warp_max(zmax);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
-  const float inv = 1.f / warp_sum(sum);
-  for (int e = lane; e < E; e += 32) c[e] = expf(z[e] - zmax) * inv + (correction ? correction[e] : 0.f);
-  __syncwarp();
-  auto best_of = [&](const float* v, int count) {          // index of the largest entry, the lowest on a tie
-    float best = -INFINITY;
-    int arg = 0x7fffffff;
-    for (int e = lane; e < count; e += 32)
-      if (v[e] > best) { best = v[e]; arg = e; }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-    }
-    return arg;
-  };
-  if (keep < groups) {
-    const int size = E / groups;
-    for (int g = lane; g < groups; g += 32) {
-      float m = -INFINITY;
-      for (int e = 0; e < size; ++e) m = fmaxf(m, c[g * size + e]);
-      gs[g] = m;
-    }
-    __syncwarp();
-    for (int k = 0; k < keep; ++k) {                       // an open group is marked by taking it out of the ranking
-      const int g = best_of(gs, groups);
-      if (lane == 0 && g < groups) gs[g] = -INFINITY;
-      __syncwarp();
-    }
-    for (int e = lane; e < E; e += 32)
-      if (gs[e / size] != -INFINITY) c[e] = -INFINITY;     // still ranked: a closed group
-    __syncwarp();
-  }
-  for (int k = 0; k < top; ++k) {
-    const int e = best_of(c, E);
-    if (lane == 0) {
-      const bool ok = e < E;                               // always, for finite logits
-      sel[(int64_t)k * n + t] = ok ? e : 0;
-      wsel[(int64_t)k * n + t] = ok ? expf(z[e] - zmax) * inv : 0.f;
-      if (ok) c[e] = -INFINITY;
-    }
-    __syncwarp();
-  }
 }
 
 // meta[0] = number of tiles, meta[1] = sorted pairs; tiles[3 * i + {0, 1, 2}] = expert, first sorted place, rows (<= tile_rows)
@@ -268,8 +302,19 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
   for (int i = threadIdx.x; i < units; i += 128) dst[i] = src[i];
 }
 
-// RELU2: C is the next product's operand (type TA), C[row] = relu(product)^2 * wsel[pair]
-template <typename TA, typename TW, bool RELU2>
+// ACT: what the product becomes before it is stored.  kActNone: C fp32, the product itself; otherwise C is the next
+// product's operand (type TA), C[row] = act(product) * wsel[pair]
+constexpr int kActNone = 0, kActRelu2 = 1, kActGelu = 2;      // relu(z)^2 | z Phi(z), the error-function form
+template <int ACT> __device__ __forceinline__ float expert_act(float z) {
+  if constexpr (ACT == kActRelu2) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  } else {
+    return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+  }
+}
+
+template <typename TA, typename TW, int ACT>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A, int64_t lda, int a_mod,
                                                        const TW* __restrict__ W, int64_t expert_stride, int64_t ldw,
                                                        const int32_t* __restrict__ perm, const int32_t* __restrict__ meta,
@@ -288,7 +333,7 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
   if (tid < kTile) {
     const int s = s0 + min(tid, M - 1);
     const int p = perm[s];
-    if constexpr (RELU2) c_w[tid] = wsel[p];
+    if constexpr (ACT != kActNone) c_w[tid] = wsel[p];
     a_row[tid] = a_mod > 0 ? p % a_mod : s;
     c_row[tid] = c_perm ? p : s;
   }
@@ -335,9 +380,8 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
     for (int j = 0; j < 4; ++j) {
       const int nn = n0 + tn + j;
       if (nn >= N) continue;
-      if constexpr (RELU2) {
-        const float z = fmaxf(acc[i][j], 0.f);
-        reinterpret_cast<TA*>(C_v)[row * ldc + nn] = TA(z * z * c_w[tm + i]);
+      if constexpr (ACT != kActNone) {
+        reinterpret_cast<TA*>(C_v)[row * ldc + nn] = TA(expert_act<ACT>(acc[i][j]) * c_w[tm + i]);
       } else {
         reinterpret_cast<float*>(C_v)[row * ldc + nn] = acc[i][j];
       }
@@ -366,7 +410,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <bool RELU2>
+template <int ACT>
 __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, int a_mod,
                                                            const __nv_bfloat16* __restrict__ W, int64_t expert_stride,
                                                            int64_t ldw, const int32_t* __restrict__ perm,
@@ -388,7 +432,7 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
   if (tid < kTile) {
     const int s = s0 + min(tid, M - 1);
     const int p = perm[s];
-    if constexpr (RELU2) c_w[tid] = wsel[p];
+    if constexpr (ACT != kActNone) c_w[tid] = wsel[p];
     a_row[tid] = a_mod > 0 ? p % a_mod : s;
     c_row[tid] = c_perm ? p : s;
   }
@@ -452,15 +496,14 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
       const int m = wm + 16 * i + (lane >> 2) + 8 * half;
       if (m >= M) continue;
       const int64_t at = (int64_t)c_row[m] * ldc;
-      if constexpr (RELU2) {
+      if constexpr (ACT != kActNone) {
         __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(C_v) + at;
         const float w = c_w[m];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int nn = n0 + wn + 8 * j + (lane & 3) * 2;
-          const float z0 = fmaxf(acc[i][j][2 * half], 0.f), z1 = fmaxf(acc[i][j][2 * half + 1], 0.f);
-          if (nn < N) crow[nn] = __float2bfloat16_rn(z0 * z0 * w);
-          if (nn + 1 < N) crow[nn + 1] = __float2bfloat16_rn(z1 * z1 * w);
+          if (nn < N) crow[nn] = __float2bfloat16_rn(expert_act<ACT>(acc[i][j][2 * half]) * w);
+          if (nn + 1 < N) crow[nn + 1] = __float2bfloat16_rn(expert_act<ACT>(acc[i][j][2 * half + 1]) * w);
         }
         continue;
       }
@@ -526,47 +569,77 @@ extern "C" int prl_moe_route(const float* logits, int64_t ld, const float* bias,
 
 // Router product, choice and grouping in two launches: x [n, W] and the router matrix [experts, W] in fp32 or bf16.
 // Needs (W + experts) * 4 bytes of shared memory; returns PRL_ERR_INVALID beyond 160 KB (use prl_gemm_any + prl_moe_route).
-extern "C" int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is_f32, const float* bias, int32_t n, int32_t W,
-                              int32_t experts, int32_t top, int32_t softmax_weights, int32_t* sel, float* wsel, int32_t* perm,
-                              int32_t* meta, int32_t* tiles, prl_stream_t st) {
+static int moe_router_impl(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is_f32, const float* bias, int32_t n, int32_t W,
+                           int32_t experts, int32_t outputs, int32_t top, int32_t softmax_weights, const ChoiceRule* rule,
+                           int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta, int32_t* tiles, prl_stream_t st) {
   PRL_CHECK_ARG(x && Wr && sel && wsel && perm && meta && tiles, "prl_moe_router: NULL argument");
-  PRL_CHECK_ARG(n >= 1 && W >= 1 && experts >= 1 && experts <= 32 * kMaxPerLane && top >= 1 && top <= experts,
-                "prl_moe_router: bad shape (experts=%d top=%d; at most %d experts)", experts, top, 32 * kMaxPerLane);
-  const size_t smem = ((size_t)W + experts) * sizeof(float);
+  PRL_CHECK_ARG(n >= 1 && W >= 1 && outputs >= 1 && outputs <= 32 * kMaxPerLane && top >= 1 && top <= outputs,
+                "prl_moe_router: bad shape (outputs=%d top=%d; at most %d outputs)", outputs, top, 32 * kMaxPerLane);
+  const size_t smem = ((size_t)W + outputs + (rule ? outputs + rule->groups : 0)) * sizeof(float);
   PRL_CHECK_ARG(smem <= 160 * 1024, "prl_moe_router: a row of %d channels does not fit in shared memory", W);
   cudaStream_t s = (cudaStream_t)st;
-  static SmemAttr attr[4] = {};
-#define PRL_RT(TX, TW, I)                                                                                              \
+  static SmemAttr attr[8] = {};
+#define PRL_RT(TX, TW, RULED, I)                                                                                       \
   do {                                                                                                                 \
-    if (smem > 48 * 1024) PRL_CUDA(ensure_smem(moe_router_kernel<TX, TW>, (int)smem, attr[I]));                        \
-    PRL_CUDA(launch_pdl((moe_router_kernel<TX, TW>), dim3(n), dim3(256), smem, s, (const TX*)x, (const TW*)Wr, bias, n, W, experts, top, \
-                        softmax_weights, sel, wsel));                                                                  \
+    if (smem > 48 * 1024) PRL_CUDA(ensure_smem(moe_router_kernel<TX, TW, RULED>, (int)smem, attr[I]));                 \
+    PRL_CUDA(launch_pdl((moe_router_kernel<TX, TW, RULED>), dim3(n), dim3(256), smem, s, (const TX*)x, (const TW*)Wr, bias, n, W, \
+                        outputs, top, softmax_weights, rule ? *rule : ChoiceRule{}, sel, wsel));                       \
   } while (0)
-  if (x_is_f32 && w_is_f32) PRL_RT(float, float, 0);
-  else if (x_is_f32) PRL_RT(float, bf16, 1);
-  else if (w_is_f32) PRL_RT(bf16, float, 2);
-  else PRL_RT(bf16, bf16, 3);
+#define PRL_RT2(TX, TW, I)                \
+  do {                                    \
+    if (rule) PRL_RT(TX, TW, true, I);    \
+    else PRL_RT(TX, TW, false, I + 4);    \
+  } while (0)
+  if (x_is_f32 && w_is_f32) PRL_RT2(float, float, 0);
+  else if (x_is_f32) PRL_RT2(float, bf16, 1);
+  else if (w_is_f32) PRL_RT2(bf16, float, 2);
+  else PRL_RT2(bf16, bf16, 3);
+#undef PRL_RT2
 #undef PRL_RT
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, kTile, perm, meta, tiles));
+  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, tile_rows, perm, meta, tiles));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
 
-// Choice among outputs whose logits are already there (columns of a projection buffer), and the grouping of the pairs by expert:
-// `outputs` = experts + identity outputs; see moe_choose_kernel.  tile_rows: 64 for prl_moe_gemm, 256 for prl_moe_gemm_tc.  keep == groups (e.g. 1, 1): every output is open.
-extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
-                              int32_t top, int32_t groups, int32_t keep, int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm,
+extern "C" int prl_moe_router(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is_f32, const float* bias, int32_t n, int32_t W,
+                              int32_t experts, int32_t top, int32_t softmax_weights, int32_t* sel, float* wsel, int32_t* perm,
                               int32_t* meta, int32_t* tiles, prl_stream_t st) {
+  return moe_router_impl(x, x_is_f32, Wr, w_is_f32, bias, n, W, experts, experts, top, softmax_weights, nullptr, kTile, sel, wsel, perm,
+                         meta, tiles, st);
+}
+
+static bool choice_rule_ok(int experts, int outputs, const ChoiceRule& r) {
+  return experts >= 1 && outputs >= experts && outputs <= 1024 && r.groups >= 1 && outputs % r.groups == 0 && r.keep >= 1 &&
+         r.keep <= r.groups && r.top >= 1 && r.top <= outputs / r.groups * r.keep && (r.group_top == 1 || r.group_top == 2);
+}
+
+// prl_moe_router with the scoring, ranking and weighting of prl_moe_choose (router rows = outputs).
+extern "C" int prl_moe_router_choose(const void* x, int32_t x_is_f32, const void* Wr, int32_t w_is_f32, const float* correction, int32_t n,
+                                     int32_t W, int32_t experts, int32_t outputs, int32_t top, int32_t groups, int32_t keep,
+                                     int32_t group_top, int32_t sigmoid, int32_t renorm, float scale, int32_t tile_rows, int32_t* sel,
+                                     float* wsel, int32_t* perm, int32_t* meta, int32_t* tiles, prl_stream_t st) {
+  const ChoiceRule rule{correction, top, groups, keep, group_top, sigmoid, renorm, scale};
+  PRL_CHECK_ARG(choice_rule_ok(experts, outputs, rule) && (tile_rows == kTile || tile_rows == 256),
+                "prl_moe_router_choose: bad shape (experts=%d outputs=%d top=%d groups=%d keep=%d)", experts, outputs, top, groups, keep);
+  return moe_router_impl(x, x_is_f32, Wr, w_is_f32, nullptr, n, W, experts, outputs, top, 0, &rule, tile_rows, sel, wsel, perm, meta,
+                         tiles, st);
+}
+
+// Choice among outputs whose logits are already there (columns of a projection buffer), and the grouping of the pairs by expert:
+// `outputs` = experts + identity outputs; see ChoiceRule.  tile_rows: 64 for prl_moe_gemm, 256 for prl_moe_gemm_tc.  keep == groups (e.g. 1, 1): every output is open.
+extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* correction, int32_t n, int32_t experts, int32_t outputs,
+                              int32_t top, int32_t groups, int32_t keep, int32_t group_top, int32_t sigmoid, int32_t renorm, float scale,
+                              int32_t tile_rows, int32_t* sel, float* wsel, int32_t* perm, int32_t* meta, int32_t* tiles,
+                              prl_stream_t st) {
   PRL_CHECK_ARG(tile_rows == kTile || tile_rows == 256, "prl_moe_choose: row tiles of 64 or 256");
   PRL_CHECK_ARG(logits && sel && wsel && perm && meta && tiles, "prl_moe_choose: NULL argument");
-  PRL_CHECK_ARG(n >= 1 && experts >= 1 && outputs >= experts && outputs <= 1024 && ld >= outputs && groups >= 1 &&
-                outputs % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= outputs / groups * keep,
+  const ChoiceRule rule{correction, top, groups, keep, group_top, sigmoid, renorm, scale};
+  PRL_CHECK_ARG(n >= 1 && ld >= outputs && choice_rule_ok(experts, outputs, rule),
                 "prl_moe_choose: bad shape (experts=%d outputs=%d top=%d groups=%d keep=%d)", experts, outputs, top, groups, keep);
   cudaStream_t s = (cudaStream_t)st;
   PRL_CUDA(launch_pdl(moe_choose_kernel, dim3((n + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32),
-                      (size_t)kChooseWarps * (outputs + groups) * sizeof(float), s, logits, ld, correction, n, outputs, top, groups,
-                      keep, sel, wsel));
+                      (size_t)kChooseWarps * (outputs + groups) * sizeof(float), s, logits, ld, n, outputs, rule, sel, wsel));
   PRL_LAUNCH_CHECK();
   PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, tile_rows, perm, meta, tiles));
   PRL_LAUNCH_CHECK();
@@ -582,12 +655,12 @@ extern "C" int prl_moe_gather(const void* x_bf16, const int32_t* perm, const int
   return PRL_OK;
 }
 
-template <bool RELU2>
+template <int ACT>
 static int moe_gemm_impl(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
                          int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta, const int32_t* tiles,
                          int64_t max_tiles, int64_t N, int64_t K, void* C, int64_t ldc, int32_t c_perm, const float* wsel,
                          prl_stream_t st) {
-  PRL_CHECK_ARG(A && W && perm && meta && tiles && C && (!RELU2 || wsel), "prl_moe_gemm: NULL argument");
+  PRL_CHECK_ARG(A && W && perm && meta && tiles && C && (ACT == kActNone || wsel), "prl_moe_gemm: NULL argument");
   PRL_CHECK_ARG(max_tiles >= 1 && max_tiles <= 65535 && N >= 1 && K >= 1 && lda >= K && ldw >= K && ldc >= N && a_mod >= 0,
                 "prl_moe_gemm: bad shape (tiles=%lld N=%lld K=%lld)", (long long)max_tiles, (long long)N, (long long)K);
   cudaStream_t s = (cudaStream_t)st;
@@ -595,14 +668,14 @@ static int moe_gemm_impl(const void* A, int32_t a_is_f32, int64_t lda, int32_t a
       ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
     dim3 grid_tc((unsigned)((N + kBN - 1) / kBN), (unsigned)max_tiles);
     static SmemAttr attr = {};
-    PRL_CUDA(ensure_smem(moe_gemm_mma_kernel<RELU2>, (int)kMmaSmem, attr));
-    PRL_CUDA(launch_pdl(moe_gemm_mma_kernel<RELU2>, grid_tc, dim3(256), kMmaSmem, s, (const bf16*)A, lda, a_mod, (const bf16*)W,
+    PRL_CUDA(ensure_smem(moe_gemm_mma_kernel<ACT>, (int)kMmaSmem, attr));
+    PRL_CUDA(launch_pdl(moe_gemm_mma_kernel<ACT>, grid_tc, dim3(256), kMmaSmem, s, (const bf16*)A, lda, a_mod, (const bf16*)W,
                         expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm, wsel));
     PRL_LAUNCH_CHECK();
     return PRL_OK;
   }
   dim3 grid((unsigned)((N + kTile - 1) / kTile), (unsigned)max_tiles);
-#define PRL_MG(TA, TW) PRL_CUDA(launch_pdl((moe_gemm_kernel<TA, TW, RELU2>), grid, dim3(256), (size_t)0, s, (const TA*)A, lda, a_mod, (const TW*)W, \
+#define PRL_MG(TA, TW) PRL_CUDA(launch_pdl((moe_gemm_kernel<TA, TW, ACT>), grid, dim3(256), (size_t)0, s, (const TA*)A, lda, a_mod, (const TW*)W, \
                                            expert_stride, ldw, perm, meta, tiles, (int)N, (int)K, C, ldc, c_perm, wsel))
   if (a_is_f32 && w_is_f32) PRL_MG(float, float);
   else if (a_is_f32) PRL_MG(float, bf16);
@@ -617,18 +690,22 @@ extern "C" int prl_moe_gemm(const void* A, int32_t a_is_f32, int64_t lda, int32_
                             int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
                             const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, float* C, int64_t ldc,
                             int32_t c_perm, prl_stream_t st) {
-  return moe_gemm_impl<false>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles, N, K, C, ldc,
+  return moe_gemm_impl<kActNone>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles, N, K, C, ldc,
                               c_perm, nullptr, st);
 }
 
-// First product of squared-ReLU experts: act[s] = relu(A[row of s] W_e^T)^2 * wsel[pair of s], in the operand type of A and in
-// sorted order, i.e. the second product's operand (its weight on the expert's OUTPUT: that product is linear).
-extern "C" int prl_moe_gemm_relu2(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
-                                  int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
-                                  const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, const float* wsel, void* act,
-                                  int64_t ld_act, prl_stream_t st) {
-  return moe_gemm_impl<true>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles, N, K, act,
-                             ld_act, 0, wsel, st);
+// First product of ungated experts: out[s] = act(A[row of s] W_e^T) * wsel[pair of s], in the operand type of A and in sorted
+// order, i.e. the second product's operand (its weight on the expert's OUTPUT: that product is linear).  act 1: relu(z)^2,
+// 2: gelu(z) in its error-function form.
+extern "C" int prl_moe_gemm_act(const void* A, int32_t a_is_f32, int64_t lda, int32_t a_mod, const void* W, int32_t w_is_f32,
+                                int64_t expert_stride, int64_t ldw, const int32_t* perm, const int32_t* meta,
+                                const int32_t* tiles, int64_t max_tiles, int64_t N, int64_t K, int32_t act, const float* wsel,
+                                void* out, int64_t ld_out, prl_stream_t st) {
+  PRL_CHECK_ARG(act == kActRelu2 || act == kActGelu, "prl_moe_gemm_act: unknown activation %d", act);
+  return act == kActRelu2 ? moe_gemm_impl<kActRelu2>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles,
+                                                     N, K, out, ld_out, 0, wsel, st)
+                          : moe_gemm_impl<kActGelu>(A, a_is_f32, lda, a_mod, W, w_is_f32, expert_stride, ldw, perm, meta, tiles, max_tiles,
+                                                    N, K, out, ld_out, 0, wsel, st);
 }
 
 extern "C" int prl_moe_glu(const float* gate_up, int64_t ld, int64_t pairs, int32_t F, const int32_t* perm,

@@ -21,7 +21,11 @@ adds the "one norm" block: mixer and feed-forward of a layer read the same norme
 so a layer is one input projection, one output product over both branches and one closing kernel; softmax attention whose
 keys and values may be another layer's, rotary frequencies scaled in bands, a gated feed-forward with a tanh-form gelu,
 squared-ReLU experts chosen by corrected softmax shares inside the best expert groups, outputs of the router that hand the
-input through, and a gated shared expert.
+input through, and a gated shared expert.  "Modadra" (`.from_modadra`) adds the "pre_norm" block (x <- x + m f(norm(x)) for
+every sublayer, m a constant of the model): windowed attention with plain rotary positions, a constant one in the softmax
+denominator and one gate per head beside the gated delta rule, each normed over the width before the two are averaged;
+ungated gelu experts chosen by corrected sigmoid scores inside the best groups (ranked by their two best) and weighted by
+their share of the chosen scores; tanh-capped logits.
 
 Numerics: the residual stream, every norm, softmax, router-like gate, decay, step size and recurrent state are fp32.
 GEMM operands and the KV cache are bf16, or fp32 when the arena is fp32 (the true-fp32 mode: CUDA-core GEMMs with fp32
@@ -70,6 +74,7 @@ class AttnSpec:
     v_mix: int = 0              # 1: this layer's values are kept for later layers; 2: v <- (1 - l) v + l v_first, l = `vmix`
     v_mix_tensor: bool = False  # the checkpoint has a `vmix` scalar for this layer (used only when v_mix == 2)
     sink: bool = False          # a learned logit per head in the softmax denominator (no key, no value)
+    unit_sink: bool = False     # the same with a logit fixed at zero: one is added to the denominator, nothing is learned
     weights: str = "softmax"    # "sigmoid": weight = sigmoid(score + pb[h]) for every visible key, not normalised
     q_temp: tuple = (0.0, 1.0)  # (coef, every): q times 1 + coef * ln(floor((pos + 1) / every) + 1)
     talking: bool = False       # the heads' weights are mixed by the matrix `talk` [heads, heads] before they meet the values
@@ -164,6 +169,10 @@ class MoeSpec:
     keep_groups: int = 1        # only outputs of the best `keep_groups` of them can be chosen
     correction: bool = False    # a learned offset per output joins the scores for the choice, not for the weights
     shared_gate: bool = False   # the shared expert's output times the sigmoid of one logit per token
+    # ... and to those of the "pre_norm" block (score "sigmoid" with the choice rules above)
+    group_top: int = 1          # a group is ranked by the sum of this many (1 or 2) of its best choice scores
+    renorm: bool = False        # the chosen scores are divided by their sum
+    act: str = "relu2"          # ungated experts: "relu2" | "gelu" (error-function form)
 
     @property
     def outputs(self) -> int:
@@ -218,6 +227,7 @@ class LayerSpec:
                                     # | "attention" | "latent_attention" | "sigmoid_delta" (attention without a softmax ||
                                     #   gated delta rule): the layers normed after the sum ("post_ln")
                                     # | "mlstm" and "attention" are also the mixers of the "one_norm" block
+                                    # | "attn_delta" (softmax attention || gated delta rule): the "pre_norm" block
     weights_of: int                 # index of the layer whose tensors this layer uses (its own index if it has its own)
     gla: GlaSpec | None = None
     attn: AttnSpec | None = None
@@ -248,6 +258,22 @@ class JointRows:
 
 
 @dataclass(frozen=True)
+class AttnDeltaRows:
+    """Columns of the projection buffer of an 'attn_delta' layer:
+    [left q | k | v || right q | k | v | right gate | left gate | step | decay | padding]; everything with a head size comes
+    first, so that head sizes of a multiple of four keep every part on a 16-byte boundary."""
+    k: int
+    v: int
+    right: int      # first convolved channel of the right mixer
+    right_g: int
+    left_g: int
+    b: int
+    a: int
+    end: int
+    total: int      # a multiple of eight
+
+
+@dataclass(frozen=True)
 class HybridConfig:
     vocab_size: int
     width: int
@@ -263,6 +289,9 @@ class HybridConfig:
     pair_embed: tuple | None = None  # (buckets, mul_prev, mul_cur): hashed (previous, current) token table `bigram`
     block: str = "out_norm"         # "post_ln": x <- norm(skip_scale * x + f(x)) for every sublayer, f reads x itself
                                     # "one_norm": x <- x + (mixer(h) + ff(h)), h = norm(x)
+                                    # "pre_norm": x <- x + residual_mult * f(norm(x)) for every sublayer
+    residual_mult: float = 1.0
+    logit_softcap: float = 0.0      # > 0: logits <- softcap * tanh(logits / softcap)
     skip_scale: float = 1.0
     tied_head: bool = False         # logits = embed . x: no separate `head` tensor
 
@@ -542,6 +571,60 @@ class HybridConfig:
         cfg.validate()
         return cfg
 
+    # ---- the "Modadra" reading of config.json ---------------------------------------------------------------------
+    @staticmethod
+    def from_modadra(d: dict, tensor_shapes: dict | None = None) -> "HybridConfig":
+        """config.json of a Modadra checkpoint: pre-normed sublayers with a scaled residual (`residual_mult`), every mixer
+        attention beside the gated delta rule, a routed or no feed-forward.  Whether a router has a correction and an
+        attention its head gates is read off the tensor names when a file is at hand."""
+        shapes = tensor_shapes or {}
+        layers = []
+        for i, L in enumerate(d["layers"]):
+            has = (lambda name: f"l{i}.{name}" in shapes) if shapes else (lambda name: True)
+            if L["type"] != "parallel":
+                raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+            a, r, f, mlp = L["mixer"]["left"], L["mixer"]["right"], L.get("mlp"), None
+            if f is not None:
+                if f.get("kind", "moe") != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {f.get('kind')!r}")
+                q = f["router"]
+                g = q.get("groups") or {}
+                count = int(g.get("count", 1))
+                moe = MoeSpec(int(q["experts"]), int(q["top"]), int(f["expert"]["ff"]), 0.0, score="sigmoid", weight_on="output",
+                              weight_scale=float(q.get("scale", 1.0)), groups=count, keep_groups=int(g.get("keep", count)),
+                              correction=has("mlp.correction"), group_top=2, renorm=True, act="gelu")
+                mlp = MlpSpec(ff=0, limit=0.0, kind="moe", moe=moe)
+            rot = a.get("rot") or {}
+            attn = AttnSpec(int(a["heads"]), int(a.get("kv_heads", a["heads"])), int(a["dim"]), int(a.get("vdim", a["dim"])),
+                            int(rot.get("dims", 0)), float(rot.get("base", 10000.0)), float(a["scale"]),
+                            window=int((a.get("mask") or {}).get("size", 0)), gate=has("mix.left.g"), gate_per_head=True, rot_half=True,
+                            unit_sink=True)
+            gd = GatedDeltaSpec(int(r["heads"]), int(r.get("kv_heads", r["heads"])), int(r["dim"]), int(r.get("vdim", r["dim"])),
+                                int(r["conv"]))
+            layers.append(LayerSpec("attn_delta", i, attn=attn, gdelta=gd, left_scale=0.5, right_scale=0.5, mlp=mlp))
+        cfg = HybridConfig(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), 1.0, tuple(layers), block="pre_norm",
+                           residual_mult=float(d.get("residual_mult", 1.0)), logit_softcap=float(d.get("logit_softcap") or 0.0))
+        cfg.validate()
+        return cfg
+
+    def _validate_pre_norm(self) -> None:
+        if self.logit_softcap < 0:
+            raise ValueError(f"bad logit cap {self.logit_softcap}")
+        for i, L in enumerate(self.layers):
+            if L.kind != "attn_delta":
+                raise ValueError(f"layer run {i}: the mixers of the 'pre_norm' block are attention beside the gated delta rule")
+            a, g = L.attn, L.gdelta
+            if (min(a.heads, a.kv_heads, a.dim, a.vdim) < 1 or a.heads % a.kv_heads or a.rot_dims % 2 or not 0 <= a.rot_dims <= a.dim
+                    or a.dim > 1024 or a.vdim > 512 or a.window < 0):
+                raise ValueError(f"layer run {i}: bad attention geometry {a}")
+            if min(g.heads, g.kv_heads, g.dim, g.vdim) < 1 or g.heads % g.kv_heads or not 1 <= g.conv <= 16 or g.dim > 256:
+                raise ValueError(f"layer run {i}: bad gated-delta geometry {g}")
+            if L.mlp is not None:
+                e = L.mlp.moe
+                if (L.mlp.kind != "moe" or e.experts < 1 or e.ff < 1 or e.outputs > 1024 or e.groups < 1 or e.outputs % e.groups
+                        or not 1 <= e.keep_groups <= e.groups or not 1 <= e.top <= e.outputs // e.groups * e.keep_groups):
+                    raise ValueError(f"layer run {i}: bad router {e}")
+
     def _validate_one_norm(self) -> None:
         for i, L in enumerate(self.layers):
             if L.kind not in ("mlstm", "attention"):
@@ -576,6 +659,8 @@ class HybridConfig:
     def validate(self) -> None:
         if self.block == "one_norm":
             return self._validate_one_norm()
+        if self.block == "pre_norm":
+            return self._validate_pre_norm()
         if self.norm_kind == "tanh":
             if not 1 <= self.streams <= 8 or any(L.kind not in ("latent", "delta") for L in self.layers):
                 raise ValueError("the multi-stream program runs latent-attention and delta-rule layers over 1 to 8 streams")
@@ -660,7 +745,7 @@ class HybridConfig:
             if L.kind in ("latent", "delta"):
                 out += [(name, shape) for name, shape, _ in self._stream_layer_tensors(i, L)]
                 continue
-            if self.block in ("post_ln", "one_norm"):
+            if self.block in ("post_ln", "one_norm", "pre_norm"):
                 out += [(name, shape) for name, shape, _ in self._layer_tensors(i, L)]
                 continue
             if L.kind == "gla":
@@ -840,7 +925,47 @@ class HybridConfig:
         return JointRows(mix, mix, sg, router, (at + 7) // 8 * 8)
 
     def _layer_tensors(self, i: int, L: LayerSpec) -> list:
-        return self._postln_layer_tensors(i, L) if self.block == "post_ln" else self._joint_layer_tensors(i, L)
+        return {"post_ln": self._postln_layer_tensors, "one_norm": self._joint_layer_tensors,
+                "pre_norm": self._prenorm_layer_tensors}[self.block](i, L)
+
+    @staticmethod
+    def attn_delta_rows(L: LayerSpec) -> "AttnDeltaRows":
+        """Row layout of the fused input projection of an 'attn_delta' layer."""
+        a, g = L.attn, L.gdelta
+        k = a.heads * a.dim
+        v = k + a.kv_heads * a.dim
+        right = v + a.kv_heads * a.vdim
+        right_g = right + g.conv_channels
+        left_g = right_g + g.heads * g.vdim
+        b = left_g + (a.heads if a.gate else 0)
+        end = b + 2 * g.heads
+        return AttnDeltaRows(k, v, right, right_g, left_g, b, b + g.heads, end, (end + 7) // 8 * 8)
+
+    def _prenorm_layer_tensors(self, i: int, L: LayerSpec) -> list:
+        """(fused tensor, shape, [(checkpoint tensor or None = padding, rows)] in row order) of a layer of the 'pre_norm'
+        block: all projections of both mixers are ONE fused tensor `mix.in` (see AttnDeltaRows)."""
+        W, p, out = self.width, f"l{i}.", []
+        one = lambda name, shape: out.append((p + name, shape, [(p + name, shape[0])]))
+        a, g, C = L.attn, L.gdelta, self.attn_delta_rows(L)
+        gq, gv = g.kv_heads * g.dim, g.heads * g.vdim
+        parts = [(p + "mix.left.q", C.k), (p + "mix.left.k", C.v - C.k), (p + "mix.left.v", C.right - C.v), (p + "mix.right.q", gq),
+                 (p + "mix.right.k", gq), (p + "mix.right.v", gv), (p + "mix.right.g", gv)]
+        parts += [(p + "mix.left.g", a.heads)] if a.gate else []
+        parts += [(p + "mix.right.b", g.heads), (p + "mix.right.a", g.heads), (None, C.total - C.end)]
+        out.append((p + "mix.in", (C.total, W), parts))
+        one("mix.left.o", (W, a.heads * a.vdim))
+        out.append((p + "mix.right.conv", (g.conv_channels, g.conv),
+                    [(p + "mix.right.q.conv", gq), (p + "mix.right.k.conv", gq), (p + "mix.right.v.conv", gv)]))
+        one("mix.right.A_log", (g.heads,)); one("mix.right.dt_bias", (g.heads,)); one("mix.right.norm", (g.vdim,))
+        one("mix.right.o", (W, gv)); one("mix.left.out", (W,)); one("mix.right.out", (W,)); one("norm1", (W,))
+        if L.mlp is not None:
+            e = L.mlp.moe
+            one("norm2", (W,)); one("mlp.router", (e.outputs, W))
+            if e.correction:
+                one("mlp.correction", (e.outputs,))
+            out.append((p + "mlp.experts.up", (e.experts * e.ff, W), [(f"{p}mlp.e{k}.up", e.ff) for k in range(e.experts)]))
+            out.append((p + "mlp.experts.down", (e.experts * W, e.ff), [(f"{p}mlp.e{k}.down", W) for k in range(e.experts)]))
+        return out
 
     def _joint_layer_tensors(self, i: int, L: LayerSpec) -> list:
         """(fused tensor, shape, [(checkpoint tensor or None = padding, rows)] in row order) of a layer of the 'one_norm'
@@ -906,7 +1031,7 @@ class HybridConfig:
                 for fused, _, parts in self._stream_layer_tensors(i, L):
                     rows(fused, parts)
                 continue
-            if self.block in ("post_ln", "one_norm"):
+            if self.block in ("post_ln", "one_norm", "pre_norm"):
                 for fused, _, parts in self._layer_tensors(i, L):
                     rows(fused, parts)
                 continue
@@ -1086,10 +1211,11 @@ class _Rows:
                 wide_o = max(wide_o, a.heads * a.kv_rank, a.heads * a.vdim)
                 wide_o2 = max(wide_o2, a.heads * a.dim, a.heads * a.vdim)
                 wide_q = max(wide_q, a.heads * (a.kv_rank + a.rot_dim))
-            elif L.kind == "sigmoid_delta":
+            elif L.kind in ("sigmoid_delta", "attn_delta"):
                 a, g = L.attn, L.gdelta
                 nq = a.heads * a.dim
-                wide_p = max(wide_p, nq + a.kv_heads * (a.dim + a.vdim) + g.in_rows)
+                wide_p = max(wide_p, cfg.attn_delta_rows(L).total if L.kind == "attn_delta"
+                             else nq + a.kv_heads * (a.dim + a.vdim) + g.in_rows)
                 wide_q, wide_aux = max(wide_q, nq), max(wide_aux, g.conv_channels)
                 wide_o = max(wide_o, a.heads * a.vdim, g.heads * g.vdim)
                 wide_o2 = max(wide_o2, g.heads * g.vdim)
@@ -1233,7 +1359,7 @@ class HybridEngine(EngineCore):
             self.prev_token = self.states.add("prev_token", (1,), dtype=torch.int32)
         self.rot_mag: dict[int, float] = {}
         for i, L in enumerate(cfg.layers):               # one cache / state per layer RUN, also where weights are shared
-            if L.kind in ("attention", "sigmoid_delta"):
+            if L.kind in ("attention", "sigmoid_delta", "attn_delta"):
                 a = L.attn
                 # head size 128 in bf16 without window, sink or cap: the tcgen05 prompt kernel and the TMA decode kernel
                 self.tc_attn[i] = (cfg.block == "one_norm" and not self.f32 and a.dim == 128 and a.vdim == 128
@@ -1248,7 +1374,7 @@ class HybridEngine(EngineCore):
                     self.v_pool[i] = torch.zeros(self.n_pages, a.kv_heads, PAGE_SIZE, a.vdim, dtype=self.op_dtype, device=d)
                 f, self.rot_mag[i] = rotary_table(a.rot_dims, a.rot_base, a.rot_scaling, a.rot_scaling_kind)
                 self.rot_freq[i] = torch.tensor(f or [0.0], dtype=torch.float64, device=d)
-                if L.kind == "sigmoid_delta":
+                if L.gdelta is not None:
                     g = L.gdelta
                     self.conv_state[i] = self.states.add(f"l{i}.conv", (g.conv_channels, max(g.conv - 1, 1)))
                     n = int(lib.prl_delta_state_floats(g.heads, g.dim, g.vdim))
@@ -1318,6 +1444,9 @@ class HybridEngine(EngineCore):
         conv_ch = max([L.gdelta.conv_channels for L in cfg.layers if L.gdelta is not None], default=0)
         if conv_ch:                                      # the short convolutions of the gated delta rule have no bias
             self.zero_bias = torch.zeros(conv_ch, dtype=torch.float32, device=d)
+        sinks = max([L.attn.heads for L in cfg.layers if L.attn is not None and L.attn.unit_sink], default=0)
+        if sinks:                                        # sink logits fixed at zero
+            self.zero_sink = torch.zeros(sinks, dtype=torch.float32, device=d)
         if cfg.positions == "sinusoid":
             W = cfg.width
             self.pos_freq = torch.tensor([10000.0 ** (-2.0 * k / W) for k in range((W + 1) // 2)], dtype=torch.float64, device=d)
@@ -1372,7 +1501,7 @@ class HybridEngine(EngineCore):
             return [(L.mlstm.heads, L.mlstm.dim, L.mlstm.vdim + 1)]
         if L.kind == "parallel_lin":
             return [(L.lin.heads, L.lin.dim, L.lin.vdim)]
-        if L.kind in ("latent", "delta", "attention", "latent_attention", "sigmoid_delta"):
+        if L.kind in ("latent", "delta", "attention", "latent_attention", "sigmoid_delta", "attn_delta"):
             return []                      # the delta rules have a scan of their own (delta_scan.cu), walked token by token
         return [(L.ssd.heads, L.ssd.state, L.ssd.vdim)]
 
@@ -1410,6 +1539,8 @@ class HybridEngine(EngineCore):
             return self._postln_layers(R, n, ns, max_q, row_pos, seg_pos0, trace)
         if cfg.block == "one_norm":
             return self._joint_layers(R, n, ns, max_q, row_pos, seg_pos0, trace, decode)
+        if cfg.block == "pre_norm":
+            return self._prenorm_layers(R, n, ns, max_q, row_pos, seg_pos0, trace)
         W, eps, vec = cfg.width, cfg.eps, self.vec
         seg_start, seg_len, seg_slot = R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr()
         P, x, xa = R.P.data_ptr(), R.x.data_ptr(), R.xa.data_ptr()
@@ -1535,14 +1666,14 @@ class HybridEngine(EngineCore):
     def _pre_gain(self, i: int):
         """Gain of the norm in front of run i's mixer (None: the mixer reads x as it is)."""
         L = self.cfg.layers[i]
-        return self.vec[f"l{L.weights_of}.norm1"] if L.sandwich else None
+        return self.vec[f"l{L.weights_of}.norm1"] if L.sandwich or self.cfg.block == "pre_norm" else None
 
     def _next_gain(self, i: int, after_mixer: bool):
         """Gain of the input norm of whatever reads x after this sublayer of run i: the run's feed-forward, the next
         run's mixer, or nothing (the opening of a pass and the model's last norm read x itself)."""
         L = self.cfg.layers[i]
         if after_mixer and L.mlp is not None:
-            return self.vec[f"l{L.weights_of}.norm2"] if L.sandwich else None
+            return self.vec[f"l{L.weights_of}.norm2"] if L.sandwich or self.cfg.block == "pre_norm" else None
         if i + 1 < len(self.cfg.layers) and self.cfg.layers[i + 1].opens_pass is None:
             return self._pre_gain(i + 1)
         return None
@@ -1810,28 +1941,38 @@ class HybridEngine(EngineCore):
         _lib.check(lib.prl_gemm_tn_dual(src1.data_ptr(), p1, K1, src2.data_ptr(), p2, K2, n, N, k, out.data_ptr(), st))
         return k
 
-    def _choose_and_run_experts(self, R, n, w, e, ld, off_router) -> torch.Tensor:
-        """Squared-ReLU experts chosen from the router's columns of R.P; returns [top][n][W] fp32 (R.moe_out), in which the
-        slices of choices that hand the input through (R.sel >= experts) are not written."""
+    def _choose_and_run_experts(self, R, n, w, e, ld=0, off_router=None) -> torch.Tensor:
+        """Ungated experts (squared ReLU or gelu) chosen from the router's columns of R.P, or (off_router None) by the router
+        `mlp.router` of R.xa; returns [top][n][W] fp32 (R.moe_out), in which the slices of choices that hand the input through
+        (R.sel >= experts) are not written."""
         lib, st, W, f32 = self.lib, self._st, self.cfg.width, int(self.f32)
         corr = self.vec[w + "mlp.correction"].data_ptr() if e.correction else None
         pairs, up, down = n * e.top, self.arena.ptr(w + "mlp.experts.up"), self.arena.ptr(w + "mlp.experts.down")
         # enough rows per expert for 256-row tiles: the tcgen05 grouped GEMM over gathered rows
         tc = (pairs >= self.moe_tc_rows * e.experts and n > 128 and W % 8 == 0 and e.ff % 8 == 0 and min(W, e.ff) >= 64
               and not (self.f32 or self.force_plain_gemm))
-        _lib.check(lib.prl_moe_choose(R.P.data_ptr() + 4 * off_router, ld, corr, n, e.experts, e.outputs, e.top, e.groups,
-                                      e.keep_groups, 256 if tc else 64, R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(),
-                                      R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), st))
+        rule = (e.top, e.groups, e.keep_groups, e.group_top, int(e.score == "sigmoid"), int(e.renorm), e.weight_scale, 256 if tc else 64,
+                R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(), R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), st)
+        if off_router is not None:
+            _lib.check(lib.prl_moe_choose(R.P.data_ptr() + 4 * off_router, ld, corr, n, e.experts, e.outputs, *rule))
+        elif (W + 3 * e.outputs) * 4 <= 160 * 1024 and not self.unfused_router:
+            _lib.check(lib.prl_moe_router_choose(R.xa.data_ptr(), f32, self.arena.ptr(w + "mlp.router"), f32, corr, n, W, e.experts,
+                                                 e.outputs, *rule))
+        else:
+            _lib.check(lib.prl_gemm_any(R.xa.data_ptr(), f32, W, self.arena.ptr(w + "mlp.router"), f32, W, n, e.outputs, W,
+                                        R.router.data_ptr(), e.outputs, st))
+            _lib.check(lib.prl_moe_choose(R.router.data_ptr(), e.outputs, corr, n, e.experts, e.outputs, *rule))
+        unit = {"relu2": 1, "gelu": 2}[e.act]
         table = (R.perm.data_ptr(), R.moe_meta.data_ptr(), R.moe_tiles.data_ptr())
         act, out = R.moe_act.data_ptr(), R.moe_out.data_ptr()
         if tc:      # the gathered rows live where the second product's output goes: they are consumed before it is written
             _lib.check(lib.prl_moe_gather(R.xa.data_ptr(), *table[:2], n, pairs, W, out, st))
-            _lib.check(lib.prl_moe_gemm_tc(out, pairs, up, e.experts, e.ff, W, *table, R.wsel.data_ptr(), act, e.ff, st))
-            _lib.check(lib.prl_moe_gemm_tc(act, pairs, down, e.experts, W, e.ff, *table, None, out, W, st))
+            _lib.check(lib.prl_moe_gemm_tc(out, pairs, up, e.experts, e.ff, W, *table, R.wsel.data_ptr(), unit, act, e.ff, st))
+            _lib.check(lib.prl_moe_gemm_tc(act, pairs, down, e.experts, W, e.ff, *table, None, 0, out, W, st))
             return R.moe_out
         table += (int(lib.prl_moe_max_tiles(pairs, e.experts)),)
-        _lib.check(lib.prl_moe_gemm_relu2(R.xa.data_ptr(), f32, W, n, up, f32, e.ff * W, W, *table, e.ff, W, R.wsel.data_ptr(), act,
-                                          e.ff, st))
+        _lib.check(lib.prl_moe_gemm_act(R.xa.data_ptr(), f32, W, n, up, f32, e.ff * W, W, *table, e.ff, W, unit, R.wsel.data_ptr(), act,
+                                        e.ff, st))
         _lib.check(lib.prl_moe_gemm(act, f32, e.ff, 0, down, f32, W * e.ff, e.ff, *table, W, e.ff, out, W, 1, st))
         return R.moe_out
 
@@ -1916,23 +2057,75 @@ class HybridEngine(EngineCore):
                                         vec[w + "mix.left.talk"].data_ptr() if a.talking else None, 1, R.ya.data_ptr(), n,
                                         int(not self.force_plain_attn), self.attn_ws.data_ptr(), self.attn_ws.numel(), st))
         k0 = self._mm(R.ya, no, w + "mix.left.o", W, R.y0, n, split=True)
-        # -- right: convolutions + SiLU over [q | k | v], then the scan
-        gq, gv, ch = g.kv_heads * g.dim, g.heads * g.vdim, g.conv_channels
-        _lib.check(lib.prl_conv_silu(P, ld, left, n, ch, g.conv, vec[w + "mix.right.conv"].data_ptr(), self.zero_bias.data_ptr(),
-                                     R.row_slot.data_ptr(), R.row_back.data_ptr(), self.conv_state[i].data_ptr(),
-                                     R.aux.data_ptr(), st))
-        _lib.check(lib.prl_conv_state_update(P, ld, left, ch, g.conv, seg_start, seg_len, seg_slot, ns,
-                                             self.conv_state[i].data_ptr(), st))
-        _lib.check(lib.prl_gated_delta_scan(R.aux.data_ptr(), ch, 0, gq, 2 * gq, P, ld, left + ch, left + ch + g.heads,
-                                            vec[w + "mix.right.A_log"].data_ptr(), vec[w + "mix.right.dt_bias"].data_ptr(),
-                                            g.unit_eps, g.heads, g.kv_heads, g.dim, g.vdim, n, R.dprep.data_ptr(), seg_start,
-                                            seg_len, seg_slot, ns, max_q, self.delta_state[i].data_ptr(), R.o.data_ptr(), gv,
-                                            st))
-        _lib.check(lib.prl_gate_norm(R.o.data_ptr(), 1, gv, P + 4 * (left + ch + 2 * g.heads), ld,
-                                     vec[w + "mix.right.norm"].data_ptr(), g.vdim, g.vdim, n, gv, 0, 0, 1, self.cfg.eps,
-                                     R.yb.data_ptr(), f32, st))
+        # -- right
+        gv, ch = g.heads * g.vdim, g.conv_channels
+        self._gated_delta_cell(R, n, i, g, w + "mix.right.", segs, max_q, P, ld, left, left + ch, left + ch + g.heads,
+                               left + ch + 2 * g.heads)
         k1 = self._mm(R.yb, gv, w + "mix.right.o", W, R.y1, n, split=True)
         return k0, k1
+
+    # ---- the 'pre_norm' block: x <- x + m f(norm(x)) for every sublayer ---------------------------------------------------
+    def _prenorm_layers(self, R, n, ns, max_q, row_pos, seg_pos0, trace=None) -> None:
+        """Layer program of the 'pre_norm' block.  R.xa always holds the next sublayer's normed input: every closing kernel
+        norms the branches, adds them to the residual and leaves the next norm's output."""
+        cfg, vec, m = self.cfg, self.vec, self.cfg.residual_mult
+        segs = (R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr(), ns)
+        if cfg.layers:
+            _lib.check(self.lib.prl_rmsnorm_rows(R.x.data_ptr(), None, self._pre_gain(0).data_ptr(), cfg.eps, n, cfg.width,
+                                                 R.xa.data_ptr(), int(self.f32), self._st))
+        for i, L in enumerate(cfg.layers):
+            w = f"l{L.weights_of}."
+            k0, k1 = self._attn_delta_mixer(R, n, i, L, w, segs, max_q, row_pos, seg_pos0)
+            self._close(R, n, R.y0, k0, gain0=vec[w + "mix.left.out"], s0=L.left_scale * m, y1=R.y1, k1=k1,
+                        gain1=vec[w + "mix.right.out"], s1=L.right_scale * m, next_gain=self._next_gain(i, True))
+            if L.mlp is not None:
+                y = self._choose_and_run_experts(R, n, w, L.mlp.moe)
+                self._close(R, n, y, L.mlp.moe.top, s0=m, next_gain=self._next_gain(i, False))
+            if trace is not None:
+                trace.append(R.x[:n * cfg.width].view(n, cfg.width).clone())
+
+    def _attn_delta_mixer(self, R, n, i, L, w, segs, max_q, row_pos, seg_pos0):
+        """Windowed softmax attention (one added to the denominator, one gate per head) beside the gated delta rule, both from
+        ONE projection (AttnDeltaRows).  Returns the split-K slice counts of the two output projections (R.y0, R.y1)."""
+        a, g, lib, st, vec, f32, W = L.attn, L.gdelta, self.lib, self._st, self.vec, int(self.f32), self.cfg.width
+        seg_start, seg_len, seg_slot, ns = segs
+        C, P = self.cfg.attn_delta_rows(L), R.P.data_ptr()
+        ld, no = C.total, a.heads * a.vdim
+        self._mm(R.xa, W, w + "mix.in", ld, R.P, n)
+        # -- left
+        bt = (self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE)
+        kv = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr())
+        _lib.check(lib.prl_attn_front(P, ld, 0, C.k, C.v, n, a.heads, a.kv_heads, a.dim, a.vdim, None, None, None, 0, None, None, a.dim,
+                                      self.cfg.eps, a.rot_dims, self.rot_freq[i].data_ptr(), self.rot_mag[i], 0, 0, None, None,
+                                      row_pos.data_ptr(), R.row_slot.data_ptr(), *bt, R.q.data_ptr(), *kv, f32, st))
+        sink = self.zero_sink.data_ptr() if a.unit_sink else None
+        _lib.check(lib.prl_attn_any_sink(R.q.data_ptr(), *kv, a.vdim, f32, *bt, seg_start, seg_len, seg_pos0.data_ptr(), seg_slot, ns,
+                                         max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, 0, a.softcap, sink,
+                                         0 if a.gate else 1, R.o.data_ptr() if a.gate else R.ya.data_ptr(), st))
+        if a.gate:
+            _lib.check(lib.prl_gate_heads(R.o.data_ptr(), 1, no, P + 4 * C.left_g, ld, n, a.heads, a.vdim, R.ya.data_ptr(), f32, st))
+        k0 = self._mm(R.ya, no, w + "mix.left.o", W, R.y0, n, split=True)
+        # -- right
+        self._gated_delta_cell(R, n, i, g, w + "mix.right.", segs, max_q, P, ld, C.right, C.b, C.a, C.right_g)
+        k1 = self._mm(R.yb, g.heads * g.vdim, w + "mix.right.o", W, R.y1, n, split=True)
+        return k0, k1
+
+    def _gated_delta_cell(self, R, n, i, g, p, segs, max_q, P, ld, off, off_b, off_a, off_g) -> None:
+        """From the projections in P (rows ld apart: q | k | v at `off`, step, decay and gate columns) to the cell's normed and
+        gated output R.yb."""
+        lib, st, vec, f32 = self.lib, self._st, self.vec, int(self.f32)
+        seg_start, seg_len, seg_slot, ns = segs
+        gq, gv, ch = g.kv_heads * g.dim, g.heads * g.vdim, g.conv_channels
+        conv = self.conv_state[i].data_ptr()
+        _lib.check(lib.prl_conv_silu(P, ld, off, n, ch, g.conv, vec[p + "conv"].data_ptr(), self.zero_bias.data_ptr(),
+                                     R.row_slot.data_ptr(), R.row_back.data_ptr(), conv, R.aux.data_ptr(), st))
+        _lib.check(lib.prl_conv_state_update(P, ld, off, ch, g.conv, seg_start, seg_len, seg_slot, ns, conv, st))
+        _lib.check(lib.prl_gated_delta_scan(R.aux.data_ptr(), ch, 0, gq, 2 * gq, P, ld, off_b, off_a, vec[p + "A_log"].data_ptr(),
+                                            vec[p + "dt_bias"].data_ptr(), g.unit_eps, g.heads, g.kv_heads, g.dim, g.vdim, n,
+                                            R.dprep.data_ptr(), seg_start, seg_len, seg_slot, ns, max_q,
+                                            self.delta_state[i].data_ptr(), R.o.data_ptr(), gv, st))
+        _lib.check(lib.prl_gate_norm(R.o.data_ptr(), 1, gv, P + 4 * off_g, ld, vec[p + "norm"].data_ptr(), g.vdim, g.vdim, n, gv, 0, 0, 1,
+                                     self.cfg.eps, R.yb.data_ptr(), f32, st))
 
     # ---- the multi-stream program: latent attention and delta-rule layers ------------------------------------------------
     def _stream_weights(self, i: int, q: str):
@@ -2123,6 +2316,10 @@ class HybridEngine(EngineCore):
             _lib.check(lib.prl_rmsnorm_rows(R.x.data_ptr(), rows, self.vec["final.norm"].data_ptr(), cfg.eps, n_out, cfg.width,
                                             R.xa.data_ptr(), int(self.f32), st))
 
+    def _cap_logits(self, logits, n) -> None:
+        if self.cfg.logit_softcap > 0:
+            _lib.check(self.lib.prl_soft_cap(logits.data_ptr(), n * self.cfg.vocab_size, self.cfg.logit_softcap, self._st))
+
     # ---- one token for every slot (captured into the engine's CUDA graph) ---------------------------------------------
     def _step_kernels(self) -> None:
         cfg, lib, R, B = self.cfg, self.lib, self._dec, self.B
@@ -2132,6 +2329,7 @@ class HybridEngine(EngineCore):
         self._layers(R, B, B, 1, self.positions, self.positions, decode=True)
         self._final_norm(R, None, B)
         self._mm(R.xa, cfg.width, self.head_name, cfg.vocab_size, self.logits, B)
+        self._cap_logits(self.logits, B)
 
     # ---- a packed batch of prompt portions (prefill chunks, token streams) --------------------------------------------
     def _forward_rows(self, segs, want_rows, trace=None):
@@ -2182,4 +2380,5 @@ class HybridEngine(EngineCore):
         self._final_norm(R, R.want.data_ptr(), nw)
         out = torch.empty(nw, cfg.vocab_size, dtype=torch.float32, device=self.dev)
         self._mm(R.xa, cfg.width, self.head_name, cfg.vocab_size, out, nw)
+        self._cap_logits(out, nw)
         return out

@@ -123,6 +123,11 @@ def _futetar_config(config: dict, shapes: dict):
     return HybridConfig.from_futetar(config, shapes)
 
 
+def _modadra_config(config: dict, shapes: dict):
+    from .hybrid import HybridConfig
+    return HybridConfig.from_modadra(config, shapes)
+
+
 def _hybrid_engine():
     from .hybrid import HybridEngine
     return HybridEngine
@@ -134,6 +139,7 @@ register(Family("Belelorn", _belelorn_config, _hybrid_engine, (torch.bfloat16, t
 register(Family("Pametar", _pametar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 register(Family("Kolotar", _kolotar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 register(Family("Futetar", _futetar_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
+register(Family("Modadra", _modadra_config, _hybrid_engine, (torch.bfloat16, torch.float32)))
 
 
 def parse_dtype(name: str) -> torch.dtype:

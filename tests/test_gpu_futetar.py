@@ -290,7 +290,7 @@ def test_choice_kernel_against_the_oracle(cuda_device, n):
         wsel, meta = torch.zeros(top, n, device=cuda_device), torch.zeros(4, **i32)
         tiles = torch.zeros(3 * int(lib.prl_moe_max_tiles(top * n, experts)), **i32)
         zd, cd = z.to(cuda_device), corr.to(cuda_device)
-        _lib.check(lib.prl_moe_choose(zd.data_ptr(), E + 3, cd.data_ptr(), n, experts, E, top, groups, keep, 64, sel.data_ptr(), wsel.data_ptr(),
+        _lib.check(lib.prl_moe_choose(zd.data_ptr(), E + 3, cd.data_ptr(), n, experts, E, top, groups, keep, 1, 0, 0, 1.0, 64, sel.data_ptr(), wsel.data_ptr(),
                                       perm.data_ptr(), meta.data_ptr(), tiles.data_ptr(), _lib.stream_ptr()))
         torch.cuda.synchronize()
         score = torch.softmax(z[:, :E].double(), -1)
@@ -414,12 +414,12 @@ def test_grouped_gemm_of_many_rows(cuda_device, n, W, ff, experts, identity, top
     wsel, tiles = torch.zeros(top, n, device=cuda_device), torch.zeros(3 * int(lib.prl_moe_max_tiles(top * n, experts)), **i32)
     st = _lib.stream_ptr()
     table = (perm.data_ptr(), meta.data_ptr(), tiles.data_ptr())
-    _lib.check(lib.prl_moe_choose(z.data_ptr(), E, None, n, experts, E, top, 1, 1, 256, sel.data_ptr(), wsel.data_ptr(), *table, st))
+    _lib.check(lib.prl_moe_choose(z.data_ptr(), E, None, n, experts, E, top, 1, 1, 1, 0, 0, 1.0, 256, sel.data_ptr(), wsel.data_ptr(), *table, st))
     xs, act = torch.zeros(top * n, W, dtype=torch.bfloat16, device=cuda_device), torch.zeros(top * n, ff, dtype=torch.bfloat16, device=cuda_device)
     out = torch.full((top * n, W), float("nan"), device=cuda_device)
     _lib.check(lib.prl_moe_gather(x.data_ptr(), *table[:2], n, top * n, W, xs.data_ptr(), st))
-    _lib.check(lib.prl_moe_gemm_tc(xs.data_ptr(), top * n, up.data_ptr(), experts, ff, W, *table, wsel.data_ptr(), act.data_ptr(), ff, st))
-    _lib.check(lib.prl_moe_gemm_tc(act.data_ptr(), top * n, down.data_ptr(), experts, W, ff, *table, None, out.data_ptr(), W, st))
+    _lib.check(lib.prl_moe_gemm_tc(xs.data_ptr(), top * n, up.data_ptr(), experts, ff, W, *table, wsel.data_ptr(), 1, act.data_ptr(), ff, st))
+    _lib.check(lib.prl_moe_gemm_tc(act.data_ptr(), top * n, down.data_ptr(), experts, W, ff, *table, None, 0, out.data_ptr(), W, st))
     torch.cuda.synchronize()
     assert int(meta[1]) == int((sel < experts).sum())
     for k in range(top):
