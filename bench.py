@@ -57,7 +57,7 @@ def parse():
     ap.add_argument("--no-rollout", action="store_true", help="N = 1: skip the full-rollout run through the plugin API")
     ap.add_argument("--rollout-tokens", type=int, default=8192, help="max_tokens of the full-rollout component")
     ap.add_argument("--splits", default="", help="learner counts of the split runs, e.g. '2,4' (default: by N)")
-    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "hybrid", "belelorn", "pametar", "kolotar", "futetar"],
+    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "hybrid", "belelorn", "pametar", "kolotar", "futetar", "modadra"],
                     help="hybrid: prefill / decode throughput of the hybrid decoder family (GLA, attention + state-space "
                          "layers) beside the Qwen2 engine at equal sizes, and its kernels against their rooflines "
                          "(tools/hybrid_bench.py); belelorn: the same for the Belelorn design (mLSTM, windowed attention "
@@ -66,7 +66,8 @@ def parse():
                          "the Kolotar design (windowed attention with a sink, latent attention, attention without a softmax "
                          "beside the gated delta rule, norms after the sum) beside Pametar and Qwen2; futetar: the Futetar design "
                          "(mixer and feed-forward behind one norm, memory cells, attention over shared caches, grouped routing) "
-                         "beside Belelorn and Qwen2; "
+                         "beside Belelorn and Qwen2; modadra: the Modadra design (windowed attention beside the gated delta rule in "
+                         "every layer, gelu experts) beside Kolotar and Qwen2; "
                          "the default workload and its JSON line are unchanged")
     ap.add_argument("--sizes", default="w2048,w4096", help="--arch hybrid: model sizes to compare")
     return ap.parse_args()
@@ -623,9 +624,10 @@ def run_hybrid(args):
     sampler = ClockSampler(0)
     sampler.start()
     sizes = args.sizes.split(",")
-    which = args.arch if args.arch in ("belelorn", "pametar", "kolotar", "futetar") else "hybrid"
+    which = args.arch if args.arch in ("belelorn", "pametar", "kolotar", "futetar", "modadra") else "hybrid"
     runner = {"belelorn": hybrid_bench.run_belelorn, "pametar": hybrid_bench.run_pametar,
-              "kolotar": hybrid_bench.run_kolotar, "futetar": hybrid_bench.run_futetar}.get(which, hybrid_bench.run)
+              "kolotar": hybrid_bench.run_kolotar, "futetar": hybrid_bench.run_futetar,
+              "modadra": hybrid_bench.run_modadra}.get(which, hybrid_bench.run)
     res = runner(sizes, prompt=4096, context=2048, batch=32, steps=args.steps, warm=max(3, args.warmup))
     clocks = sampler.stop()
     first = res[sizes[0]][which]
@@ -639,7 +641,7 @@ def run_hybrid(args):
 
 if __name__ == "__main__":
     a = parse()
-    if a.arch in ("hybrid", "belelorn", "pametar", "kolotar", "futetar"):
+    if a.arch in ("hybrid", "belelorn", "pametar", "kolotar", "futetar", "modadra"):
         run_hybrid(a)
     elif a.impl == "reference":
         run_reference(a)

@@ -902,6 +902,25 @@ int prl_gated_delta_scan(const float* C, int64_t ldc, int32_t off_q, int32_t off
                          int32_t kh, int32_t dk, int32_t dv, int32_t n_rows, float* scratch, const int32_t* seg_start,
                          const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg, int32_t max_len, float* state,
                          float* out, int64_t ld_out, prl_stream_t stream);
+/* the whole cell (csrc/gated_delta.cu): convolution + SiLU of q | k | v at column `off` of P with its carried inputs, unit
+ * vectors, decay and step, the recurrence, per-head RMS norm with gain [dv], SiLU gate (column off_g), out [row][heads * dv].
+ * _step: segments of one token (or idle).  _split: pieces of up to 64 tokens side by side (tables as for prl_gla_scan_split);
+ * C [n_rows][2 kh dk + heads dv], scratch [n_rows][prl_gated_delta_split_floats], S0 [n_sub][heads][dk][dv], D [n_rows][heads
+ * dv], all fp32; dv > 128: the raw read-out is left in D instead of `out` */
+int32_t prl_gated_delta_step_fits(int32_t heads, int32_t kh, int32_t dk, int32_t dv, int32_t taps);
+int prl_gated_delta_step(const float* P, int64_t ldp, int32_t off, int32_t off_b, int32_t off_a, int32_t off_g,
+                         const float* conv_w, int32_t taps, const float* A_log, const float* dt_bias, float unit_eps,
+                         const float* gain, float eps, int32_t heads, int32_t kh, int32_t dk, int32_t dv,
+                         const int32_t* seg_start, const int32_t* seg_len, const int32_t* seg_slot, int32_t n_seg,
+                         float* conv_state, float* state, void* out, int32_t f32, prl_stream_t stream);
+int64_t prl_gated_delta_split_floats(int32_t heads, int32_t dk);
+int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, int32_t off_b, int32_t off_a, int32_t off_g,
+                          const float* conv_w, int32_t taps, const float* A_log, const float* dt_bias, float unit_eps,
+                          const float* gain, float eps, int32_t heads, int32_t kh, int32_t dk, int32_t dv, int32_t n_rows,
+                          const int32_t* row_slot, const int32_t* row_back, const int32_t* seg_start, const int32_t* seg_len,
+                          const int32_t* seg_slot, int32_t n_seg, const int32_t* seg_sub0, const int32_t* seg_nsub,
+                          const int32_t* sub_start, const int32_t* sub_len, int32_t n_sub, float* C, float* scratch, float* S0,
+                          float* D, float* conv_state, float* state, void* out, int32_t f32, prl_stream_t stream);
 
 #ifdef __cplusplus
 }

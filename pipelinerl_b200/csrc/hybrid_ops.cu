@@ -506,6 +506,106 @@ __global__ void joint_close_kernel(const float* __restrict__ y0, int ns0, int64_
   }
 }
 
+// sublayer_close_kernel for rows of a multiple of four channels: a thread keeps NC groups of four channels of the row (and of
+// the second branch) in registers from the sums to the normed store.
+template <typename T, int NC>
+__global__ void sublayer_close_vec_kernel(const float* __restrict__ y0, int64_t ld0, int ns0, int64_t stride0,
+                                          const float* __restrict__ gain0, float s0, const float* __restrict__ y1, int64_t ld1,
+                                          int ns1, int64_t stride1, const float* __restrict__ gain1, float s1,
+                                          const float* __restrict__ post_gain, const float* __restrict__ bias, int add,
+                                          const float* __restrict__ next_gain, float eps, int W, float* __restrict__ x,
+                                          T* __restrict__ xa) {
+  pdl_wait();
+  __shared__ float red[32];
+  const int64_t r = blockIdx.x, at = r * W;
+  const int n4 = W / 4;
+  auto sumsq = [](const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; };
+  auto scaled = [](const float4& a, float f, const float* g) {       // a * f * g (g NULL: a * f)
+    if (!g) return make_float4(a.x * f, a.y * f, a.z * f, a.w * f);
+    const float4 w = ld4(g);
+    return make_float4(a.x * f * w.x, a.y * f * w.y, a.z * f * w.z, a.w * f * w.w);
+  };
+  float4 v[NC], xr[NC];
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    v[u] = xr[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c < n4 && add) xr[u] = ld4(x + at + 4 * c);
+  }
+#pragma unroll 4
+  for (int k = 0; k < ns0; ++k)
+#pragma unroll
+    for (int u = 0; u < NC; ++u) {
+      const int c = threadIdx.x + u * blockDim.x;
+      if (c < n4) add4(v[u], ld4(y0 + k * stride0 + r * ld0 + 4 * c));
+    }
+  float f0 = s0;
+  if (gain0) {
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NC; ++u) ss += sumsq(v[u]);
+    f0 = s0 / sqrtf(block_sum(ss, red) / (float)W + eps);
+  }
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c < n4) v[u] = scaled(v[u], f0, gain0 ? gain0 + 4 * c : nullptr);
+  }
+  if (y1) {
+    float4 b[NC];
+#pragma unroll
+    for (int u = 0; u < NC; ++u) b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int k = 0; k < ns1; ++k)
+#pragma unroll
+      for (int u = 0; u < NC; ++u) {
+        const int c = threadIdx.x + u * blockDim.x;
+        if (c < n4) add4(b[u], ld4(y1 + k * stride1 + r * ld1 + 4 * c));
+      }
+    float f1 = s1;
+    if (gain1) {
+      float ss = 0.f;
+#pragma unroll
+      for (int u = 0; u < NC; ++u) ss += sumsq(b[u]);
+      f1 = s1 / sqrtf(block_sum(ss, red) / (float)W + eps);
+    }
+#pragma unroll
+    for (int u = 0; u < NC; ++u) {
+      const int c = threadIdx.x + u * blockDim.x;
+      if (c < n4) add4(v[u], scaled(b[u], f1, gain1 ? gain1 + 4 * c : nullptr));
+    }
+  }
+  if (post_gain) {
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NC; ++u) ss += sumsq(v[u]);
+    const float fp = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+    for (int u = 0; u < NC; ++u) {
+      const int c = threadIdx.x + u * blockDim.x;
+      if (c < n4) v[u] = scaled(v[u], fp, post_gain + 4 * c);
+    }
+  }
+  float sx = 0.f;
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c < n4) {
+      if (bias) add4(v[u], ld4(bias + 4 * c));
+      add4(v[u], xr[u]);
+      st4(x + at + 4 * c, v[u]);
+      sx += sumsq(v[u]);
+    }
+  }
+  float fn = 1.f;
+  if (next_gain) fn = 1.f / sqrtf(block_sum(sx, red) / (float)W + eps);
+#pragma unroll
+  for (int u = 0; u < NC; ++u) {
+    const int c = threadIdx.x + u * blockDim.x;
+    if (c < n4) st4(xa + at + 4 * c, next_gain ? scaled(v[u], fn, next_gain + 4 * c) : v[u]);
+  }
+}
+
 // Attention front end with PER-HEAD unit norms: q and k get their biases (NULL: none), every head of q and of k is
 // divided by its own root mean square over `dim` and multiplied by a gain (NULL: none; indexed head * dim + channel);
 // q goes to the query buffer, k into the paged cache.  The value written beside it is either the key as projected
@@ -1106,6 +1206,21 @@ extern "C" int prl_sublayer_close(const float* y0, int64_t ld0, int32_t n_split0
                                   const float* y1, int64_t ld1, int32_t n_split1, const float* gain1, float s1,
                                   const float* post_gain, const float* bias, int32_t add, const float* next_gain, float eps,
                                   int32_t n, int32_t W, float* x, void* xa, int32_t f32, prl_stream_t st) {
+  const uintptr_t bits = (uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)x | (uintptr_t)xa | (uintptr_t)next_gain | (uintptr_t)gain0 |
+                         (uintptr_t)gain1 | (uintptr_t)post_gain | (uintptr_t)bias;
+  if (y0 && x && xa && n >= 1 && W >= 4 && W % 4 == 0 && W <= 16384 && ld0 >= W && ld0 % 4 == 0 && n_split0 >= 1 &&
+      (!y1 || (ld1 >= W && ld1 % 4 == 0 && n_split1 >= 1)) && (bits & 15) == 0) {
+    const int n4 = W / 4, nc = n > 256 ? (n4 <= 256 ? 1 : n4 <= 1024 ? 2 : 4) : (n4 <= 1024 ? 1 : 4);
+    const int th = ((n4 + nc - 1) / nc + 31) / 32 * 32;
+    const int64_t st0 = (int64_t)n * ld0, st1 = (int64_t)n * ld1;
+#define PRL_SC(T, NC) PRL_CUDA(launch_pdl((sublayer_close_vec_kernel<T, NC>), dim3(n), dim3(th), (size_t)0, (cudaStream_t)st, y0, ld0, n_split0, st0, gain0, s0, \
+                                          y1, ld1, n_split1, st1, gain1, s1, post_gain, bias, add, next_gain, eps, W, x, (T*)xa))
+    if (f32) { if (nc == 1) PRL_SC(float, 1); else if (nc == 2) PRL_SC(float, 2); else PRL_SC(float, 4); }
+    else { if (nc == 1) PRL_SC(bf16, 1); else if (nc == 2) PRL_SC(bf16, 2); else PRL_SC(bf16, 4); }
+#undef PRL_SC
+    PRL_LAUNCH_CHECK();
+    return PRL_OK;
+  }
   return sublayer_close_impl(y0, ld0, n_split0, gain0, s0, y1, ld1, n_split1, gain1, s1, post_gain, bias, add, next_gain, eps, n,
                              W, nullptr, nullptr, 0, x, xa, f32, st);
 }

@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const flo
 }
 
 // Router and choice in one kernel: logits[e] = x . Wr[e] in fp32 (block per row, the row staged in shared memory, warps
-// take experts in turn, a lane sums every 32nd channel, then the warp's shuffle tree: a fixed order), then the top-k
+// take experts in turn, a lane sums every 32nd group of channels, then the warp's shuffle tree: a fixed order), then the top-k
 // pass of moe_route_kernel over the logits in shared memory (RULED: choose_row instead, with scratch behind the logits).
 template <typename TX, typename TW, bool RULED>
 __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ Wr,
@@ -189,17 +189,33 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ 
                                                          int softmax_weights, ChoiceRule rule, int32_t* __restrict__ sel,
                                                          float* __restrict__ wsel) {
   pdl_wait();
-  extern __shared__ float rsm[];       // [W] the row | [E] logits | RULED: [E] choice scores | [groups] group scores
+  extern __shared__ __align__(16) float rsm[];       // [W] the row | [E] logits | RULED: [E] choice scores | [groups] group scores
   float* xs = rsm;
   float* z = rsm + W;
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   for (int c = threadIdx.x; c < W; c += blockDim.x) xs[c] = to_f32(x[(int64_t)t * W + c]);
   __syncthreads();
+  constexpr int V = 16 / sizeof(TW);              // router weights per 16-byte load
+  const bool vec = W % V == 0 && ((uintptr_t)Wr & 15) == 0;
   for (int e = warp; e < E; e += nw) {
     const TW* w = Wr + (int64_t)e * W;
     float a = 0.f;
+    if (vec) {                                    // a lane sums its channels in ascending order
+#pragma unroll 4
+      for (int c = V * lane; c < W; c += 32 * V) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(w + c);
+        const TW* wv = reinterpret_cast<const TW*>(&raw);
+#pragma unroll
+        for (int j = 0; j < V; j += 4) {
+          const float4 xv = *reinterpret_cast<const float4*>(xs + c + j);
+          a = fmaf(xv.x, to_f32(wv[j]), a); a = fmaf(xv.y, to_f32(wv[j + 1]), a);
+          a = fmaf(xv.z, to_f32(wv[j + 2]), a); a = fmaf(xv.w, to_f32(wv[j + 3]), a);
+        }
+      }
+    } else {
 #pragma unroll 8
-    for (int c = lane; c < W; c += 32) a = fmaf(xs[c], to_f32(w[c]), a);
+      for (int c = lane; c < W; c += 32) a = fmaf(xs[c], to_f32(w[c]), a);
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
     if (lane == 0) z[e] = a + (bias ? bias[e] : 0.f);

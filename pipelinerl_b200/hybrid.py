@@ -1219,7 +1219,7 @@ class _Rows:
                 wide_q, wide_aux = max(wide_q, nq), max(wide_aux, g.conv_channels)
                 wide_o = max(wide_o, a.heads * a.vdim, g.heads * g.vdim)
                 wide_o2 = max(wide_o2, g.heads * g.vdim)
-                wide_prep = max(wide_prep, 5 * g.heads * g.dim)
+                wide_prep = max(wide_prep, 5 * g.heads * g.dim, int(eng.lib.prl_gated_delta_split_floats(g.heads, g.dim)))
             elif L.kind == "gla":
                 g = L.gla
                 nq, nv = g.heads * g.dim, g.heads * g.vdim
@@ -1284,7 +1284,7 @@ class _Rows:
         self.act = torch.zeros(n * wide_f, dtype=T, device=d)
         if wide_vfirst:                                         # the first value-blending layer's values of the batch's rows
             self.vfirst = torch.zeros(n * wide_vfirst, **f32)
-        if wide_prep:                                           # u | a u | w | k | r of the gated delta rule
+        if wide_prep:                                           # vectors of the gated delta rule's walk, or products of its pieces
             self.dprep = torch.zeros(n * wide_prep, **f32)
         if cfg.loop_times:                                      # the embedding output and [x | x0], operand type
             self.x0a = torch.zeros(n * W, dtype=T, device=d)
@@ -1335,7 +1335,7 @@ class HybridEngine(EngineCore):
         self.force_plain_gemm = False      # tests: route every GEMM through the CUDA-core kernel
         self.unfused_glu = False           # tests: gate_up GEMM + activation kernel instead of the GEMM's gated epilogue
         self.force_plain_attn = False      # tests: the any-geometry attention kernel also where the tcgen05 ones fit
-        self.unfused_cell = False          # tests: the matrix-memory cell's token step as separate kernels
+        self.unfused_cell = False          # tests: the token step of a memory cell (mLSTM, gated delta rule) as separate kernels
         self.moe_tc_rows = 48              # routed pairs per expert from which the tcgen05 grouped GEMM runs (tests lower it)
         self.unfused_router = False        # tests: router logits through the GEMM and a separate choice kernel
         # Long prompt portions run their recurrences as side-by-side pieces (prl_*_scan_split): same values up to fp32
@@ -1501,8 +1501,10 @@ class HybridEngine(EngineCore):
             return [(L.mlstm.heads, L.mlstm.dim, L.mlstm.vdim + 1)]
         if L.kind == "parallel_lin":
             return [(L.lin.heads, L.lin.dim, L.lin.vdim)]
-        if L.kind in ("latent", "delta", "attention", "latent_attention", "sigmoid_delta", "attn_delta"):
-            return []                      # the delta rules have a scan of their own (delta_scan.cu), walked token by token
+        if L.gdelta is not None:
+            return [(L.gdelta.heads, L.gdelta.dim, L.gdelta.vdim)]      # csrc/gated_delta.cu
+        if L.kind in ("latent", "delta", "attention", "latent_attention"):
+            return []                      # the delta rule with a decay per channel is walked token by token (delta_scan.cu)
         return [(L.ssd.heads, L.ssd.state, L.ssd.vdim)]
 
     def kv_bytes_per_token(self) -> int:
@@ -2087,12 +2089,20 @@ class HybridEngine(EngineCore):
     def _attn_delta_mixer(self, R, n, i, L, w, segs, max_q, row_pos, seg_pos0):
         """Windowed softmax attention (one added to the denominator, one gate per head) beside the gated delta rule, both from
         ONE projection (AttnDeltaRows).  Returns the split-K slice counts of the two output projections (R.y0, R.y1)."""
-        a, g, lib, st, vec, f32, W = L.attn, L.gdelta, self.lib, self._st, self.vec, int(self.f32), self.cfg.width
+        a, g, W = L.attn, L.gdelta, self.cfg.width
+        C = self.cfg.attn_delta_rows(L)
+        self._mm(R.xa, W, w + "mix.in", C.total, R.P, n)
+        self._gated_window_attn(R, n, i, a, C, segs, max_q, row_pos, seg_pos0)
+        k0 = self._mm(R.ya, a.heads * a.vdim, w + "mix.left.o", W, R.y0, n, split=True)
+        self._gated_delta_cell(R, n, i, g, w + "mix.right.", segs, max_q, R.P.data_ptr(), C.total, C.right, C.b, C.a, C.right_g)
+        k1 = self._mm(R.yb, g.heads * g.vdim, w + "mix.right.o", W, R.y1, n, split=True)
+        return k0, k1
+
+    def _gated_window_attn(self, R, n, i, a, C, segs, max_q, row_pos, seg_pos0) -> None:
+        """Softmax attention from the projections in R.P (AttnDeltaRows) to the gated heads R.ya."""
+        lib, st, f32 = self.lib, self._st, int(self.f32)
         seg_start, seg_len, seg_slot, ns = segs
-        C, P = self.cfg.attn_delta_rows(L), R.P.data_ptr()
-        ld, no = C.total, a.heads * a.vdim
-        self._mm(R.xa, W, w + "mix.in", ld, R.P, n)
-        # -- left
+        P, ld, no = R.P.data_ptr(), C.total, a.heads * a.vdim
         bt = (self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE)
         kv = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr())
         _lib.check(lib.prl_attn_front(P, ld, 0, C.k, C.v, n, a.heads, a.kv_heads, a.dim, a.vdim, None, None, None, 0, None, None, a.dim,
@@ -2104,28 +2114,35 @@ class HybridEngine(EngineCore):
                                          0 if a.gate else 1, R.o.data_ptr() if a.gate else R.ya.data_ptr(), st))
         if a.gate:
             _lib.check(lib.prl_gate_heads(R.o.data_ptr(), 1, no, P + 4 * C.left_g, ld, n, a.heads, a.vdim, R.ya.data_ptr(), f32, st))
-        k0 = self._mm(R.ya, no, w + "mix.left.o", W, R.y0, n, split=True)
-        # -- right
-        self._gated_delta_cell(R, n, i, g, w + "mix.right.", segs, max_q, P, ld, C.right, C.b, C.a, C.right_g)
-        k1 = self._mm(R.yb, g.heads * g.vdim, w + "mix.right.o", W, R.y1, n, split=True)
-        return k0, k1
 
     def _gated_delta_cell(self, R, n, i, g, p, segs, max_q, P, ld, off, off_b, off_a, off_g) -> None:
         """From the projections in P (rows ld apart: q | k | v at `off`, step, decay and gate columns) to the cell's normed and
-        gated output R.yb."""
+        gated output R.yb: single tokens in one kernel, long portions as pieces, everything else token by token."""
         lib, st, vec, f32 = self.lib, self._st, self.vec, int(self.f32)
         seg_start, seg_len, seg_slot, ns = segs
         gq, gv, ch = g.kv_heads * g.dim, g.heads * g.vdim, g.conv_channels
-        conv = self.conv_state[i].data_ptr()
+        conv, state, norm = self.conv_state[i].data_ptr(), self.delta_state[i].data_ptr(), vec[p + "norm"].data_ptr()
+        head = (P, ld, off, off_b, off_a, off_g, vec[p + "conv"].data_ptr(), g.conv, vec[p + "A_log"].data_ptr(),
+                vec[p + "dt_bias"].data_ptr(), g.unit_eps, norm, self.cfg.eps, g.heads, g.kv_heads, g.dim, g.vdim)
+        gate = (R.o.data_ptr(), 1, gv, P + 4 * off_g, ld, norm, g.vdim, g.vdim, n, gv, 0, 0, 1, self.cfg.eps, R.yb.data_ptr(), f32, st)
+        if n == ns and not self.unfused_cell and lib.prl_gated_delta_step_fits(g.heads, g.kv_heads, g.dim, g.vdim, g.conv):
+            _lib.check(lib.prl_gated_delta_step(*head, seg_start, seg_len, seg_slot, ns, conv, state, R.yb.data_ptr(), f32, st))
+            return
+        if R.n_sub:
+            _lib.check(lib.prl_gated_delta_split(*head, n, R.row_slot.data_ptr(), R.row_back.data_ptr(), seg_start, seg_len, seg_slot, ns,
+                                                 R.seg_sub[0].data_ptr(), R.seg_sub[1].data_ptr(), R.sub[0].data_ptr(),
+                                                 R.sub[1].data_ptr(), R.n_sub, R.aux.data_ptr(), R.dprep.data_ptr(),
+                                                 R.scratch.data_ptr(), R.o.data_ptr(), conv, state, R.yb.data_ptr(), f32, st))
+            if g.vdim > 128:                 # wider than a CTA of the read-out: its rows come raw
+                _lib.check(lib.prl_gate_norm(*gate))
+            return
         _lib.check(lib.prl_conv_silu(P, ld, off, n, ch, g.conv, vec[p + "conv"].data_ptr(), self.zero_bias.data_ptr(),
                                      R.row_slot.data_ptr(), R.row_back.data_ptr(), conv, R.aux.data_ptr(), st))
         _lib.check(lib.prl_conv_state_update(P, ld, off, ch, g.conv, seg_start, seg_len, seg_slot, ns, conv, st))
         _lib.check(lib.prl_gated_delta_scan(R.aux.data_ptr(), ch, 0, gq, 2 * gq, P, ld, off_b, off_a, vec[p + "A_log"].data_ptr(),
                                             vec[p + "dt_bias"].data_ptr(), g.unit_eps, g.heads, g.kv_heads, g.dim, g.vdim, n,
-                                            R.dprep.data_ptr(), seg_start, seg_len, seg_slot, ns, max_q,
-                                            self.delta_state[i].data_ptr(), R.o.data_ptr(), gv, st))
-        _lib.check(lib.prl_gate_norm(R.o.data_ptr(), 1, gv, P + 4 * off_g, ld, vec[p + "norm"].data_ptr(), g.vdim, g.vdim, n, gv, 0, 0, 1,
-                                     self.cfg.eps, R.yb.data_ptr(), f32, st))
+                                            R.dprep.data_ptr(), seg_start, seg_len, seg_slot, ns, max_q, state, R.o.data_ptr(), gv, st))
+        _lib.check(lib.prl_gate_norm(*gate))
 
     # ---- the multi-stream program: latent attention and delta-rule layers ------------------------------------------------
     def _stream_weights(self, i: int, q: str):
@@ -2331,6 +2348,23 @@ class HybridEngine(EngineCore):
         self._mm(R.xa, cfg.width, self.head_name, cfg.vocab_size, self.logits, B)
         self._cap_logits(self.logits, B)
 
+    def stage_pieces(self, R: _Rows, starts: list, lens: list) -> None:
+        """Piece tables of a batch of segments (first rows, lengths) whose recurrences run as side-by-side pieces."""
+        R.n_sub = 0
+        if not self.split_scan or max(lens) < self.split_min_rows:
+            return
+        step = min(self.piece_tokens, int(self.lib.prl_lin_scan_piece_tokens()))
+        sub, seg_sub = [[], []], [[], []]
+        for start, k in zip(starts, lens):
+            seg_sub[0].append(len(sub[0]))
+            seg_sub[1].append((k + step - 1) // step)
+            sub[0] += range(start, start + k, step)
+            sub[1] += [min(step, k - c) for c in range(0, k, step)]
+        if len(sub[0]) <= R.max_sub:              # else: many short segments beside the long one, walk them token by token
+            R.n_sub = len(sub[0])
+            R.sub[:, :R.n_sub].copy_(torch.tensor(sub, dtype=torch.int32), non_blocking=True)
+            R.seg_sub[:, :len(starts)].copy_(torch.tensor(seg_sub, dtype=torch.int32), non_blocking=True)
+
     # ---- a packed batch of prompt portions (prefill chunks, token streams) --------------------------------------------
     def _forward_rows(self, segs, want_rows, trace=None):
         cfg, lib = self.cfg, self.lib
@@ -2351,19 +2385,7 @@ class HybridEngine(EngineCore):
             at += k
         ns = len(segs)
         i32 = torch.int32
-        R.n_sub = 0
-        if self.split_scan and max(k for _, _, k in segs) >= self.split_min_rows:
-            step = min(self.piece_tokens, int(lib.prl_lin_scan_piece_tokens()))
-            sub, seg_sub = [[], []], [[], []]
-            for start, k in zip(meta[0], meta[1]):
-                seg_sub[0].append(len(sub[0]))
-                seg_sub[1].append((k + step - 1) // step)
-                sub[0] += range(start, start + k, step)
-                sub[1] += [min(step, k - c) for c in range(0, k, step)]
-            if len(sub[0]) <= R.max_sub:          # else: many short segments beside the long one, walk them token by token
-                R.n_sub = len(sub[0])
-                R.sub[:, :R.n_sub].copy_(torch.tensor(sub, dtype=i32), non_blocking=True)
-                R.seg_sub[:, :ns].copy_(torch.tensor(seg_sub, dtype=i32), non_blocking=True)
+        self.stage_pieces(R, meta[0], meta[1])
         R.tokens[:n].copy_(torch.tensor(toks, dtype=i32), non_blocking=True)
         R.row_pos[:n].copy_(torch.tensor(pos, dtype=i32), non_blocking=True)
         R.row_slot[:n].copy_(torch.tensor(slot, dtype=i32), non_blocking=True)

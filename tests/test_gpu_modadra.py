@@ -369,6 +369,66 @@ def test_tensor_core_prompt_attention(cuda_device, dim, vdim, window):
         assert mc.rel_err(f, ref) < BF16_TOL and mc.rel_err(p, ref) < BF16_TOL
 
 
+CELLS = [(4, 2, 12, 8, 3), (3, 1, 10, 13, 4), (2, 2, 32, 48, 2), (4, 2, 64, 64, 4), (2, 1, 128, 128, 4), (2, 1, 40, 132, 1), (1, 1, 200, 20, 4),
+         (6, 2, 5, 40, 6)]       # heads, q / k heads, key size, value size, taps
+
+
+@pytest.mark.parametrize("heads,kv,dk,dv,taps", CELLS)
+def test_pieces_of_the_gated_delta_rule(cuda_device, heads, kv, dk, dv, taps):
+    """Long portions as side-by-side pieces (off in fp32 unless asked for) against the oracle and the token-by-token walk: one
+    piece that is not full, several, pieces of other lengths, portions that continue a state, and single tokens of another
+    sequence beside them.  Memories that last (decays near one) make a wrong state at a piece's border show in every row
+    behind it."""
+    config = mc.model([P(window=5, r_heads=heads, r_kv_heads=kv, r_dim=dk, r_vdim=dv, conv=taps)], width=40)
+    for shift in (-3.0, 1.0):
+        wt = mc.weights(config, 27)
+        wt["l0.mix.right.A_log"] = mc.bf16_round(wt["l0.mix.right.A_log"] + shift)
+        wt["l0.mix.left.out"] = mc.bf16_round(wt["l0.mix.left.out"] * 0.1)
+        toks, other = mc.tokens_for(config, 300, seed=21), mc.tokens_for(config, 20, seed=22)
+        ref, oref = mc.oracle_logits(config, wt, toks), mc.oracle_logits(config, wt, other)
+        eng = mc.build_engine(config, wt, torch.float32, cuda_device, prefill_chunk=320)
+        walked = mc.stream_logits(eng, toks, [300])
+        eng.split_scan, eng.split_min_rows = True, 2
+        for step in (64, 23):
+            eng.piece_tokens = step
+            for portions in ([300], [64, 65, 2, 100], [130, 1, 2, 3]):
+                got = mc.stream_logits(eng, toks, portions)
+                assert mc.rel_err(got, ref) < F32_TOL and mc.rel_err(got, walked) < 2e-5
+        a, b = eng.open_stream(), eng.open_stream()
+        rows = [[], []]
+        for k, (na, nb) in enumerate([(100, 5), (70, 1), (2, 1), (128, 13)]):
+            at, bt = sum(x.shape[0] for x in rows[0]), sum(x.shape[0] for x in rows[1])
+            lg = eng.feed([(a, toks[at:at + na], list(range(na))), (b, other[bt:bt + nb], list(range(nb)))]).double().cpu()
+            rows[0].append(lg[:na]); rows[1].append(lg[na:])
+        eng.close_stream(a); eng.close_stream(b)
+        assert mc.rel_err(torch.cat(rows[0]), ref) < F32_TOL and mc.rel_err(torch.cat(rows[1]), oref) < F32_TOL
+
+
+@pytest.mark.parametrize("heads,kv,dk,dv,taps", CELLS)
+def test_token_step_of_the_gated_delta_rule(cuda_device, heads, kv, dk, dv, taps):
+    """The one-kernel token step against the separate kernels and the oracle, behind a prompt, with an idle slot beside it, and
+    with the state handed from one path to the other in the middle."""
+    config = mc.model([P(window=5, r_heads=heads, r_kv_heads=kv, r_dim=dk, r_vdim=dv, conv=taps)], width=40)
+    wt = mc.weights(config, 28)
+    wt["l0.mix.left.out"] = mc.bf16_round(wt["l0.mix.left.out"] * 0.1)
+    toks = mc.tokens_for(config, 60, seed=23)
+    ref = mc.oracle_logits(config, wt, toks)
+    eng = mc.build_engine(config, wt, torch.float32, cuda_device)
+    assert eng.lib.prl_gated_delta_step_fits(heads, kv, dk, dv, taps)
+    assert mc.rel_err(mc.stream_logits(eng, toks, []), ref) < F32_TOL
+    eng.unfused_cell = True
+    separate = mc.stream_logits(eng, toks, [])
+    eng.unfused_cell = False
+    assert mc.rel_err(mc.stream_logits(eng, toks, []), separate) < 2e-5
+    s, out, at = eng.open_stream(), [], 0
+    for k in (7, 1, 1, 1, 2, 1, 1, 20):
+        eng.unfused_cell = at % 2 == 0
+        out.append(eng.feed([(s, toks[at:at + k], list(range(k)))]))
+        at += k
+    eng.close_stream(s)
+    assert mc.rel_err(torch.cat(out).double().cpu(), ref[:at]) < F32_TOL
+
+
 def test_long_decoding(cuda_device):
     """A short prompt and 400 single tokens over six page borders and several windows, in fp32 against the oracle."""
     config = mc.model([P(mlp=M(), window=150), P(window=64)])

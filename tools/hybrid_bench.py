@@ -121,6 +121,20 @@ def futetar_config(s):
     return dict(architecture="Futetar", vocab=s["vocab"], width=W, norm=dict(eps=1e-5), layers=[block[i % 4] for i in range(s["layers"])])
 
 
+def modadra_config(s):
+    """Eight layers of windowed attention (heads of 128, 64 rotated channels, window 1024) beside the gated delta rule (heads
+    of 128 x 128 on half as many q / k heads, four taps), as in the Kolotar model, every layer with routed experts of the
+    dense ff's active width (four of sixteen experts of ff / 4, three of four groups)."""
+    W, ff, H, G = s["width"], s["ff"], s["heads"], s["kv"]
+    routed = dict(kind="moe", router=dict(experts=16, top=4, scale=1.5, groups=dict(count=4, keep=3)), expert=dict(ff=ff // 4))
+    par = dict(type="parallel", mlp=routed,
+               mixer=dict(left=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024),
+                                    rot=dict(base=1e6, dims=64)),
+                          right=dict(heads=W // 128, kv_heads=max(1, W // 256), dim=128, vdim=128, conv=4)))
+    return dict(architecture="Modadra", vocab=s["vocab"], width=W, norm=dict(eps=1e-5), residual_mult=0.5, logit_softcap=30.0,
+                layers=[par] * s["layers"])
+
+
 def peaks():
     try:
         p = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())
@@ -666,6 +680,122 @@ def run_futetar(sizes, prompt, context, batch, steps, warm, kernels=True, e2e=Tr
     return res
 
 
+def run_modadra(sizes, prompt, context, batch, steps, warm, kernels=True, e2e=True, others=True):
+    """Modadra beside Kolotar (the closest design: windowed attention with a sink, the gated delta rule, routed experts in
+    every layer) and the Qwen2 engine at equal width / depth / active ff / attention heads."""
+    from pipelinerl_b200.engine import DecodeEngine
+    from pipelinerl_b200.hybrid import HybridConfig, HybridEngine
+    from pipelinerl_b200.model import ModelConfig, ParamArena
+    dev = torch.device("cuda:0")
+    timer = Timer()
+    res = {}
+    for name in sizes:
+        s = SIZES[name]
+        kw = dict(max_batch=batch, max_seq_len=max(prompt, context) + 256, max_new_tokens=warm + steps + 8, device=dev,
+                  prefill_chunk=1024)
+        entry = {}
+        models = {"modadra": (HybridEngine, HybridConfig.from_modadra(modadra_config(s)))}
+        if others:
+            models = {"qwen2": (DecodeEngine, ModelConfig(vocab_size=s["vocab"], hidden_size=s["width"], intermediate_size=s["ff"],
+                                                          num_layers=s["layers"], num_q_heads=s["heads"], num_kv_heads=s["kv"])),
+                      "kolotar": (HybridEngine, HybridConfig.from_kolotar(kolotar_config(s))), **models}
+        for model, (cls, cfg) in models.items():
+            eng = cls(cfg, ParamArena(cfg, dev).init_random(seed=1), **kw)
+            if e2e:
+                entry[model] = end_to_end(eng, s["vocab"], prompt, context, batch, steps, warm)
+                entry[model]["params_M"] = round(cfg.num_params() / 1e6)
+            if kernels and model in ("modadra", "kolotar"):
+                table = kernel_table_modadra if model == "modadra" else kernel_table_kolotar
+                entry[f"kernels_{model}" if model != "modadra" else "kernels"] = table(eng, s, batch, 1024, timer)
+            del eng
+            torch.cuda.empty_cache()
+        if e2e and others:
+            for other in ("qwen2", "kolotar"):
+                entry[f"modadra_over_{other}"] = {k: round(entry["modadra"][f"{k}_tokens_per_s"] / entry[other][f"{k}_tokens_per_s"], 3)
+                                                  for k in ("prefill", "decode")}
+        res[name] = entry
+    return res
+
+
+def kernel_table_modadra(eng, s, batch, chunk, timer):
+    """The parts of a Modadra layer alone, at the decode shape (`batch` one-token segments at position 2047) and the prefill
+    shape (one segment of `chunk` rows whose sequence already holds `chunk` tokens): the engine's own methods on its buffers;
+    weight streams, caches, states and row kernels against the measured copy bandwidth, products of many rows and attention
+    against the measured bf16 GEMM rate, the recurrence against the SMs' fp32 FMA rate."""
+    from pipelinerl_b200 import _lib
+    from pipelinerl_b200.cache import PAGE_SIZE
+    from pipelinerl_b200.hybrid import _Rows
+    lib, cfg = eng.lib, eng.cfg
+    hbm, tflops, how = peaks()
+    fma_tflops = 148 * 128 * 2 * 1.965e9 / 1e12
+    W, i, L, m = cfg.width, 0, cfg.layers[0], cfg.residual_mult
+    a, g, e, C, w = L.attn, L.gdelta, L.mlp.moe, cfg.attn_delta_rows(L), "l0."
+    no, gv = a.heads * a.vdim, g.heads * g.vdim
+    out = {"peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "fp32_fma_tflops": round(fma_tflops, 1), "source": how}}
+    i32 = dict(dtype=torch.int32, device=eng.dev)
+    ctx = 2047
+    pages_per = (ctx + PAGE_SIZE) // PAGE_SIZE
+    for b in range(batch):
+        eng.block_table[b, :pages_per].copy_(torch.arange(1 + b * pages_per, 1 + (b + 1) * pages_per, **i32))
+    for pools in (eng.k_pool, eng.v_pool):
+        for pool in pools.values():
+            pool.normal_(0, 0.5)
+    for shape, n, ns in (("decode", batch, batch), ("prefill", chunk, 1)):
+        decode = shape == "decode"
+        R = _Rows(eng, n, pieces=not decode)
+        R.P.normal_(0, 0.5); R.xa.normal_(0, 0.5); R.x.normal_(0, 0.5); R.ya.normal_(0, 0.5); R.yb.normal_(0, 0.5)
+        pos0 = ctx if decode else chunk
+        if decode:
+            R.seg.copy_(torch.stack([torch.arange(n, **i32), torch.ones(n, **i32), torch.full((n,), ctx, **i32), torch.arange(n, **i32)]))
+            R.row_slot.copy_(torch.arange(n, **i32)); R.row_pos.fill_(ctx)
+        else:
+            R.seg[:, :1].copy_(torch.tensor([[0], [n], [pos0], [0]], **i32))
+            R.row_slot.zero_(); R.row_pos.copy_(torch.arange(pos0, pos0 + n, **i32)); R.row_back.copy_(torch.arange(n, **i32))
+            eng.stage_pieces(R, [0], [n])
+        eng._st = _lib.stream_ptr()
+        segs = (R.seg[0].data_ptr(), R.seg[1].data_ptr(), R.seg[3].data_ptr(), ns)
+        max_q = 1 if decode else n
+        seen = sum(min(a.window or p + 1, p + 1) for p in ([ctx] * n if decode else range(pos0, pos0 + n)))
+        cached = seen if decode else min(pos0, (a.window or pos0) - 1) + n
+        t, hb, fl = {}, {}, {}
+        t["in_product"] = timer.events(lambda: eng._mm(R.xa, W, w + "mix.in", C.total, R.P, n))
+        hb["in_product"], fl["in_product"] = (C.total + n) * W * 2 + n * C.total * 4, 2.0 * n * C.total * W
+        t["attention"] = timer.events(lambda: eng._gated_window_attn(R, n, i, a, C, segs, max_q, R.row_pos, R.seg[2]))
+        hb["attention"], fl["attention"] = cached * a.kv_heads * (a.dim + a.vdim) * 2, 2.0 * seen * a.heads * (a.dim + a.vdim)
+        t["gated_delta_cell"] = timer.events(lambda: eng._gated_delta_cell(R, n, i, g, w + "mix.right.", segs, max_q, R.P.data_ptr(), C.total,
+                                                                           C.right, C.b, C.a, C.right_g))
+        hb["gated_delta_cell"] = 2 * ns * g.heads * g.dim * g.vdim * 4 + n * ((g.conv_channels + gv) * 4 + gv * 2)
+        t["left_o_product"] = timer.events(lambda: eng._mm(R.ya, no, w + "mix.left.o", W, R.y0, n, split=True))
+        hb["left_o_product"], fl["left_o_product"] = no * (W + n) * 2 + n * W * 4, 2.0 * n * no * W
+        t["mixer_close"] = timer.events(lambda: eng._close(R, n, R.y0, 1, gain0=eng.vec[w + "mix.left.out"], s0=0.5 * m, y1=R.y1, k1=1,
+                                                           gain1=eng.vec[w + "mix.right.out"], s1=0.5 * m, next_gain=eng.vec[w + "norm2"]))
+        hb["mixer_close"] = n * W * (4 * 4 + 2)
+        rule = (e.top, e.groups, e.keep_groups, e.group_top, 1, 1, e.weight_scale, 64, R.sel.data_ptr(), R.wsel.data_ptr(), R.perm.data_ptr(),
+                R.moe_meta.data_ptr(), R.moe_tiles.data_ptr(), eng._st)
+        t["router"] = timer.events(lambda: _lib.check(lib.prl_moe_router_choose(
+            R.xa.data_ptr(), 0, eng.arena.ptr(w + "mlp.router"), 0, eng.vec[w + "mlp.correction"].data_ptr(), n, W, e.experts, e.outputs, *rule)))
+        hb["router"] = (e.experts + n) * W * 2
+        t["routed_experts"] = timer.events(lambda: eng._choose_and_run_experts(R, n, w, e))
+        live = n * e.top
+        used = len(torch.unique(R.sel[:live]))
+        hb["routed_experts"], fl["routed_experts"] = used * 2 * e.ff * W * 2 + live * (W * 6 + e.ff * 4), 4.0 * live * e.ff * W
+        t["ff_close"] = timer.events(lambda: eng._close(R, n, R.moe_out, e.top, s0=m, next_gain=eng.vec[w + "norm1"]))
+        hb["ff_close"] = n * W * (4 * 2 + 2) + live * W * 4
+        row = {k: {"us": round(v * 1e3, 1)} for k, v in t.items()}
+        for k in t:
+            if decode or k not in fl:
+                row[k]["of_hbm"] = round(hb[k] / t[k] / 1e6 / hbm, 3)
+            else:
+                row[k]["of_bf16_peak"] = round(fl[k] / t[k] / 1e9 / tflops, 3)
+        row["gated_delta_cell"]["of_fp32_fma"] = round(5.0 * 2 * n * g.heads * g.dim * g.vdim / t["gated_delta_cell"] / 1e9 / fma_tflops, 3)
+        out[shape] = row
+        del R
+    eng.block_table.zero_()
+    for b in range(batch):
+        eng.states.reset(b)
+    return out
+
+
 def kernel_table_futetar(eng, s, batch, chunk, timer):
     """The parts of the Futetar layers alone, at the decode shape (`batch` one-token segments at position 2047) and the
     prefill shape (one segment of `chunk` rows whose sequence already holds `chunk` tokens): the engine's own methods on its
@@ -999,12 +1129,15 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--only-kernels", action="store_true", help="skip the end-to-end runs (a small case for a profiler)")
-    ap.add_argument("--design", default="povurax", choices=["povurax", "belelorn", "pametar", "kolotar", "futetar"], help="which hybrid design is measured")
+    ap.add_argument("--design", default="povurax", choices=["povurax", "belelorn", "pametar", "kolotar", "futetar", "modadra"], help="which hybrid design is measured")
     ap.add_argument("--alone", action="store_true", help="--design belelorn: skip the Qwen2 and Povurax runs beside it")
     a = ap.parse_args()
     from pipelinerl_b200 import _lib
     before = _lib.launch_count()
-    if a.design == "futetar":
+    if a.design == "modadra":
+        res = run_modadra(a.sizes.split(","), a.prompt, a.context, a.batch, a.steps, a.warmup, kernels=not a.no_kernels,
+                          e2e=not a.only_kernels, others=not a.alone)
+    elif a.design == "futetar":
         res = run_futetar(a.sizes.split(","), a.prompt, a.context, a.batch, a.steps, a.warmup, kernels=not a.no_kernels,
                           e2e=not a.only_kernels, others=not a.alone)
     elif a.design == "kolotar":
