@@ -802,6 +802,13 @@ int prl_attn_any_sink(const void* q, const void* k_pool, const void* v_pool, int
                       const int32_t* seg_len, const int32_t* seg_pos0, const int32_t* seg_slot, int32_t n_seg, int32_t max_q,
                       int32_t H, int32_t G, int32_t dim, int32_t vdim, float scale, int32_t window, int32_t keep_first,
                       float softcap, const float* sink, int32_t out_is_t, void* out, prl_stream_t stream);
+/* ... and one gate per query head: the head's output times sigmoid(gate[row * ldg + head]) (NULL: none) */
+int prl_attn_any_gated(const void* q, const void* k_pool, const void* v_pool, int32_t ldv, int32_t f32,
+                       const int32_t* block_table, int32_t max_blocks, int32_t page_size, const int32_t* seg_start,
+                       const int32_t* seg_len, const int32_t* seg_pos0, const int32_t* seg_slot, int32_t n_seg, int32_t max_q,
+                       int32_t H, int32_t G, int32_t dim, int32_t vdim, float scale, int32_t window, int32_t keep_first,
+                       float softcap, const float* sink, const float* gate, int64_t ldg, int32_t out_is_t, void* out,
+                       prl_stream_t stream);
 /* tensor-core attention over a latent cache (bf16): q [n][H][kd], pool [page][page_size][kd], values = the first `rank`
  * channels of the key rows, optional per-head sink logit; out bf16 [n][H][rank].  prl_attn_latent_fits says whether the
  * geometry is built (kd, rank multiples of 16, rank <= 256, pages of a multiple of 32 tokens) */

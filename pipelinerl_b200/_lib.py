@@ -349,6 +349,7 @@ _SIGNATURES = {
                                     C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_int32,
                                     C.c_int32, C.c_int32, C.c_float, C.c_int32, C.c_int32, C.c_float, C.c_void_p, C.c_int32,
                                     C.c_void_p, C.c_void_p]),
+    "prl_attn_any_gated": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_int32, C.c_int32, C.c_int32, C.c_float, C.c_int32, C.c_int32, C.c_float, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_void_p, C.c_void_p]),
     "prl_attn_latent_fits": (C.c_int32, [C.c_int32, C.c_int32, C.c_int32]),
     "prl_attn_latent_splits": (C.c_int32, [C.c_int32, C.c_int32]),
     "prl_attn_latent_workspace_bytes": (C.c_size_t, [C.c_int32, C.c_int32, C.c_int32]),

@@ -26,7 +26,11 @@ bool attn_mma_fits(int dim, int vdim, const void* q, const void* k_pool, const v
 int attn_mma_launch(const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
                     const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int max_q, int H,
                     int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, const float* sink,
-                    int out_is_bf16, void* out, cudaStream_t st);
+                    const float* gate, int64_t ldg, int out_is_bf16, void* out, cudaStream_t st);
+int attn_mma_decode_launch(const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
+                           const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int H, int G,
+                           int dim, int vdim, float scale, int window, int keep_first, float softcap, const float* sink,
+                           const float* gate, int64_t ldg, int out_is_bf16, void* out, cudaStream_t st);
 
 namespace {
 
@@ -37,6 +41,8 @@ template <typename T> __device__ __forceinline__ float cvt(T v);
 template <> __device__ __forceinline__ float cvt<float>(float v) { return v; }
 template <> __device__ __forceinline__ float cvt<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
 
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+
 template <typename T, int VR, bool OUT_T, int RW>
 __global__ void __launch_bounds__(256) attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
                                                        const T* __restrict__ v_pool, const int32_t* __restrict__ block_table,
@@ -44,7 +50,8 @@ __global__ void __launch_bounds__(256) attn_any_kernel(const T* __restrict__ q, 
                                                        const int32_t* __restrict__ seg_len, const int32_t* __restrict__ seg_pos0,
                                                        const int32_t* __restrict__ seg_slot, int H, int G, int dim, int vdim,
                                                        float scale, int window, int keep_first, float softcap,
-                                                       int ldv, const float* __restrict__ sink, void* __restrict__ out_v) {
+                                                       int ldv, const float* __restrict__ sink, const float* __restrict__ gate, int64_t ldg,
+    void* __restrict__ out_v) {
   pdl_wait();   // launched with the programmatic-serialization attribute like the engine's other step kernels; no early
                 // trigger: letting the next grid become resident early measured +3 ms on a 4096-token prefill and +-0 on decode
   // RW consecutive query rows per warp (kWarpsPerCta * RW per CTA): a staged key tile is scored against all of them in
@@ -181,7 +188,8 @@ __global__ void __launch_bounds__(256) attn_any_kernel(const T* __restrict__ q, 
 #pragma unroll
       for (int i = 0; i < VR; ++i) acc[r][i] *= corr;
     }
-    const float inv = 1.f / l[r];
+    float inv = 1.f / l[r];
+    if (gate) inv *= sigmoid_f(gate[(row0 + my_i) * ldg + h]);
 #pragma unroll
     for (int i = 0; i < VR; ++i) {
       const int c = lane + 32 * i;
@@ -196,7 +204,7 @@ __global__ void __launch_bounds__(256) attn_any_kernel(const T* __restrict__ q, 
 template <typename T, int VR, bool OUT_T, int RW>
 int launch_attn_rw(const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
                    const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int max_q, int H,
-                   int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink,
+                   int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink, const float* gate, int64_t ldg,
                    void* out, cudaStream_t st) {
   constexpr int kRows = kWarpsPerCta * RW;
   const size_t smem = ((size_t)kKeysPerTile * (dim + 1) + (size_t)kKeysPerTile * vdim + (size_t)kRows * dim) * sizeof(float);
@@ -204,7 +212,7 @@ int launch_attn_rw(const void* q, const void* kp, const void* vp, const int32_t*
   if (smem > 48 * 1024) PRL_CUDA(ensure_smem(attn_any_kernel<T, VR, OUT_T, RW>, (int)smem, attr));
   dim3 grid((max_q + kRows - 1) / kRows, H, n_seg);
   PRL_CUDA(launch_pdl((attn_any_kernel<T, VR, OUT_T, RW>), dim3(grid), dim3(256), (size_t)(smem), st, (const T*)q, (const T*)kp, (const T*)vp, bt, max_blocks, page_size, ss, sl,
-                      sp, sslot, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out));
+                      sp, sslot, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -213,13 +221,13 @@ int launch_attn_rw(const void* q, const void* kp, const void* vp, const int32_t*
 template <typename T, int VR, bool OUT_T>
 int launch_attn(const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
                 const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int max_q, int H,
-                int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink,
+                int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink, const float* gate, int64_t ldg,
                 void* out, cudaStream_t st) {
   if (max_q >= 64 && VR <= 4)
     return launch_attn_rw<T, VR, OUT_T, 4>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim,
-                                           scale, window, keep_first, softcap, ldv, sink, out, st);
+                                           scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st);
   return launch_attn_rw<T, VR, OUT_T, 1>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim,
-                                         scale, window, keep_first, softcap, ldv, sink, out, st);
+                                         scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st);
 }
 
 // ---- single-token segments (a decode step) ------------------------------------------------------------------------------
@@ -254,7 +262,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) attn_decode_any_kernel(
     const T* __restrict__ q, const T* __restrict__ k_pool, const T* __restrict__ v_pool, const int32_t* __restrict__ block_table,
     int max_blocks, int page_size, const int32_t* __restrict__ seg_start, const int32_t* __restrict__ seg_len,
     const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ seg_slot, int H, int G, int dim, int vdim, float scale,
-    int window, int keep_first, float softcap, int ldv, const float* __restrict__ sink, void* __restrict__ out_v) {
+    int window, int keep_first, float softcap, int ldv, const float* __restrict__ sink, const float* __restrict__ gate, int64_t ldg,
+    void* __restrict__ out_v) {
   pdl_wait();
   extern __shared__ float sm[];
   const int seg = blockIdx.y;
@@ -395,15 +404,16 @@ __global__ void __launch_bounds__(kDecWarps * 32) attn_decode_any_kernel(
       den = fmaf(wgt, pw[vdim + 1], den);
     }
     const int64_t o = (row * H + h0 + hh) * vdim + c;
-    if constexpr (OUT_T) reinterpret_cast<T*>(out_v)[o] = T(num / den);
-    else reinterpret_cast<float*>(out_v)[o] = num / den;
+    const float y = gate ? num / den * sigmoid_f(gate[row * ldg + h0 + hh]) : num / den;
+    if constexpr (OUT_T) reinterpret_cast<T*>(out_v)[o] = T(y);
+    else reinterpret_cast<float*>(out_v)[o] = y;
   }
 }
 
 template <typename T, int VR, bool OUT_T>
 int launch_attn_decode(const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
                        const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int H, int G,
-                       int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink,
+                       int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink, const float* gate, int64_t ldg,
                        void* out, cudaStream_t st) {
   const size_t smem = ((size_t)kDecHeads * dim + (size_t)kDecWarps * kDecHeads * (vdim + 2)) * sizeof(float);
   static SmemAttr attr = {};
@@ -411,7 +421,7 @@ int launch_attn_decode(const void* q, const void* kp, const void* vp, const int3
   const int groups = (H / G + kDecHeads - 1) / kDecHeads;
   PRL_CUDA(launch_pdl((attn_decode_any_kernel<T, VR, OUT_T>), dim3(G * groups, n_seg), dim3(kDecWarps * 32), smem, st, (const T*)q,
                       (const T*)kp, (const T*)vp, bt, max_blocks, page_size, ss, sl, sp, sslot, H, G, dim, vdim, scale, window,
-                      keep_first, softcap, ldv, sink, out));
+                      keep_first, softcap, ldv, sink, gate, ldg, out));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -419,12 +429,12 @@ int launch_attn_decode(const void* q, const void* kp, const void* vp, const int3
 template <typename T>
 int dispatch_attn(int vr, const void* q, const void* kp, const void* vp, const int32_t* bt, int max_blocks, int page_size,
                   const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int max_q, int H,
-                  int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink, int out_is_t,
+                  int G, int dim, int vdim, float scale, int window, int keep_first, float softcap, int ldv, const float* sink, const float* gate, int64_t ldg, int out_is_t,
                   void* out, cudaStream_t st) {
-#define PRL_ATTN(VR) (out_is_t ? launch_attn<T, VR, true>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out, st) \
-                               : launch_attn<T, VR, false>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out, st))
-#define PRL_ATTN_DEC(VR) (out_is_t ? launch_attn_decode<T, VR, true>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out, st) \
-                                   : launch_attn_decode<T, VR, false>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out, st))
+#define PRL_ATTN(VR) (out_is_t ? launch_attn<T, VR, true>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st) \
+                               : launch_attn<T, VR, false>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st))
+#define PRL_ATTN_DEC(VR) (out_is_t ? launch_attn_decode<T, VR, true>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st) \
+                                   : launch_attn_decode<T, VR, false>(q, kp, vp, bt, max_blocks, page_size, ss, sl, sp, sslot, n_seg, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out, st))
   if (max_q == 1 && page_size % kKeysPerTile == 0) {          // every segment is one token (or empty): the decode kernel
     if (vr <= 1) return PRL_ATTN_DEC(1);
     if (vr <= 2) return PRL_ATTN_DEC(2);
@@ -457,7 +467,7 @@ static int attn_any_impl(const void* q, const void* k_pool, const void* v_pool, 
                          const int32_t* seg_pos0, const int32_t* seg_slot, int32_t n_seg, int32_t max_q, int32_t H,
                          int32_t G, int32_t dim, int32_t vdim, float scale, int32_t window, int32_t keep_first,
                          float softcap, int32_t out_is_t, void* out, prl_stream_t st, int32_t ldv = 0,
-                         const float* sink = nullptr) {
+                         const float* sink = nullptr, const float* gate = nullptr, int64_t ldg = 0) {
   if (ldv <= 0) ldv = vdim;
   PRL_CHECK_ARG(ldv >= vdim, "prl_attn_any: value row stride %d below the value size %d", ldv, vdim);
   PRL_CHECK_ARG(q && k_pool && v_pool && block_table && seg_start && seg_len && seg_pos0 && seg_slot && out,
@@ -469,11 +479,14 @@ static int attn_any_impl(const void* q, const void* k_pool, const void* v_pool, 
   const int vr = (vdim + 31) / 32;
   if (!f32 && g_attn_tensor_cores && max_q >= kMmaMinRows && ldv == vdim && attn_mma_fits(dim, vdim, q, k_pool, v_pool))
     return attn_mma_launch(q, k_pool, v_pool, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0, seg_slot, n_seg,
-                           max_q, H, G, dim, vdim, scale, window, keep_first, softcap, sink, out_is_t, out, (cudaStream_t)st);
+                           max_q, H, G, dim, vdim, scale, window, keep_first, softcap, sink, gate, ldg, out_is_t, out, (cudaStream_t)st);
+  if (!f32 && g_attn_tensor_cores && max_q == 1 && ldv == vdim && page_size % 32 == 0 && attn_mma_fits(dim, vdim, q, k_pool, v_pool))
+    return attn_mma_decode_launch(q, k_pool, v_pool, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0, seg_slot, n_seg, H, G,
+                                  dim, vdim, scale, window, keep_first, softcap, sink, gate, ldg, out_is_t, out, (cudaStream_t)st);
   if (f32) return dispatch_attn<float>(vr, q, k_pool, v_pool, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0,
-                                       seg_slot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out_is_t, out, (cudaStream_t)st);
+                                       seg_slot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out_is_t, out, (cudaStream_t)st);
   return dispatch_attn<__nv_bfloat16>(vr, q, k_pool, v_pool, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0,
-                                      seg_slot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, out_is_t, out, (cudaStream_t)st);
+                                      seg_slot, n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, ldv, sink, gate, ldg, out_is_t, out, (cudaStream_t)st);
 }
 
 extern "C" int prl_attn_any(const void* q, const void* k_pool, const void* v_pool, int32_t f32, const int32_t* block_table,
@@ -507,4 +520,15 @@ extern "C" int prl_attn_any_sink(const void* q, const void* k_pool, const void* 
                                  prl_stream_t st) {
   return attn_any_impl(q, k_pool, v_pool, f32, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0, seg_slot,
                        n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, out_is_t, out, st, ldv, sink);
+}
+
+// As prl_attn_any_sink with one gate per query head: the head's output times sigmoid(gate[row * ldg + head]).
+extern "C" int prl_attn_any_gated(const void* q, const void* k_pool, const void* v_pool, int32_t ldv, int32_t f32,
+                                  const int32_t* block_table, int32_t max_blocks, int32_t page_size, const int32_t* seg_start,
+                                  const int32_t* seg_len, const int32_t* seg_pos0, const int32_t* seg_slot, int32_t n_seg,
+                                  int32_t max_q, int32_t H, int32_t G, int32_t dim, int32_t vdim, float scale, int32_t window,
+                                  int32_t keep_first, float softcap, const float* sink, const float* gate, int64_t ldg,
+                                  int32_t out_is_t, void* out, prl_stream_t st) {
+  return attn_any_impl(q, k_pool, v_pool, f32, block_table, max_blocks, page_size, seg_start, seg_len, seg_pos0, seg_slot,
+                       n_seg, max_q, H, G, dim, vdim, scale, window, keep_first, softcap, out_is_t, out, st, ldv, sink, gate, ldg);
 }

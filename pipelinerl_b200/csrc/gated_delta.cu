@@ -61,15 +61,19 @@ __device__ __forceinline__ float4 lds4(const float* p) { return *reinterpret_cas
 // `cols_pad` are zero.  `vec`: every source row starts on a 16-byte boundary and cols is a multiple of four.
 __device__ __forceinline__ void stage_tile(float* dst, int ld_dst, const float* src, int64_t ld_src, int rows, int live, int cols,
                                            int cols_pad, bool vec) {
-  if (vec) {
-    const int per = cols_pad / 4;
-    for (int i = threadIdx.x; i < rows * per; i += kThreads) {
-      const int r = i / per, c = (i - r * per) * 4;
-      const bool on = r < live && c < cols;
-      cp16z(dst + r * ld_dst + c, src + (on ? r * ld_src + c : 0), on ? 16 : 0);
+  if (vec) {                       // a thread keeps its column and steps over the rows
+    const int per = cols_pad / 4, step = blockDim.x / per, c = threadIdx.x % per * 4;
+    int r = threadIdx.x / per;
+    if (r < step) {
+      const float* p = src + r * ld_src + c;
+      float* d = dst + r * ld_dst + c;
+      for (; r < rows; r += step, p += step * ld_src, d += step * ld_dst) {
+        const bool on = r < live && c < cols;
+        cp16z(d, on ? p : src, on ? 16 : 0);
+      }
     }
   } else {
-    for (int i = threadIdx.x; i < rows * cols_pad; i += kThreads) {
+    for (int i = threadIdx.x; i < rows * cols_pad; i += blockDim.x) {
       const int r = i / cols_pad, c = i - r * cols_pad;
       const bool on = r < live && c < cols;
       cp4z(dst + r * ld_dst + c, src + (on ? r * ld_src + c : 0), on ? 4 : 0);
@@ -332,6 +336,97 @@ __global__ void __launch_bounds__(kThreads) gated_delta_front_kernel(SplitArgs a
   }
 }
 
+// The same for head sizes of a multiple of four and TAPS taps: a warp runs one head over kFrontRows consecutive rows, four
+// channels per lane, so that a row's inputs are read once and serve the taps of the rows behind it from registers.
+constexpr int kFrontRows = 4;
+template <int TAPS>
+__global__ void __launch_bounds__(kThreads) gated_delta_front_tile_kernel(SplitArgs a, int n_rows) {
+  pdl_wait();
+  constexpr int keep = TAPS - 1, RT = kFrontRows;
+  const int row0 = blockIdx.x * RT, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int dk = a.dk, dv = a.dv, H = a.heads, ch = 2 * a.kh * dk + H * dv;
+  int slot[RT], back[RT];
+#pragma unroll
+  for (int r = 0; r < RT; ++r) {
+    slot[r] = row0 + r < n_rows ? a.row_slot[row0 + r] : -1;
+    back[r] = row0 + r < n_rows ? a.row_back[row0 + r] : 0;
+  }
+  const int h = blockIdx.y * (kThreads / 32) + warp;
+  if (h < 2 * a.kh + H) {
+    const bool unit = h < 2 * a.kh;
+    const int c0 = unit ? h * dk : 2 * a.kh * dk + (h - 2 * a.kh) * dv, groups = (unit ? dk : dv) / 4;
+    const float* p = a.P + (int64_t)row0 * a.ldp + a.off;
+    for (int g0 = 0; g0 < groups; g0 += 64) {             // a head with unit length has at most 64 groups: one pass
+      float4 v[2][RT];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int g = g0 + lane + 32 * u;
+        if (g >= groups) {
+#pragma unroll
+          for (int r = 0; r < RT; ++r) v[u][r] = make_float4(0.f, 0.f, 0.f, 0.f);
+          continue;
+        }
+        const int c = c0 + 4 * g;
+        float4 x[keep + RT];                              // inputs of rows row0 - keep .. row0 + RT - 1 (of this batch only)
+#pragma unroll
+        for (int j = 0; j < keep + RT; ++j) {
+          const bool in = j < keep ? keep - j <= back[0] : row0 + j - keep < n_rows;
+          x[j] = in ? *reinterpret_cast<const float4*>(p + (int64_t)(j - keep) * a.ldp + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        float w[4][TAPS];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) w[e][k] = a.conv_w[(int64_t)(c + e) * TAPS + k];
+#pragma unroll
+        for (int r = 0; r < RT; ++r) {
+          float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (slot[r] >= 0) {
+#pragma unroll
+            for (int k = keep; k >= 0; --k) {             // oldest first
+              float4 in = x[keep + r - k];
+              if (k > back[r]) {                          // before this batch: the carried inputs
+                const float* st = a.conv_state + ((int64_t)slot[r] * ch + c) * keep + keep - (k - back[r]);
+                in = make_float4(st[0], st[keep], st[2 * keep], st[3 * keep]);
+              }
+              acc.x = fmaf(w[0][keep - k], in.x, acc.x); acc.y = fmaf(w[1][keep - k], in.y, acc.y);
+              acc.z = fmaf(w[2][keep - k], in.z, acc.z); acc.w = fmaf(w[3][keep - k], in.w, acc.w);
+            }
+          }
+          v[u][r] = make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w));
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RT; ++r) {
+        float f = 1.f;
+        if (unit) {
+          float ss = 0.f;
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+            ss += v[u][r].x * v[u][r].x + v[u][r].y * v[u][r].y + v[u][r].z * v[u][r].z + v[u][r].w * v[u][r].w;
+          f = (h < a.kh ? 1.f / sqrtf((float)dk) : 1.f) / sqrtf(warp_sum(ss) + a.unit_eps);
+        }
+        if (slot[r] < 0) continue;
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int g = g0 + lane + 32 * u;
+          if (g < groups)
+            *reinterpret_cast<float4*>(a.C + (int64_t)(row0 + r) * ch + c0 + 4 * g) =
+                make_float4(v[u][r].x * f, v[u][r].y * f, v[u][r].z * f, v[u][r].w * f);
+        }
+      }
+    }
+  }
+  if (blockIdx.y == 0)
+    for (int i = threadIdx.x; i < RT * H; i += kThreads) {
+      const int r = i / H, hh = i - r * H;
+      const int64_t row = row0 + r;
+      if (row >= n_rows || a.row_slot[row] < 0) continue;
+      a.gates[row * 2 * H + hh] = log_decay(a.A_log[hh], a.P[row * a.ldp + a.off_a + hh] + a.dt_bias[hh]);
+      a.gates[row * 2 * H + H + hh] = sigmoid_f(a.P[row * a.ldp + a.off_b + hh]);
+    }
+}
+
 // A, E, U and W of one (piece, value head); the running sums of the log decays replace them in `gates`.
 __global__ void __launch_bounds__(kThreads, 2) gated_delta_piece_kernel(SplitArgs a) {
   pdl_wait();
@@ -383,7 +478,7 @@ __global__ void __launch_bounds__(kThreads, 2) gated_delta_piece_kernel(SplitArg
       for (int i = 0; i < 4; ++i) {
         const float4 k4 = lds4(Ks + (ty + 16 * i) * ldk + c), q4 = lds4(Qs + (ty + 16 * i) * ldk + c);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j <= i; ++j) {            // blocks above the diagonal are not needed
           kk[i][j] = fmaf(k4.x, s4[j].x, kk[i][j]); kk[i][j] = fmaf(k4.y, s4[j].y, kk[i][j]);
           kk[i][j] = fmaf(k4.z, s4[j].z, kk[i][j]); kk[i][j] = fmaf(k4.w, s4[j].w, kk[i][j]);
           qk[i][j] = fmaf(q4.x, s4[j].x, qk[i][j]); qk[i][j] = fmaf(q4.y, s4[j].y, qk[i][j]);
@@ -435,9 +530,10 @@ __global__ void __launch_bounds__(kThreads, 2) gated_delta_piece_kernel(SplitArg
 }
 
 // The pieces of a segment in order, for one value head and a tile of 32 value columns: D = U - W S, S <- G S + (K G / G_t)^T D.
-// STAGES tiles of (W, K) in shared memory.
+// STAGES tiles of (W, K) in shared memory.  The two halves of the CTA split the key channels of W S.
+constexpr int kWalkThreads = 512;
 template <int STAGES>
-__global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs a) {
+__global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   const int col0 = blockIdx.x * kWalkCols, head = blockIdx.y, seg = blockIdx.z;
@@ -455,7 +551,7 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
   __shared__ float gend;
   // the convolution's last inputs become the segment's state (the front end has read the old ones)
   const int keep = a.taps - 1;
-  for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kThreads + tid; c < ch && keep > 0; c += gridDim.x * gridDim.y * kThreads) {
+  for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kWalkThreads + tid; c < ch && keep > 0; c += gridDim.x * gridDim.y * kWalkThreads) {
     float* st = a.conv_state + ((int64_t)slot * ch + c) * keep;
     const int64_t last = (int64_t)a.seg_start[seg] + slen - 1;
     for (int j = 0; j < keep; ++j) {              // ascending: st[j + slen] is still the old input
@@ -464,7 +560,7 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
     }
   }
   float* state = a.state + ((int64_t)slot * H + head) * dv * dk;
-  for (int i = tid; i < kWalkCols * dk4; i += kThreads) {
+  for (int i = tid; i < kWalkCols * dk4; i += kWalkThreads) {
     const int c = i / dk4, k = i - c * dk4;
     S[k * ldc + c] = (col0 + c < dv && k < dk) ? state[(int64_t)(col0 + c) * dk + k] : 0.f;
   }
@@ -479,8 +575,9 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
     cp_commit();
   };
   if (STAGES > 1) stage(0);
-  const int ty = tid >> 4, tx = tid & 15;         // D: rows ty + 16 i, columns 2 tx, 2 tx + 1
-  const int cg = tid & 7, kg = tid >> 3;          // S: columns 4 cg .., key channels 4 (kg + 32 m) ..
+  const int half = tid >> 8, ty = tid >> 4 & 15, tx = tid & 15;      // D: rows ty + 16 i, columns 2 tx, 2 tx + 1
+  const int k_mid = (dk4 / 4 + 1) / 2 * 4, k_lo = half ? k_mid : 0, k_hi = half ? dk4 : k_mid;
+  const int cg = tid & 15, kg = tid >> 4;         // S: columns 2 cg, 2 cg + 1, key channels 4 (kg + 32 m) ..
   for (int i = 0; i < np; ++i) {
     const int64_t r0 = a.sub_start[first + i];
     const int len = a.sub_len[first + i];
@@ -499,17 +596,10 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         const int t = ty + 16 * m, col = col0 + 2 * tx + c;
-        u[m][c] = (t < len && col < dv) ? a.D[((r0 + t) * H + head) * dv + col] : 0.f;
+        u[m][c] = (half == 0 && t < len && col < dv) ? a.D[((r0 + t) * H + head) * dv + col] : 0.f;
       }
     __syncthreads();
-    {   // S at the piece's start, for the read-out
-      float* dst = a.S0 + ((int64_t)(first + i) * H + head) * dk * dv;
-      for (int j = tid; j < dk * kWalkCols; j += kThreads) {
-        const int k = j / kWalkCols, c = j - k * kWalkCols;
-        if (col0 + c < dv) dst[(int64_t)k * dv + col0 + c] = S[k * ldc + c];
-      }
-    }
-    for (int k = 0; k < dk4; k += 4) {
+    for (int k = k_lo; k < k_hi; k += 4) {
       float2 s[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[e] = *reinterpret_cast<const float2*>(S + (k + e) * ldc + 2 * tx);
@@ -522,40 +612,64 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
         u[m][0] = fmaf(-w.w, s[3].x, u[m][0]); u[m][1] = fmaf(-w.w, s[3].y, u[m][1]);
       }
     }
+    if (half) {
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      const int t = ty + 16 * m;
-#pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        const int col = col0 + 2 * tx + c;
-        if (t < len && col < dv) a.D[((r0 + t) * H + head) * dv + col] = u[m][c];
+      for (int m = 0; m < 4; ++m) *reinterpret_cast<float2*>(Ds + (ty + 16 * m) * ldc + 2 * tx) = make_float2(u[m][0], u[m][1]);
+    }
+    __syncthreads();
+    if (half) {     // S at the piece's start, for the read-out
+      float* dst = a.S0 + ((int64_t)(first + i) * H + head) * dk * dv + col0;
+      if (a.vec) {
+        for (int j = tid & 255; j < dk * (kWalkCols / 4); j += 256) {
+          const int k = j >> 3, c = (j & 7) * 4;
+          if (col0 + c < dv) *reinterpret_cast<float4*>(dst + (int64_t)k * dv + c) = lds4(S + k * ldc + c);
+        }
+      } else {
+        for (int j = tid & 255; j < dk * kWalkCols; j += 256) {
+          const int k = j / kWalkCols, c = j - k * kWalkCols;
+          if (col0 + c < dv) dst[(int64_t)k * dv + c] = S[k * ldc + c];
+        }
       }
-      *reinterpret_cast<float2*>(Ds + t * ldc + 2 * tx) = make_float2(u[m][0] * fin[t], u[m][1] * fin[t]);
+    } else {
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        const int t = ty + 16 * m;
+        float2* d2 = reinterpret_cast<float2*>(Ds + t * ldc + 2 * tx);
+        const float2 other = *d2;
+        u[m][0] += other.x; u[m][1] += other.y;
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int col = col0 + 2 * tx + c;
+          if (t < len && col < dv) a.D[((r0 + t) * H + head) * dv + col] = u[m][c];
+        }
+        *d2 = make_float2(u[m][0] * fin[t], u[m][1] * fin[t]);
+      }
     }
     __syncthreads();                              // D complete, every read of the old S done
     const float ge = gend;
     for (int k0 = 4 * kg; k0 < dk4; k0 += 128) {
-      float4 acc[4];
+      float2 acc[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        acc[e] = lds4(S + (k0 + e) * ldc + 4 * cg);
-        acc[e].x *= ge; acc[e].y *= ge; acc[e].z *= ge; acc[e].w *= ge;
+        acc[e] = *reinterpret_cast<const float2*>(S + (k0 + e) * ldc + 2 * cg);
+        acc[e].x *= ge; acc[e].y *= ge;
       }
 #pragma unroll 8
       for (int t = 0; t < kPieceMax; ++t) {
-        const float4 kv = lds4(Kt + t * ldk + k0), d = lds4(Ds + t * ldc + 4 * cg);
-        acc[0].x = fmaf(kv.x, d.x, acc[0].x); acc[0].y = fmaf(kv.x, d.y, acc[0].y); acc[0].z = fmaf(kv.x, d.z, acc[0].z); acc[0].w = fmaf(kv.x, d.w, acc[0].w);
-        acc[1].x = fmaf(kv.y, d.x, acc[1].x); acc[1].y = fmaf(kv.y, d.y, acc[1].y); acc[1].z = fmaf(kv.y, d.z, acc[1].z); acc[1].w = fmaf(kv.y, d.w, acc[1].w);
-        acc[2].x = fmaf(kv.z, d.x, acc[2].x); acc[2].y = fmaf(kv.z, d.y, acc[2].y); acc[2].z = fmaf(kv.z, d.z, acc[2].z); acc[2].w = fmaf(kv.z, d.w, acc[2].w);
-        acc[3].x = fmaf(kv.w, d.x, acc[3].x); acc[3].y = fmaf(kv.w, d.y, acc[3].y); acc[3].z = fmaf(kv.w, d.z, acc[3].z); acc[3].w = fmaf(kv.w, d.w, acc[3].w);
+        const float4 kv = lds4(Kt + t * ldk + k0);
+        const float2 d = *reinterpret_cast<const float2*>(Ds + t * ldc + 2 * cg);
+        acc[0].x = fmaf(kv.x, d.x, acc[0].x); acc[0].y = fmaf(kv.x, d.y, acc[0].y);
+        acc[1].x = fmaf(kv.y, d.x, acc[1].x); acc[1].y = fmaf(kv.y, d.y, acc[1].y);
+        acc[2].x = fmaf(kv.z, d.x, acc[2].x); acc[2].y = fmaf(kv.z, d.y, acc[2].y);
+        acc[3].x = fmaf(kv.w, d.x, acc[3].x); acc[3].y = fmaf(kv.w, d.y, acc[3].y);
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(S + (k0 + e) * ldc + 4 * cg) = acc[e];
+      for (int e = 0; e < 4; ++e) *reinterpret_cast<float2*>(S + (k0 + e) * ldc + 2 * cg) = acc[e];
     }
     __syncthreads();                              // the next piece's copies and gates overwrite what was read here
   }
   cp_wait<0>();
-  for (int i = tid; i < kWalkCols * dk; i += kThreads) {
+  for (int i = tid; i < kWalkCols * dk; i += kWalkThreads) {
     const int c = i / dk, k = i - c * dk;
     if (col0 + c < dv) state[(int64_t)(col0 + c) * dk + k] = S[k * ldc + c];
   }
@@ -564,7 +678,7 @@ __global__ void __launch_bounds__(kThreads, 1) gated_delta_walk_kernel(SplitArgs
 // O = G * (Q S_0) + E D of one (piece, value head), 128 value columns per pass; NORM (dv <= 128): the head norm, the gain and
 // the gate, into `out`; otherwise the raw read-out replaces D.
 template <typename T, bool NORM>
-__global__ void __launch_bounds__(kThreads) gated_delta_read_kernel(SplitArgs a) {
+__global__ void __launch_bounds__(kThreads, 3) gated_delta_read_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   constexpr int kStep = 32, lda = kStep + 4, ldb = kOutCols + 4;
@@ -740,7 +854,12 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
   PRL_CHECK_ARG(((uintptr_t)scratch & 15) == 0, "prl_gated_delta_split: the scratch must be 16-byte aligned");
   a.vec = dk % 4 == 0 && dv % 4 == 0 && (((uintptr_t)C | (uintptr_t)S0 | (uintptr_t)D) & 15) == 0;
   cudaStream_t s = (cudaStream_t)st_;
-  PRL_CUDA(launch_pdl(gated_delta_front_kernel, dim3(n_rows), dim3(kThreads), (size_t)0, s, a));
+  const bool tiled = a.vec && taps >= 2 && taps <= 4 && off % 4 == 0 && ldp % 4 == 0 && ((uintptr_t)P & 15) == 0;
+  const dim3 gf((n_rows + kFrontRows - 1) / kFrontRows, (2 * kh + heads + kThreads / 32 - 1) / (kThreads / 32));
+  if (tiled && taps == 2) PRL_CUDA(launch_pdl(gated_delta_front_tile_kernel<2>, gf, dim3(kThreads), (size_t)0, s, a, n_rows));
+  else if (tiled && taps == 3) PRL_CUDA(launch_pdl(gated_delta_front_tile_kernel<3>, gf, dim3(kThreads), (size_t)0, s, a, n_rows));
+  else if (tiled) PRL_CUDA(launch_pdl(gated_delta_front_tile_kernel<4>, gf, dim3(kThreads), (size_t)0, s, a, n_rows));
+  else PRL_CUDA(launch_pdl(gated_delta_front_kernel, dim3(n_rows), dim3(kThreads), (size_t)0, s, a));
   PRL_LAUNCH_CHECK();
   const int dk4 = (dk + 3) & ~3, ldk = dk4 + 4;
   const size_t sm_piece = ((size_t)2 * kPieceMax * ldk + kPieceMax * (kPieceMax + 4)) * sizeof(float);
@@ -754,10 +873,10 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
   static SmemAttr at_walk[2] = {};
   if (stages == 2) {
     PRL_CUDA(ensure_smem(gated_delta_walk_kernel<2>, (int)sm_walk, at_walk[0]));
-    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<2>, gw, dim3(kThreads), sm_walk, s, a));
+    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<2>, gw, dim3(kWalkThreads), sm_walk, s, a));
   } else {
     PRL_CUDA(ensure_smem(gated_delta_walk_kernel<1>, (int)sm_walk, at_walk[1]));
-    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<1>, gw, dim3(kThreads), sm_walk, s, a));
+    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<1>, gw, dim3(kWalkThreads), sm_walk, s, a));
   }
   PRL_LAUNCH_CHECK();
   const size_t sm_read = (size_t)2 * (kPieceMax * 36 + 32 * (kOutCols + 4)) * sizeof(float);

@@ -1867,15 +1867,11 @@ class HybridEngine(EngineCore):
                                       self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE, R.q.data_ptr(),
                                       self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr(), f32, st))
         sink = vec[w + "mix.sink"].data_ptr() if a.sink else None
-        gated = a.gate and a.gate_per_head
-        _lib.check(lib.prl_attn_any_sink(R.q.data_ptr(), self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr(), a.vdim, f32,
-                                         self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE, seg_start, seg_len,
-                                         seg_pos0.data_ptr(), seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale,
-                                         a.window, 0, a.softcap, sink, 0 if gated else 1,
-                                         R.o.data_ptr() if gated else R.ya.data_ptr(), st))
-        if gated:
-            _lib.check(lib.prl_gate_heads(R.o.data_ptr(), 1, no, P + 4 * (nq + nk + nv), ld, n, a.heads, a.vdim, R.ya.data_ptr(),
-                                          f32, st))
+        gate = P + 4 * (nq + nk + nv) if a.gate and a.gate_per_head else None
+        _lib.check(lib.prl_attn_any_gated(R.q.data_ptr(), self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr(), a.vdim, f32,
+                                          self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE, seg_start, seg_len,
+                                          seg_pos0.data_ptr(), seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale,
+                                          a.window, 0, a.softcap, sink, gate, ld, 1, R.ya.data_ptr(), st))
         return self._mm(R.ya, no, w + "mix.o", W, R.y0, n, split=True)
 
     # ---- the 'one_norm' block: x <- x + (mixer(h) + ff(h)), h = norm(x) --------------------------------------------------
@@ -2102,18 +2098,16 @@ class HybridEngine(EngineCore):
         """Softmax attention from the projections in R.P (AttnDeltaRows) to the gated heads R.ya."""
         lib, st, f32 = self.lib, self._st, int(self.f32)
         seg_start, seg_len, seg_slot, ns = segs
-        P, ld, no = R.P.data_ptr(), C.total, a.heads * a.vdim
+        P, ld = R.P.data_ptr(), C.total
         bt = (self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE)
         kv = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr())
         _lib.check(lib.prl_attn_front(P, ld, 0, C.k, C.v, n, a.heads, a.kv_heads, a.dim, a.vdim, None, None, None, 0, None, None, a.dim,
                                       self.cfg.eps, a.rot_dims, self.rot_freq[i].data_ptr(), self.rot_mag[i], 0, 0, None, None,
                                       row_pos.data_ptr(), R.row_slot.data_ptr(), *bt, R.q.data_ptr(), *kv, f32, st))
         sink = self.zero_sink.data_ptr() if a.unit_sink else None
-        _lib.check(lib.prl_attn_any_sink(R.q.data_ptr(), *kv, a.vdim, f32, *bt, seg_start, seg_len, seg_pos0.data_ptr(), seg_slot, ns,
-                                         max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, 0, a.softcap, sink,
-                                         0 if a.gate else 1, R.o.data_ptr() if a.gate else R.ya.data_ptr(), st))
-        if a.gate:
-            _lib.check(lib.prl_gate_heads(R.o.data_ptr(), 1, no, P + 4 * C.left_g, ld, n, a.heads, a.vdim, R.ya.data_ptr(), f32, st))
+        _lib.check(lib.prl_attn_any_gated(R.q.data_ptr(), *kv, a.vdim, f32, *bt, seg_start, seg_len, seg_pos0.data_ptr(), seg_slot, ns,
+                                          max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, 0, a.softcap, sink,
+                                          P + 4 * C.left_g if a.gate else None, ld, 1, R.ya.data_ptr(), st))
 
     def _gated_delta_cell(self, R, n, i, g, p, segs, max_q, P, ld, off, off_b, off_a, off_g) -> None:
         """From the projections in P (rows ld apart: q | k | v at `off`, step, decay and gate columns) to the cell's normed and
