@@ -434,6 +434,15 @@ int prl_paged_attn_prefill_tc(const void* q_bf16 /*[q_rows,n_q,128]*/, int32_t q
                               const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs, int32_t max_q_len,
                               int32_t n_q, int32_t n_kv, int32_t head_dim, int32_t page_size, float sm_scale,
                               void* out_bf16 /*[rows,n_q*128]*/, prl_stream_t stream);
+/* with a sliding window (0: none), a sink logit per head [n_q] that joins the denominator only and a gate per head and row: the
+ * head's output times sigmoid(gate[row * ld_gate + head]) (NULL: none) */
+int prl_paged_attn_prefill_tc_gated(const void* q_bf16 /*[q_rows,n_q,128]*/, int32_t q_rows, const void* kv_cache_bf16,
+                              int64_t n_pages, int32_t n_layers, int32_t layer, const int32_t* block_table,
+                              int32_t max_blocks, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                              const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs, int32_t max_q_len,
+                              int32_t n_q, int32_t n_kv, int32_t head_dim, int32_t page_size, float sm_scale,
+                              int32_t window, const float* sink,
+                              const float* gate, int64_t ld_gate, void* out_bf16 /*[rows,n_q*128]*/, prl_stream_t stream);
 /* Learner attention (hot path 2): block-diagonal causal attention over ONE packed row and its backward -- the
  * flash-attn varlen call the reference makes through HF with packed position_ids
  * (pipelinerl/finetune/rl/__init__.py:204 forward, finetune_loop.py:716-725 backward; conf/finetune/base.yaml:12-13,64).

@@ -3,8 +3,8 @@
 // scores, grouped key/value heads, output in bf16 or fp32).
 //
 // CTA = 4 warps = 64 consecutive query rows of one (segment, query head); a warp owns 16 rows.  Keys are walked in
-// tiles of 64 at absolute multiples of 64 (so the order of summation does not depend on how a prompt was cut), two
-// buffers deep; tiles that no row of the CTA can see -- between the kept first tokens and the window -- are skipped.  Per tile: K and V
+// tiles of 64 at absolute multiples of 64 (so the order of summation does not depend on how a prompt was cut); tiles
+// that no row of the CTA can see -- between the kept first tokens and the window -- are skipped.  Per tile: K and V
 // rows come from the paged pools by cp.async (16 bytes per copy, zero fill past the sequence's end), S = Q K^T by
 // mma.sync m16n8k16 (bf16 in, fp32 out) with operands read by ldmatrix from padded, conflict-free rows; scale, cap and
 // mask in fp32 registers; an fp32 online softmax per row (the four lanes of a row exchange by shuffles); P rounded to
@@ -63,8 +63,8 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(const bf16* __restrict__ 
   constexpr int LDV = DV + kPadH, CHV = DV / 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* Qs = reinterpret_cast<bf16*>(smem_raw);      // [64][LD]
-  bf16* tiles = Qs + kRows * LD;                     // two buffers of K [64][LD] | V [64][LDV]
-  const int tile_halves = kKeys * (LD + LDV);
+  bf16* Ks = Qs + kRows * LD;                        // [64][LD]
+  bf16* Vs = Ks + kKeys * LD;                        // [64][LDV]
   const int seg = blockIdx.z, h = blockIdx.y;
   const int len = seg_len[seg];
   const int i0 = blockIdx.x * kRows;
@@ -101,10 +101,9 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(const bf16* __restrict__ 
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
 
-  // K and V rows of the tile at k0 into a buffer; tile t + 1 arrives while tile t is worked on
-  auto stage = [&](int k0, int buf) {
-    bf16* Ks = tiles + buf * tile_halves;
-    bf16* Vs = Ks + kKeys * LD;
+  for (int k0 = 0; k0 <= last_pos; k0 += kKeys) {
+    if (k0 >= sink_end && k0 + kKeys <= win_lo) continue;              // CTA-uniform: between the kept tokens and the window
+    __syncthreads();                                                   // every warp is done with the previous tile
     for (int c = tid; c < kKeys * CH; c += 128) {
       const int j = c / CH, cc = c - j * CH;
       const int kt = k0 + j;
@@ -121,23 +120,11 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(const bf16* __restrict__ 
       const int64_t at = (((int64_t)bt[kk / page_size] * G + g) * page_size + kk % page_size) * DV + cc * 8;
       cp16(Vs + j * LDV + cc * 8, v_pool + at, ok ? 16 : 0);
     }
-  };
-  // tiles no row of the CTA can see -- between the kept first tokens and the window -- are skipped
-  auto next_tile = [&](int k0) { return (k0 >= sink_end && k0 + kKeys <= win_lo) ? win_lo / kKeys * kKeys : k0; };
-  int buf = 0, k0 = next_tile(0);
-  stage(k0, 0);
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  for (int kn; k0 <= last_pos; k0 = kn, buf ^= 1) {
-    kn = next_tile(k0 + kKeys);
-    if (kn <= last_pos) stage(kn, buf ^ 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const bf16* Ks = tiles + buf * tile_halves;
-    const bf16* Vs = Ks + kKeys * LD;
-    auto work = [&]() {
-    if (w_first > last_pos || k0 > w_last) return;                     // warp-uniform: no rows, or the tile is in the future
-    if (k0 + kKeys <= w_lo && k0 >= keep_first) return;                // hidden from every row of the warp
+    if (w_first > last_pos || k0 > w_last) continue;                   // warp-uniform: no rows, or the tile is in the future
+    if (k0 + kKeys <= w_lo && k0 >= keep_first) continue;              // hidden from every row of the warp
     // ---- S = Q K^T (16 x 64 per warp)
     float s[kKeys / 8][4];
 #pragma unroll
@@ -213,9 +200,6 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(const bf16* __restrict__ 
         mma16816(o[2 * j + 1], a, b[2], b[3]);
       }
     }
-    };
-    work();
-    __syncthreads();                                                   // every warp is done with the buffer refilled next
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
@@ -248,7 +232,7 @@ int launch_mma(const void* q, const void* kp, const void* vp, const int32_t* bt,
                const int32_t* ss, const int32_t* sl, const int32_t* sp, const int32_t* sslot, int n_seg, int max_q, int H, int G,
                int dim, float scale, int window, int keep_first, float softcap, const float* sink, const float* gate, int64_t ldg, void* out,
                cudaStream_t st) {
-  const size_t smem = ((size_t)(kRows + 2 * kKeys) * (dim + kPadH) + (size_t)2 * kKeys * (DV + kPadH)) * sizeof(bf16);
+  const size_t smem = ((size_t)(kRows + kKeys) * (dim + kPadH) + (size_t)kKeys * (DV + kPadH)) * sizeof(bf16);
   static SmemAttr attr = {};
   if (smem > 48 * 1024) PRL_CUDA(ensure_smem(attn_mma_kernel<D, DV, OUT_BF16>, (int)smem, attr));
   dim3 grid((max_q + kRows - 1) / kRows, H, n_seg);

@@ -50,6 +50,11 @@ struct TcPrefillParams {
   // sequence z covers rows [seq_q_start[z], seq_q_start[z] + seq_q_len[z]) and its keys are those same rows
   int col_k, col_v;              // element column of K / V head 0
   float* lse;                    // [rows, n_q] log2-domain log-sum-exp of the scaled scores (may be NULL)
+  // options of the paged form (generation 2 only)
+  int window;                    // > 0: a query sees only the last `window` positions, itself included
+  const float* sink;             // [n_q] a logit per head in the softmax denominator (no key, no value), or NULL
+  const float* gate;             // [rows][ld_gate] logits: a head's output times sigmoid(gate[row * ld_gate + head]), or NULL
+  int64_t ld_gate;
   long long* timing;             // measurement only (prl_attn_debug_timing): per-phase cycle sums of one CTA, else NULL
 };
 
@@ -381,7 +386,9 @@ attn_fwd_v2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
   const int n_valid = t0 >= q_len ? 0 : ((q_len - t0) < p.nq ? (q_len - t0) : p.nq);
   const int pair_rows = ((qtile | 1) + 1) * p.nq;
   const int kv_end = pos0 + (pair_rows < q_len ? pair_rows : q_len);
-  const int n_it = (kv_end + kKeys - 1) / kKeys;
+  // with a window the walk starts at the first step the pair's first row still sees
+  const int it0 = (!kContig && p.window > 0) ? max(0, pos0 + (qtile & ~1) * p.nq - p.window + 1) / kKeys : 0;
+  const int n_it = (kv_end + kKeys - 1) / kKeys - it0;
   const int last_page = (kv_end - 1) / kPageT;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -416,7 +423,7 @@ attn_fwd_v2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         const uint32_t ph = (uint32_t)((it / kSt) & 1);
         ptx::mbar_wait(empty_bar + 8u * (uint32_t)s, ph ^ 1u);
         ptx::mbar_arrive_expect_tx(full_bar + 8u * (uint32_t)s, (uint32_t)(2 * kTile16K));
-        int pg = 2 * it + (int)rank;
+        int pg = 2 * (it + it0) + (int)rank;
         if (pg > last_page) pg = last_page;
         int row, c0;
         if (kContig) {
@@ -524,11 +531,16 @@ attn_fwd_v2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         for (int e = 0; e < 128; ++e) sv[e] = __uint_as_float(su[e]);
       }
       const long long c2 = clock64();
-      if (i * kKeys + kKeys - 1 > pos_first) {              // some (row, key) of this step is causally masked
-        const int key0 = i * kKeys;
+      const int key0 = (i + it0) * kKeys;
+      if (key0 + kKeys - 1 > pos_first) {                   // some (row, key) of this step is causally masked
 #pragma unroll
         for (int e = 0; e < 128; ++e)
           if (key0 + e > qpos) sv[e] = -INFINITY;
+      }
+      if (!kContig && p.window > 0 && key0 <= pos_first + p.nq - 1 - p.window) {   // ... or has left some row's window
+#pragma unroll
+        for (int e = 0; e < 128; ++e)
+          if (key0 + e <= qpos - p.window) sv[e] = -INFINITY;
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four independent chains of 3-input maxima (FMNMX3):
 #pragma unroll                                                       // 64 instructions for the 128 scores of a row
@@ -540,7 +552,9 @@ attn_fwd_v2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       const float m_new = mx * p.scale_log2;                // scale > 0: max commutes with the scaling
       const long long c3 = clock64();
       if (j == 0) {
-        m_ref = (m_new == -INFINITY) ? 0.f : m_new;
+        // nothing visible yet: without a window the reference is free (key 0 comes first); with one it stays far below
+        // every score, so that the first visible step sets it (the rescale then multiplies an O of zeros by zero)
+        m_ref = (m_new == -INFINITY) ? ((!kContig && p.window > 0) ? -1e30f : 0.f) : m_new;
       } else {
         const bool need = m_new > m_ref + 8.f;              // rows of a warp decide together (TMEM ops are warp-wide)
         if (__any_sync(0xffffffffu, need)) {
@@ -609,12 +623,17 @@ attn_fwd_v2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       if (n1 > 0) { const float2 x = xchg[m]; m1 = x.x; l1 = x.y; }
       const bool use1 = n1 > 0 && l1 > 0.f;
       const bool use0 = l_run > 0.f;
-      const float m_all = use0 ? (use1 ? fmaxf(m_ref, m1) : m_ref) : m1;
+      float m_all = use0 ? (use1 ? fmaxf(m_ref, m1) : m_ref) : m1;
+      const float sk = (!kContig && p.sink) ? p.sink[kvh * p.R + r] * 1.4426950408889634f : -INFINITY;
+      if (!kContig) m_all = fmaxf(m_all, sk);
       const float f0 = use0 ? ex2(m_ref - m_all) : 0.f;
       const float f1 = use1 ? ex2(m1 - m_all) : 0.f;
-      const float l_tot = f0 * l_run + f1 * l1;
-      const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+      float l_tot = f0 * l_run + f1 * l1;
+      if (!kContig) l_tot += ex2(sk - m_all);               // no sink: exp2(-inf) = 0
       const bool valid = qi < n_valid && qi < p.nq;
+      float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+      if (!kContig && p.gate && valid)
+        inv *= 1.f / (1.f + expf(-p.gate[(int64_t)(row0 + qi) * p.ld_gate + kvh * p.R + r]));
       __nv_bfloat16* dst = p.out + ((int64_t)(row0 + qi) * p.n_q + (kvh * p.R + r)) * kDT;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
@@ -670,12 +689,14 @@ extern "C" int prl_attn_set_prefill_generation(int32_t gen) {
   return PRL_OK;
 }
 
-extern "C" int prl_paged_attn_prefill_tc(const void* q, int32_t q_rows, const void* kv_cache, int64_t n_pages,
-                                         int32_t n_layers, int32_t layer, const int32_t* block_table,
-                                         int32_t max_blocks, const int32_t* seq_q_start, const int32_t* seq_q_len,
-                                         const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs,
-                                         int32_t max_q_len, int32_t n_q, int32_t n_kv, int32_t head_dim,
-                                         int32_t page_size, float sm_scale, void* out_bf16, prl_stream_t stream_) {
+static int prefill_tc_impl(const void* q, int32_t q_rows, const void* kv_cache, int64_t n_pages,
+                           int32_t n_layers, int32_t layer, const int32_t* block_table,
+                           int32_t max_blocks, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                           const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs,
+                           int32_t max_q_len, int32_t n_q, int32_t n_kv, int32_t head_dim,
+                           int32_t page_size, float sm_scale, int32_t window, const float* sink, const float* gate,
+                           int64_t ld_gate, void* out_bf16, prl_stream_t stream_) {
+  PRL_CHECK_ARG(window >= 0 && (!gate || ld_gate >= n_q), "prl_paged_attn_prefill_tc: bad window or gate");
   PRL_CHECK_ARG(q && kv_cache && block_table && seq_q_start && seq_q_len && seq_pos0 && seq_slot && out_bf16,
                 "prl_paged_attn_prefill_tc: NULL argument");
   PRL_CHECK_ARG(head_dim == kDT && page_size == kPageT, "prl_paged_attn_prefill_tc: head_dim must be 128 and page_size 64");
@@ -691,6 +712,7 @@ extern "C" int prl_paged_attn_prefill_tc(const void* q, int32_t q_rows, const vo
   p.nq = 128 / p.R;
   p.n_pages = n_pages; p.layer = layer; p.scale_log2 = sm_scale * 1.4426950408889634f;
   p.col_k = p.col_v = 0; p.lse = nullptr; p.timing = nullptr;
+  p.window = window; p.sink = sink; p.gate = gate; p.ld_gate = ld_gate;
   CUtensorMap tq, tkv;
   int rc = make_tmap_2d_bf16(&tkv, kv_cache, kDT, (uint64_t)total_rows, kDT * 2, 64, kPageT);
   if (rc) return rc;
@@ -700,7 +722,7 @@ extern "C" int prl_paged_attn_prefill_tc(const void* q, int32_t q_rows, const vo
   const int smem = 2 * kTile16K + 2 * kStageBytesT + 4 * kTile16K + 1024 + 8 * 20 + 2 * 128 * 4 + 16;
   static SmemAttr smem_attr = {};
   dim3 grid((unsigned)(((max_q_len + p.nq - 1) / p.nq + 1) & ~1), (unsigned)n_kv, (unsigned)n_seqs);  // pairs of q tiles
-  if (g_prefill_generation == 2) {      // ping-pong softmax groups, P and O in TMEM (see attn_fwd_v2_kernel)
+  if (g_prefill_generation == 2 || window || sink || gate) {      // ping-pong softmax groups, P and O in TMEM (see attn_fwd_v2_kernel)
     static SmemAttr smem_attr2 = {};
     PRL_CUDA(ensure_smem(attn_fwd_v2_kernel<false>, smem, smem_attr2));
     attn_fwd_v2_kernel<false><<<grid, kThreadsT, (size_t)smem, (cudaStream_t)stream_>>>(tq, tkv, p);
@@ -710,6 +732,31 @@ extern "C" int prl_paged_attn_prefill_tc(const void* q, int32_t q_rows, const vo
   }
   PRL_LAUNCH_CHECK();
   return PRL_OK;
+}
+
+
+extern "C" int prl_paged_attn_prefill_tc(const void* q, int32_t q_rows, const void* kv_cache, int64_t n_pages,
+                                         int32_t n_layers, int32_t layer, const int32_t* block_table,
+                                         int32_t max_blocks, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                                         const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs,
+                                         int32_t max_q_len, int32_t n_q, int32_t n_kv, int32_t head_dim,
+                                         int32_t page_size, float sm_scale, void* out_bf16, prl_stream_t stream_) {
+  return prefill_tc_impl(q, q_rows, kv_cache, n_pages, n_layers, layer, block_table, max_blocks, seq_q_start, seq_q_len, seq_pos0,
+                         seq_slot, n_seqs, max_q_len, n_q, n_kv, head_dim, page_size, sm_scale, 0, nullptr, nullptr, 0, out_bf16, stream_);
+}
+
+// ... with a sliding window (0: none), a sink logit per head in the softmax denominator (NULL: none) and one sigmoid gate per
+// head and row (NULL: none)
+extern "C" int prl_paged_attn_prefill_tc_gated(const void* q, int32_t q_rows, const void* kv_cache, int64_t n_pages,
+                                               int32_t n_layers, int32_t layer, const int32_t* block_table,
+                                               int32_t max_blocks, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                                               const int32_t* seq_pos0, const int32_t* seq_slot, int32_t n_seqs,
+                                               int32_t max_q_len, int32_t n_q, int32_t n_kv, int32_t head_dim,
+                                               int32_t page_size, float sm_scale, int32_t window, const float* sink,
+                                               const float* gate, int64_t ld_gate, void* out_bf16, prl_stream_t stream_) {
+  return prefill_tc_impl(q, q_rows, kv_cache, n_pages, n_layers, layer, block_table, max_blocks, seq_q_start, seq_q_len, seq_pos0,
+                         seq_slot, n_seqs, max_q_len, n_q, n_kv, head_dim, page_size, sm_scale, window, sink, gate, ld_gate, out_bf16,
+                         stream_);
 }
 
 
@@ -748,6 +795,7 @@ extern "C" int prl_attn_varlen_fwd(const void* qkv, int64_t qkv_stride, int32_t 
   p.max_blocks = 0; p.n_q = n_q; p.n_kv = n_kv; p.R = n_q / n_kv; p.nq = 128 / p.R;
   p.n_pages = 0; p.layer = 0; p.scale_log2 = sm_scale * 1.4426950408889634f;
   p.col_k = n_q * kDT; p.col_v = (n_q + n_kv) * kDT; p.lse = lse; p.timing = g_fwd_timing;
+  p.window = 0; p.sink = nullptr; p.gate = nullptr; p.ld_gate = 0;
   CUtensorMap tq, tkv;
   int rc = make_tmap_2d_bf16(&tkv, qkv, (uint64_t)(n_q + 2 * n_kv) * kDT, (uint64_t)T, (uint64_t)qkv_stride * 2, 64, kPageT);
   if (rc) return rc;
@@ -796,6 +844,7 @@ extern "C" int prl_attn_varlen_fwd_kv(const void* q, int64_t q_stride, int32_t T
   p.max_blocks = 0; p.n_q = n_q; p.n_kv = n_kv; p.R = n_q / n_kv; p.nq = 128 / p.R;
   p.n_pages = 0; p.layer = 0; p.scale_log2 = sm_scale * 1.4426950408889634f;
   p.col_k = 0; p.col_v = n_kv * kDT; p.lse = lse; p.timing = nullptr;
+  p.window = 0; p.sink = nullptr; p.gate = nullptr; p.ld_gate = 0;
   CUtensorMap tq, tkv;
   int rc = make_tmap_2d_bf16(&tkv, kv, (uint64_t)(2 * n_kv) * kDT, (uint64_t)Tkv, (uint64_t)kv_stride * 2, 64, kPageT);
   if (rc) return rc;

@@ -22,9 +22,10 @@
 //        S_end = G_end S_0 + (K * (G_end / G))^T D
 //    so that D = U - W S_0 with U = (I + A)^(-1) (b * V), W = (I + A)^(-1) (b * G * K).  Four kernels: the front end
 //    (convolution, unit vectors, gates); per piece and head A, E and, by forward substitution with one column per thread, U
-//    and W; the walk over the pieces of a segment, which only carries S (two products per piece, a tile of 32 value columns per
+//    and W; the walk over the pieces of a segment, which only carries S (two products per piece, a tile of 16 value columns per
 //    CTA) and leaves D and every piece's S_0; the read-out, per piece and head again, with the head norm and the gate.  All
-//    products are register-blocked fp32 FMAs.  Decays enter as differences of running sums of logarithms, which are never
+//    products are register-blocked fp32 FMAs (a warp's shared-memory reads cost by the bytes its lanes receive, broadcast or
+//    not, so the tiles are as square and as large as the work leaves threads for).  Decays enter as differences of running sums of logarithms, which are never
 //    positive, so nothing overflows.
 #include "prl_common.cuh"
 #include <math.h>
@@ -34,7 +35,7 @@ namespace {
 
 constexpr int kThreads = 256;
 constexpr int kPieceMax = 64;      // tokens per piece
-constexpr int kWalkCols = 32;      // value columns per CTA of the walk
+constexpr int kWalkCols = 16;      // value columns per CTA of the walk
 constexpr int kOutCols = 128;      // value columns per pass of the read-out
 
 template <typename T> __device__ __forceinline__ void put(T* p, float v);
@@ -428,18 +429,39 @@ __global__ void __launch_bounds__(kThreads) gated_delta_front_tile_kernel(SplitA
 }
 
 // A, E, U and W of one (piece, value head); the running sums of the log decays replace them in `gates`.
-__global__ void __launch_bounds__(kThreads, 2) gated_delta_piece_kernel(SplitArgs a) {
+// Row s of two columns is final: take its part out of the rows behind it.  At[s][t] = A_ts (zero at and above the diagonal).
+constexpr int kPieceLd = kPieceMax + 4;
+template <int s>
+__device__ __forceinline__ void substitute(float (&x)[2][kPieceMax], const float* At) {
+  if constexpr (s < kPieceMax - 1) {
+#pragma unroll
+    for (int t4 = (s + 1) / 4 * 4; t4 < kPieceMax; t4 += 4) {
+      const float4 c4 = lds4(At + s * kPieceLd + t4);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        if (t4 > s) x[u][t4] = fmaf(-c4.x, x[u][s], x[u][t4]);
+        if (t4 + 1 > s) x[u][t4 + 1] = fmaf(-c4.y, x[u][s], x[u][t4 + 1]);
+        if (t4 + 2 > s) x[u][t4 + 2] = fmaf(-c4.z, x[u][s], x[u][t4 + 2]);
+        if (t4 + 3 > s) x[u][t4 + 3] = fmaf(-c4.w, x[u][s], x[u][t4 + 3]);
+      }
+    }
+    substitute<s + 1>(x, At);
+  }
+}
+
+constexpr int kPieceThreads = 128;
+__global__ void __launch_bounds__(kPieceThreads, 2) gated_delta_piece_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   const int piece = blockIdx.x, head = blockIdx.y, len = a.sub_len[piece];
   const int64_t row0 = a.sub_start[piece];
   const int dk = a.dk, dv = a.dv, H = a.heads, tid = threadIdx.x;
   const int dk4 = (dk + 3) & ~3, ldk = dk4 + 4, ch = 2 * a.kh * dk + H * dv, kvh = head / (H / a.kh);
-  constexpr int ldA = kPieceMax + 4;
+  constexpr int ldA = kPieceLd;
   float* Ks = sm;                                 // [64][ldk]
   float* Qs = Ks + kPieceMax * ldk;               // [64][ldk]
   float* At = Qs + kPieceMax * ldk;               // [64][ldA]: At[s][t] = A_ts
-  __shared__ float cum[kPieceMax], beta[kPieceMax];
+  __shared__ float cum[kPieceMax], beta[kPieceMax], bg[kPieceMax];      // running log decay, step, step times decay
   const float* C = a.C + row0 * ch;
   stage_tile(Ks, ldk, C + a.kh * dk + kvh * dk, ch, kPieceMax, len, dk, dk4, a.vec);
   stage_tile(Qs, ldk, C + kvh * dk, ch, kPieceMax, len, dk, dk4, a.vec);
@@ -458,82 +480,87 @@ __global__ void __launch_bounds__(kThreads, 2) gated_delta_piece_kernel(SplitArg
     cum[t0 + 1] = s;
     beta[t0] = t0 < len ? gr[(int64_t)t0 * 2 * H + H] : 0.f;
     beta[t0 + 1] = t0 + 1 < len ? gr[(int64_t)(t0 + 1) * 2 * H + H] : 0.f;
+    bg[t0] = beta[t0] * expf(cum[t0]);
+    bg[t0 + 1] = beta[t0 + 1] * expf(cum[t0 + 1]);
     if (t0 < len) gr[(int64_t)t0 * 2 * H] = s - l1;
     if (t0 + 1 < len) gr[(int64_t)(t0 + 1) * 2 * H] = s;
   }
   cp_wait<0>();
   __syncthreads();
-  {
-    const int ty = tid >> 4, tx = tid & 15;
-    float kk[4][4], qk[4][4];
+  {   // one half of the CTA forms K K^T, the other Q K^T, 8 x 8 entries per thread
+    const bool query = tid >= 64;
+    const int ty = tid >> 3 & 7, tx = tid & 7;
+    const float* As = query ? Qs : Ks;
+    float acc[8][8];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) { kk[i][j] = 0.f; qk[i][j] = 0.f; }
+      for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
     for (int c = 0; c < dk4; c += 4) {
-      float4 s4[4];
+      float4 s4[8];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) s4[j] = lds4(Ks + (tx + 16 * j) * ldk + c);
+      for (int j = 0; j < 8; ++j) s4[j] = lds4(Ks + (tx + 8 * j) * ldk + c);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float4 k4 = lds4(Ks + (ty + 16 * i) * ldk + c), q4 = lds4(Qs + (ty + 16 * i) * ldk + c);
+      for (int i = 0; i < 8; ++i) {
+        const float4 a4 = lds4(As + (ty + 8 * i) * ldk + c);
 #pragma unroll
         for (int j = 0; j <= i; ++j) {            // blocks above the diagonal are not needed
-          kk[i][j] = fmaf(k4.x, s4[j].x, kk[i][j]); kk[i][j] = fmaf(k4.y, s4[j].y, kk[i][j]);
-          kk[i][j] = fmaf(k4.z, s4[j].z, kk[i][j]); kk[i][j] = fmaf(k4.w, s4[j].w, kk[i][j]);
-          qk[i][j] = fmaf(q4.x, s4[j].x, qk[i][j]); qk[i][j] = fmaf(q4.y, s4[j].y, qk[i][j]);
-          qk[i][j] = fmaf(q4.z, s4[j].z, qk[i][j]); qk[i][j] = fmaf(q4.w, s4[j].w, qk[i][j]);
+          acc[i][j] = fmaf(a4.x, s4[j].x, acc[i][j]); acc[i][j] = fmaf(a4.y, s4[j].y, acc[i][j]);
+          acc[i][j] = fmaf(a4.z, s4[j].z, acc[i][j]); acc[i][j] = fmaf(a4.w, s4[j].w, acc[i][j]);
         }
       }
     }
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = ty + 16 * i;
+    for (int i = 0; i < 8; ++i) {
+      const int t = ty + 8 * i;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int s = tx + 16 * j;
-        const float e = s <= t ? expf(cum[t] - cum[s]) : 0.f;
-        At[s * ldA + t] = s < t ? beta[t] * e * kk[i][j] : 0.f;       // rows past the piece have beta = 0
-        if (t < len) a.E[((row0 + t) * H + head) * kPieceMax + s] = s < len ? e * qk[i][j] : 0.f;
+      for (int j = 0; j < 8; ++j) {
+        const int s = tx + 8 * j;
+        const float e = s <= t ? expf(cum[t] - cum[s]) * acc[i][j] : 0.f;
+        if (!query) At[s * ldA + t] = s < t ? beta[t] * e : 0.f;      // rows past the piece have beta = 0
+        else if (t < len) a.E[((row0 + t) * H + head) * kPieceMax + s] = s < len ? e : 0.f;
       }
     }
   }
   __syncthreads();
-  // forward substitution, one column of [b V | b G K] per thread, all 64 rows in registers
+  // forward substitution, two columns of [b V | b G K] per thread, all 64 rows in registers
   const float* V = C + 2 * a.kh * dk + head * dv;
-  for (int col = tid; col < dv + dk; col += kThreads) {
-    float x[kPieceMax];
-    if (col < dv) {
+  for (int base = tid; base < dv + dk; base += 2 * kPieceThreads) {
+    float x[2][kPieceMax];
 #pragma unroll
-      for (int t = 0; t < kPieceMax; ++t) x[t] = t < len ? beta[t] * V[(int64_t)t * ch + col] : 0.f;
-    } else {
+    for (int u = 0; u < 2; ++u) {
+      const int col = base + u * kPieceThreads;
+      if (col < dv) {
 #pragma unroll
-      for (int t = 0; t < kPieceMax; ++t) x[t] = beta[t] * expf(cum[t]) * Ks[t * ldk + col - dv];
-    }
+        for (int t = 0; t < kPieceMax; ++t) x[u][t] = t < len ? V[(int64_t)t * ch + col] : 0.f;
 #pragma unroll
-    for (int s = 0; s < kPieceMax - 1; ++s) {
+        for (int t = 0; t < kPieceMax; ++t) x[u][t] *= beta[t];
+      } else if (col < dv + dk) {
 #pragma unroll
-      for (int t4 = (s + 1) / 4 * 4; t4 < kPieceMax; t4 += 4) {
-        const float4 c4 = lds4(At + s * ldA + t4);                    // zero at and above the diagonal
-        if (t4 > s) x[t4] = fmaf(-c4.x, x[s], x[t4]);
-        if (t4 + 1 > s) x[t4 + 1] = fmaf(-c4.y, x[s], x[t4 + 1]);
-        if (t4 + 2 > s) x[t4 + 2] = fmaf(-c4.z, x[s], x[t4 + 2]);
-        if (t4 + 3 > s) x[t4 + 3] = fmaf(-c4.w, x[s], x[t4 + 3]);
+        for (int t = 0; t < kPieceMax; ++t) x[u][t] = bg[t] * Ks[t * ldk + col - dv];
+      } else {
+#pragma unroll
+        for (int t = 0; t < kPieceMax; ++t) x[u][t] = 0.f;
       }
     }
-    float* dst = col < dv ? a.D + (row0 * H + head) * dv + col : a.W + (row0 * H + head) * dk + col - dv;
-    const int64_t step = (int64_t)H * (col < dv ? dv : dk);
+    substitute<0>(x, At);
 #pragma unroll
-    for (int t = 0; t < kPieceMax; ++t)
-      if (t < len) dst[t * step] = x[t];
+    for (int u = 0; u < 2; ++u) {
+      const int col = base + u * kPieceThreads;
+      if (col >= dv + dk) continue;
+      float* dst = col < dv ? a.D + (row0 * H + head) * dv + col : a.W + (row0 * H + head) * dk + col - dv;
+      const int64_t step = (int64_t)H * (col < dv ? dv : dk);
+#pragma unroll
+      for (int t = 0; t < kPieceMax; ++t)
+        if (t < len) dst[t * step] = x[u][t];
+    }
   }
 }
 
-// The pieces of a segment in order, for one value head and a tile of 32 value columns: D = U - W S, S <- G S + (K G / G_t)^T D.
-// STAGES tiles of (W, K) in shared memory.  The two halves of the CTA split the key channels of W S.
-constexpr int kWalkThreads = 512;
+// The pieces of a segment in order, for one value head and a tile of 16 value columns: D = U - W S, S <- G S + (K G / G_t)^T D.
+// STAGES tiles of (W, K) in shared memory: two when a CTA has its SM alone, one when two CTAs share it.
 template <int STAGES>
-__global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(SplitArgs a) {
+__global__ void __launch_bounds__(kThreads, 2) gated_delta_walk_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   const int col0 = blockIdx.x * kWalkCols, head = blockIdx.y, seg = blockIdx.z;
@@ -547,11 +574,12 @@ __global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(Split
   float* bufs = sm;                               // [STAGES]: W [64][ldk] | K [64][ldk]
   float* S = bufs + STAGES * tile;                // [dk4][ldc]
   float* Ds = S + dk4 * ldc;                      // [64][ldc]: D times G_end / G_t
+  float* red = Ds + kPieceMax * ldc;              // partial sums: [4][64][16] of W S, then [dk4][16] of the update
   __shared__ float fin[kPieceMax];                // G_end / G_t
   __shared__ float gend;
   // the convolution's last inputs become the segment's state (the front end has read the old ones)
   const int keep = a.taps - 1;
-  for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kWalkThreads + tid; c < ch && keep > 0; c += gridDim.x * gridDim.y * kWalkThreads) {
+  for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kThreads + tid; c < ch && keep > 0; c += gridDim.x * gridDim.y * kThreads) {
     float* st = a.conv_state + ((int64_t)slot * ch + c) * keep;
     const int64_t last = (int64_t)a.seg_start[seg] + slen - 1;
     for (int j = 0; j < keep; ++j) {              // ascending: st[j + slen] is still the old input
@@ -560,7 +588,7 @@ __global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(Split
     }
   }
   float* state = a.state + ((int64_t)slot * H + head) * dv * dk;
-  for (int i = tid; i < kWalkCols * dk4; i += kWalkThreads) {
+  for (int i = tid; i < kWalkCols * dk4; i += kThreads) {
     const int c = i / dk4, k = i - c * dk4;
     S[k * ldc + c] = (col0 + c < dv && k < dk) ? state[(int64_t)(col0 + c) * dk + k] : 0.f;
   }
@@ -575,9 +603,15 @@ __global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(Split
     cp_commit();
   };
   if (STAGES > 1) stage(0);
-  const int half = tid >> 8, ty = tid >> 4 & 15, tx = tid & 15;      // D: rows ty + 16 i, columns 2 tx, 2 tx + 1
-  const int k_mid = (dk4 / 4 + 1) / 2 * 4, k_lo = half ? k_mid : 0, k_hi = half ? dk4 : k_mid;
-  const int cg = tid & 15, kg = tid >> 4;         // S: columns 2 cg, 2 cg + 1, key channels 4 (kg + 32 m) ..
+  const int cg = tid & 3;                         // columns 4 cg .. 4 cg + 3 in every role of the thread
+  // W S: two warps per quarter of the key channels, rows rg + 16 m
+  const int slice = tid >> 6, rg = tid >> 2 & 15, k_len = (dk4 + 15) / 16 * 4;
+  const int k_lo = min(dk4, slice * k_len), k_hi = min(dk4, k_lo + k_len);
+  // D: row dt
+  const int dt = tid >> 2;
+  // update: half of the rows, key channels 4 kg .. and 128 + 4 kg ..
+  const int half = tid >> 7, kg = tid >> 2 & 31;
+  const bool vec_col = a.vec && col0 + 4 * cg < dv;
   for (int i = 0; i < np; ++i) {
     const int64_t r0 = a.sub_start[first + i];
     const int len = a.sub_len[first + i];
@@ -590,86 +624,110 @@ __global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(Split
       fin[tid] = tid < len ? expf(end - gr[(int64_t)tid * 2 * H]) : 0.f;
       if (tid == 0) gend = expf(end);
     }
-    float u[4][2];
-#pragma unroll
-    for (int m = 0; m < 4; ++m)
-#pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        const int t = ty + 16 * m, col = col0 + 2 * tx + c;
-        u[m][c] = (half == 0 && t < len && col < dv) ? a.D[((r0 + t) * H + head) * dv + col] : 0.f;
+    float* Drow = a.D + ((r0 + dt) * H + head) * dv + col0 + 4 * cg;
+    float4 d = make_float4(0.f, 0.f, 0.f, 0.f);                       // U of row dt
+    if (dt < len) {
+      if (vec_col) d = *reinterpret_cast<const float4*>(Drow);
+      else {
+        const int left = dv - col0 - 4 * cg;
+        if (left > 0) d.x = Drow[0];
+        if (left > 1) d.y = Drow[1];
+        if (left > 2) d.z = Drow[2];
+        if (left > 3) d.w = Drow[3];
       }
-    __syncthreads();
-    for (int k = k_lo; k < k_hi; k += 4) {
-      float2 s[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[e] = *reinterpret_cast<const float2*>(S + (k + e) * ldc + 2 * tx);
-#pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        const float4 w = lds4(Ws + (ty + 16 * m) * ldk + k);
-        u[m][0] = fmaf(-w.x, s[0].x, u[m][0]); u[m][1] = fmaf(-w.x, s[0].y, u[m][1]);
-        u[m][0] = fmaf(-w.y, s[1].x, u[m][0]); u[m][1] = fmaf(-w.y, s[1].y, u[m][1]);
-        u[m][0] = fmaf(-w.z, s[2].x, u[m][0]); u[m][1] = fmaf(-w.z, s[2].y, u[m][1]);
-        u[m][0] = fmaf(-w.w, s[3].x, u[m][0]); u[m][1] = fmaf(-w.w, s[3].y, u[m][1]);
-      }
-    }
-    if (half) {
-#pragma unroll
-      for (int m = 0; m < 4; ++m) *reinterpret_cast<float2*>(Ds + (ty + 16 * m) * ldc + 2 * tx) = make_float2(u[m][0], u[m][1]);
     }
     __syncthreads();
-    if (half) {     // S at the piece's start, for the read-out
-      float* dst = a.S0 + ((int64_t)(first + i) * H + head) * dk * dv + col0;
-      if (a.vec) {
-        for (int j = tid & 255; j < dk * (kWalkCols / 4); j += 256) {
-          const int k = j >> 3, c = (j & 7) * 4;
-          if (col0 + c < dv) *reinterpret_cast<float4*>(dst + (int64_t)k * dv + c) = lds4(S + k * ldc + c);
-        }
-      } else {
-        for (int j = tid & 255; j < dk * kWalkCols; j += 256) {
-          const int k = j / kWalkCols, c = j - k * kWalkCols;
-          if (col0 + c < dv) dst[(int64_t)k * dv + c] = S[k * ldc + c];
+    {
+      float4 u[4];
+#pragma unroll
+      for (int m = 0; m < 4; ++m) u[m] = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = k_lo; k < k_hi; k += 4) {
+        const float4 s0 = lds4(S + k * ldc + 4 * cg), s1 = lds4(S + (k + 1) * ldc + 4 * cg), s2 = lds4(S + (k + 2) * ldc + 4 * cg),
+                     s3 = lds4(S + (k + 3) * ldc + 4 * cg);
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          const float4 q = lds4(Ws + (rg + 16 * m) * ldk + k);
+          u[m].x = fmaf(q.x, s0.x, u[m].x); u[m].y = fmaf(q.x, s0.y, u[m].y); u[m].z = fmaf(q.x, s0.z, u[m].z); u[m].w = fmaf(q.x, s0.w, u[m].w);
+          u[m].x = fmaf(q.y, s1.x, u[m].x); u[m].y = fmaf(q.y, s1.y, u[m].y); u[m].z = fmaf(q.y, s1.z, u[m].z); u[m].w = fmaf(q.y, s1.w, u[m].w);
+          u[m].x = fmaf(q.z, s2.x, u[m].x); u[m].y = fmaf(q.z, s2.y, u[m].y); u[m].z = fmaf(q.z, s2.z, u[m].z); u[m].w = fmaf(q.z, s2.w, u[m].w);
+          u[m].x = fmaf(q.w, s3.x, u[m].x); u[m].y = fmaf(q.w, s3.y, u[m].y); u[m].z = fmaf(q.w, s3.z, u[m].z); u[m].w = fmaf(q.w, s3.w, u[m].w);
         }
       }
-    } else {
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        const int t = ty + 16 * m;
-        float2* d2 = reinterpret_cast<float2*>(Ds + t * ldc + 2 * tx);
-        const float2 other = *d2;
-        u[m][0] += other.x; u[m][1] += other.y;
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const int col = col0 + 2 * tx + c;
-          if (t < len && col < dv) a.D[((r0 + t) * H + head) * dv + col] = u[m][c];
+      for (int m = 0; m < 4; ++m) *reinterpret_cast<float4*>(red + (slice * kPieceMax + rg + 16 * m) * kWalkCols + 4 * cg) = u[m];
+    }
+    {   // S at the piece's start, for the read-out
+      float* dst = a.S0 + ((int64_t)(first + i) * H + head) * dk * dv + col0 + 4 * cg;
+      for (int k = tid >> 2; k < dk; k += kThreads / 4) {
+        const float4 v = lds4(S + k * ldc + 4 * cg);
+        float* p = dst + (int64_t)k * dv;
+        if (vec_col) *reinterpret_cast<float4*>(p) = v;
+        else {
+          const int left = dv - col0 - 4 * cg;
+          if (left > 0) p[0] = v.x;
+          if (left > 1) p[1] = v.y;
+          if (left > 2) p[2] = v.z;
+          if (left > 3) p[3] = v.w;
         }
-        *d2 = make_float2(u[m][0] * fin[t], u[m][1] * fin[t]);
       }
     }
-    __syncthreads();                              // D complete, every read of the old S done
+    __syncthreads();
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const float4 v = lds4(red + (q * kPieceMax + dt) * kWalkCols + 4 * cg);
+      d.x -= v.x; d.y -= v.y; d.z -= v.z; d.w -= v.w;
+    }
+    if (dt < len) {
+      if (vec_col) *reinterpret_cast<float4*>(Drow) = d;
+      else {
+        const int left = dv - col0 - 4 * cg;
+        if (left > 0) Drow[0] = d.x;
+        if (left > 1) Drow[1] = d.y;
+        if (left > 2) Drow[2] = d.z;
+        if (left > 3) Drow[3] = d.w;
+      }
+    }
+    const float f = fin[dt];
+    *reinterpret_cast<float4*>(Ds + dt * ldc + 4 * cg) = make_float4(d.x * f, d.y * f, d.z * f, d.w * f);
+    __syncthreads();                              // D complete, every read of the old S and of the partial sums done
     const float ge = gend;
-    for (int k0 = 4 * kg; k0 < dk4; k0 += 128) {
-      float2 acc[4];
+    float4 acc[2][4];                             // two passes of 128 key channels
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        acc[e] = *reinterpret_cast<const float2*>(S + (k0 + e) * ldc + 2 * cg);
-        acc[e].x *= ge; acc[e].y *= ge;
-      }
+    for (int p = 0; p < 2; ++p) {
+      const int k0 = 4 * kg + 128 * p;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[p][e] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (k0 >= dk4) continue;
 #pragma unroll 8
-      for (int t = 0; t < kPieceMax; ++t) {
-        const float4 kv = lds4(Kt + t * ldk + k0);
-        const float2 d = *reinterpret_cast<const float2*>(Ds + t * ldc + 2 * cg);
-        acc[0].x = fmaf(kv.x, d.x, acc[0].x); acc[0].y = fmaf(kv.x, d.y, acc[0].y);
-        acc[1].x = fmaf(kv.y, d.x, acc[1].x); acc[1].y = fmaf(kv.y, d.y, acc[1].y);
-        acc[2].x = fmaf(kv.z, d.x, acc[2].x); acc[2].y = fmaf(kv.z, d.y, acc[2].y);
-        acc[3].x = fmaf(kv.w, d.x, acc[3].x); acc[3].y = fmaf(kv.w, d.y, acc[3].y);
+      for (int t = half * (kPieceMax / 2); t < (half + 1) * (kPieceMax / 2); ++t) {
+        const float4 kv = lds4(Kt + t * ldk + k0), v = lds4(Ds + t * ldc + 4 * cg);
+        acc[p][0].x = fmaf(kv.x, v.x, acc[p][0].x); acc[p][0].y = fmaf(kv.x, v.y, acc[p][0].y); acc[p][0].z = fmaf(kv.x, v.z, acc[p][0].z); acc[p][0].w = fmaf(kv.x, v.w, acc[p][0].w);
+        acc[p][1].x = fmaf(kv.y, v.x, acc[p][1].x); acc[p][1].y = fmaf(kv.y, v.y, acc[p][1].y); acc[p][1].z = fmaf(kv.y, v.z, acc[p][1].z); acc[p][1].w = fmaf(kv.y, v.w, acc[p][1].w);
+        acc[p][2].x = fmaf(kv.z, v.x, acc[p][2].x); acc[p][2].y = fmaf(kv.z, v.y, acc[p][2].y); acc[p][2].z = fmaf(kv.z, v.z, acc[p][2].z); acc[p][2].w = fmaf(kv.z, v.w, acc[p][2].w);
+        acc[p][3].x = fmaf(kv.w, v.x, acc[p][3].x); acc[p][3].y = fmaf(kv.w, v.y, acc[p][3].y); acc[p][3].z = fmaf(kv.w, v.z, acc[p][3].z); acc[p][3].w = fmaf(kv.w, v.w, acc[p][3].w);
       }
+      if (half)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) *reinterpret_cast<float2*>(S + (k0 + e) * ldc + 2 * cg) = acc[e];
+        for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(red + (k0 + e) * kWalkCols + 4 * cg) = acc[p][e];
     }
+    __syncthreads();
+    if (!half)
+#pragma unroll
+      for (int p = 0; p < 2; ++p) {
+        const int k0 = 4 * kg + 128 * p;
+        if (k0 >= dk4) continue;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float4* sp = reinterpret_cast<float4*>(S + (k0 + e) * ldc + 4 * cg);
+          const float4 o = lds4(red + (k0 + e) * kWalkCols + 4 * cg), v = *sp;
+          *sp = make_float4(fmaf(ge, v.x, acc[p][e].x + o.x), fmaf(ge, v.y, acc[p][e].y + o.y), fmaf(ge, v.z, acc[p][e].z + o.z),
+                            fmaf(ge, v.w, acc[p][e].w + o.w));
+        }
+      }
     __syncthreads();                              // the next piece's copies and gates overwrite what was read here
   }
   cp_wait<0>();
-  for (int i = tid; i < kWalkCols * dk; i += kWalkThreads) {
+  for (int i = tid; i < kWalkCols * dk; i += kThreads) {
     const int c = i / dk, k = i - c * dk;
     if (col0 + c < dv) state[(int64_t)(col0 + c) * dk + k] = S[k * ldc + c];
   }
@@ -677,8 +735,9 @@ __global__ void __launch_bounds__(kWalkThreads, 1) gated_delta_walk_kernel(Split
 
 // O = G * (Q S_0) + E D of one (piece, value head), 128 value columns per pass; NORM (dv <= 128): the head norm, the gain and
 // the gate, into `out`; otherwise the raw read-out replaces D.
+constexpr int kReadThreads = 128;
 template <typename T, bool NORM>
-__global__ void __launch_bounds__(kThreads, 3) gated_delta_read_kernel(SplitArgs a) {
+__global__ void __launch_bounds__(kReadThreads, 3) gated_delta_read_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   constexpr int kStep = 32, lda = kStep + 4, ldb = kOutCols + 4;
@@ -705,16 +764,16 @@ __global__ void __launch_bounds__(kThreads, 3) gated_delta_read_kernel(SplitArgs
     }
     cp_commit();
   };
-  const int ty = tid >> 4, tx = tid & 15;         // rows ty + 16 m, columns 4 tx .. and 64 + 4 tx ..
-  float acc[4][8];
+  const int ty = tid >> 4, tx = tid & 15;         // rows ty + 8 m, columns 4 tx .. and 64 + 4 tx ..
+  float acc[8][8];
 #pragma unroll
-  for (int m = 0; m < 4; ++m)
+  for (int m = 0; m < 8; ++m)
 #pragma unroll
     for (int c = 0; c < 8; ++c) acc[m][c] = 0.f;
-  float up[4];                                    // G_t
+  float up[8];                                    // G_t
 #pragma unroll
-  for (int m = 0; m < 4; ++m) {
-    const int t = ty + 16 * m;
+  for (int m = 0; m < 8; ++m) {
+    const int t = ty + 8 * m;
     up[m] = t < len ? expf(a.gates[(row0 + t) * 2 * H + head]) : 0.f;
   }
   stage(0);
@@ -724,21 +783,21 @@ __global__ void __launch_bounds__(kThreads, 3) gated_delta_read_kernel(SplitArgs
     __syncthreads();
     if (i == n1)
 #pragma unroll
-      for (int m = 0; m < 4; ++m)
+      for (int m = 0; m < 8; ++m)
 #pragma unroll
         for (int c = 0; c < 8; ++c) acc[m][c] *= up[m];
     const float* as = As + (i & 1) * kPieceMax * lda;
     const float* bs = Bs + (i & 1) * kStep * ldb;
 #pragma unroll
     for (int k = 0; k < kStep; k += 4) {
-      float4 q[4];
+      float4 q[8];
 #pragma unroll
-      for (int m = 0; m < 4; ++m) q[m] = lds4(as + (ty + 16 * m) * lda + k);
+      for (int m = 0; m < 8; ++m) q[m] = lds4(as + (ty + 8 * m) * lda + k);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float4 b0 = lds4(bs + (k + e) * ldb + 4 * tx), b1 = lds4(bs + (k + e) * ldb + 64 + 4 * tx);
 #pragma unroll
-        for (int m = 0; m < 4; ++m) {
+        for (int m = 0; m < 8; ++m) {
           const float w = e == 0 ? q[m].x : e == 1 ? q[m].y : e == 2 ? q[m].z : q[m].w;
           acc[m][0] = fmaf(w, b0.x, acc[m][0]); acc[m][1] = fmaf(w, b0.y, acc[m][1]); acc[m][2] = fmaf(w, b0.z, acc[m][2]); acc[m][3] = fmaf(w, b0.w, acc[m][3]);
           acc[m][4] = fmaf(w, b1.x, acc[m][4]); acc[m][5] = fmaf(w, b1.y, acc[m][5]); acc[m][6] = fmaf(w, b1.z, acc[m][6]); acc[m][7] = fmaf(w, b1.w, acc[m][7]);
@@ -749,8 +808,8 @@ __global__ void __launch_bounds__(kThreads, 3) gated_delta_read_kernel(SplitArgs
   }
   cp_wait<0>();
 #pragma unroll
-  for (int m = 0; m < 4; ++m) {
-    const int t = ty + 16 * m;
+  for (int m = 0; m < 8; ++m) {
+    const int t = ty + 8 * m;
     if constexpr (NORM) {
       float ss = 0.f;                             // columns past dv are zero
 #pragma unroll
@@ -865,18 +924,20 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
   const size_t sm_piece = ((size_t)2 * kPieceMax * ldk + kPieceMax * (kPieceMax + 4)) * sizeof(float);
   static SmemAttr at_piece = {};
   PRL_CUDA(ensure_smem(gated_delta_piece_kernel, (int)sm_piece, at_piece));
-  PRL_CUDA(launch_pdl(gated_delta_piece_kernel, dim3(n_sub, heads), dim3(kThreads), sm_piece, s, a));
+  PRL_CUDA(launch_pdl(gated_delta_piece_kernel, dim3(n_sub, heads), dim3(kPieceThreads), sm_piece, s, a));
   PRL_LAUNCH_CHECK();
-  const int stages = dk4 <= 128 ? 2 : 1;
-  const size_t sm_walk = ((size_t)stages * 2 * kPieceMax * ldk + (size_t)(dk4 + kPieceMax) * (kWalkCols + 4)) * sizeof(float);
   const dim3 gw((dv + kWalkCols - 1) / kWalkCols, heads, n_seg);
+  // partial sums: four quarters of the key channels for 64 rows, later one half of the update
+  const size_t red = (size_t)kWalkCols * (4 * kPieceMax > dk4 ? 4 * kPieceMax : dk4);
+  const int stages = dk4 <= 128 && (int64_t)gw.x * gw.y * gw.z <= num_sms() ? 2 : 1;
+  const size_t sm_walk = ((size_t)stages * 2 * kPieceMax * ldk + (size_t)(dk4 + kPieceMax) * (kWalkCols + 4) + red) * sizeof(float);
   static SmemAttr at_walk[2] = {};
   if (stages == 2) {
     PRL_CUDA(ensure_smem(gated_delta_walk_kernel<2>, (int)sm_walk, at_walk[0]));
-    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<2>, gw, dim3(kWalkThreads), sm_walk, s, a));
+    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<2>, gw, dim3(kThreads), sm_walk, s, a));
   } else {
     PRL_CUDA(ensure_smem(gated_delta_walk_kernel<1>, (int)sm_walk, at_walk[1]));
-    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<1>, gw, dim3(kWalkThreads), sm_walk, s, a));
+    PRL_CUDA(launch_pdl(gated_delta_walk_kernel<1>, gw, dim3(kThreads), sm_walk, s, a));
   }
   PRL_LAUNCH_CHECK();
   const size_t sm_read = (size_t)2 * (kPieceMax * 36 + 32 * (kOutCols + 4)) * sizeof(float);
@@ -885,7 +946,7 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
 #define PRL_GR(T, NORM, I)                                                                                   \
   do {                                                                                                       \
     PRL_CUDA(ensure_smem((gated_delta_read_kernel<T, NORM>), (int)sm_read, at_read[I]));                     \
-    PRL_CUDA(launch_pdl((gated_delta_read_kernel<T, NORM>), gr, dim3(kThreads), sm_read, s, a));             \
+    PRL_CUDA(launch_pdl((gated_delta_read_kernel<T, NORM>), gr, dim3(kReadThreads), sm_read, s, a));             \
   } while (0)
   if (dv > kOutCols) PRL_GR(float, false, 0);
   else if (f32) PRL_GR(float, true, 1);

@@ -1352,6 +1352,7 @@ class HybridEngine(EngineCore):
         cfg, d, lib = self.cfg, self.dev, self.lib
         self.k_pool, self.v_pool, self.conv_state, self.ssd_state, self.gla_state, self.rot_freq = {}, {}, {}, {}, {}, {}
         self.tc_attn: dict[int, bool] = {}
+        self.tc_prompt: dict[int, bool] = {}             # windowed attention whose prompts run the tcgen05 kernel
         self.lin_state, self.lin_decay, self.mlstm_state, self.mlstm_m = {}, {}, {}, {}
         self.lat_pool, self.delta_state = {}, {}
         self._head_tables: dict = {}
@@ -1364,9 +1365,11 @@ class HybridEngine(EngineCore):
                 # head size 128 in bf16 without window, sink or cap: the tcgen05 prompt kernel and the TMA decode kernel
                 self.tc_attn[i] = (cfg.block == "one_norm" and not self.f32 and a.dim == 128 and a.vdim == 128
                                    and a.heads // a.kv_heads in (1, 2, 4, 8, 16))
+                self.tc_prompt[i] = (cfg.block in ("post_ln", "pre_norm") and not self.f32 and a.dim == 128 and a.vdim == 128
+                                     and a.weights == "softmax" and not a.softcap and a.heads // a.kv_heads in (1, 2, 4, 8, 16))
                 if a.kv_from >= 0:                       # another run's cache: nothing of its own
                     self.k_pool[i], self.v_pool[i] = self.k_pool[a.kv_from], self.v_pool[a.kv_from]
-                elif self.tc_attn[i]:                    # K and V pools adjacent
+                elif self.tc_attn[i] or self.tc_prompt[i]:      # K and V pools adjacent
                     pair = torch.zeros(2, self.n_pages, a.kv_heads, PAGE_SIZE, a.dim, dtype=self.op_dtype, device=d)
                     self.k_pool[i], self.v_pool[i] = pair[0], pair[1]
                 else:
@@ -1868,10 +1871,7 @@ class HybridEngine(EngineCore):
                                       self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr(), f32, st))
         sink = vec[w + "mix.sink"].data_ptr() if a.sink else None
         gate = P + 4 * (nq + nk + nv) if a.gate and a.gate_per_head else None
-        _lib.check(lib.prl_attn_any_gated(R.q.data_ptr(), self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr(), a.vdim, f32,
-                                          self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE, seg_start, seg_len,
-                                          seg_pos0.data_ptr(), seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale,
-                                          a.window, 0, a.softcap, sink, gate, ld, 1, R.ya.data_ptr(), st))
+        self._softmax_attn(R, n, i, a, segs, max_q, seg_pos0, sink, gate, ld)
         return self._mm(R.ya, no, w + "mix.o", W, R.y0, n, split=True)
 
     # ---- the 'one_norm' block: x <- x + (mixer(h) + ff(h)), h = norm(x) --------------------------------------------------
@@ -2097,17 +2097,30 @@ class HybridEngine(EngineCore):
     def _gated_window_attn(self, R, n, i, a, C, segs, max_q, row_pos, seg_pos0) -> None:
         """Softmax attention from the projections in R.P (AttnDeltaRows) to the gated heads R.ya."""
         lib, st, f32 = self.lib, self._st, int(self.f32)
-        seg_start, seg_len, seg_slot, ns = segs
         P, ld = R.P.data_ptr(), C.total
         bt = (self.block_table.data_ptr(), self.max_blocks, PAGE_SIZE)
         kv = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr())
         _lib.check(lib.prl_attn_front(P, ld, 0, C.k, C.v, n, a.heads, a.kv_heads, a.dim, a.vdim, None, None, None, 0, None, None, a.dim,
                                       self.cfg.eps, a.rot_dims, self.rot_freq[i].data_ptr(), self.rot_mag[i], 0, 0, None, None,
                                       row_pos.data_ptr(), R.row_slot.data_ptr(), *bt, R.q.data_ptr(), *kv, f32, st))
-        sink = self.zero_sink.data_ptr() if a.unit_sink else None
-        _lib.check(lib.prl_attn_any_gated(R.q.data_ptr(), *kv, a.vdim, f32, *bt, seg_start, seg_len, seg_pos0.data_ptr(), seg_slot, ns,
-                                          max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, 0, a.softcap, sink,
-                                          P + 4 * C.left_g if a.gate else None, ld, 1, R.ya.data_ptr(), st))
+        self._softmax_attn(R, n, i, a, segs, max_q, seg_pos0, self.zero_sink.data_ptr() if a.unit_sink else None,
+                           P + 4 * C.left_g if a.gate else None, ld)
+
+    def _softmax_attn(self, R, n, i, a, segs, max_q, seg_pos0, sink, gate, ldg) -> None:
+        """Attention of R.q over run i's cache into R.ya (operand type), with the layer's window, a sink logit per head and one
+        gate per head and row (pointers, None without): the tcgen05 kernel for prompts with heads of 128, else the
+        any-geometry kernels."""
+        lib, f32 = self.lib, int(self.f32)
+        seg_start, seg_len, seg_slot, ns = segs
+        kv, bt = (self.k_pool[i].data_ptr(), self.v_pool[i].data_ptr()), (self.block_table.data_ptr(), self.max_blocks)
+        if self.tc_prompt[i] and max_q >= 32 and not self.force_plain_attn:
+            _lib.check(lib.prl_paged_attn_prefill_tc_gated(R.q.data_ptr(), n, kv[0], self.n_pages, 1, 0, *bt, seg_start, seg_len,
+                                                           seg_pos0.data_ptr(), seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim,
+                                                           PAGE_SIZE, a.scale, a.window, sink, gate, ldg, R.ya.data_ptr(), self._st))
+            return
+        _lib.check(lib.prl_attn_any_gated(R.q.data_ptr(), *kv, a.vdim, f32, *bt, PAGE_SIZE, seg_start, seg_len, seg_pos0.data_ptr(),
+                                          seg_slot, ns, max_q, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.keep_first,
+                                          a.softcap, sink, gate, ldg, 1, R.ya.data_ptr(), self._st))
 
     def _gated_delta_cell(self, R, n, i, g, p, segs, max_q, P, ld, off, off_b, off_a, off_g) -> None:
         """From the projections in P (rows ld apart: q | k | v at `off`, step, decay and gate columns) to the cell's normed and

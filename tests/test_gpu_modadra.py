@@ -358,6 +358,7 @@ def test_tensor_core_prompt_attention(cuda_device, dim, vdim, window):
     ref = mc.oracle_logits(config, wt, toks)
     eng = mc.build_engine(config, wt, torch.bfloat16, cuda_device, prefill_chunk=512)
     plans = ([330], [63, 17, 16, 130, 65, 20, 3, 2], [300])                 # the rest one by one
+    eng.tc_prompt[0] = False                                                # heads of 128 have another test
     fast = [mc.stream_logits(eng, toks, p) for p in plans]
     eng.lib.prl_attn_any_tensor_cores(0)
     try:
@@ -427,6 +428,74 @@ def test_token_step_of_the_gated_delta_rule(cuda_device, heads, kv, dk, dv, taps
         at += k
     eng.close_stream(s)
     assert mc.rel_err(torch.cat(out).double().cpu(), ref[:at]) < F32_TOL
+
+
+@pytest.mark.parametrize("heads,kv_heads,window", [(2, 1, 37), (4, 1, 64), (8, 1, 129), (3, 3, 200), (16, 1, 90), (4, 2, 0), (4, 2, 1), (2, 2, 128)])
+def test_tcgen05_prompt_attention(cuda_device, heads, kv_heads, window):
+    """Heads of 128 in bf16: the tcgen05 prompt kernel with its window, the constant sink and the head gates, against the
+    CUDA-core kernel on the same cache and against the oracle.  Portions start inside a page and a key step, rows of a tile
+    lose keys of the first step to the window, and steps of a tile may be hidden from some of its rows altogether."""
+    config = mc.model([P(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, rot_dims=32, window=window, scale=1.5 * 128 ** -0.5)], width=64)
+    wt = mc.weights(config, 9)
+    toks = mc.tokens_for(config, 520, seed=3)
+    ref = mc.oracle_logits(config, wt, toks)
+    eng = mc.build_engine(config, wt, torch.bfloat16, cuda_device, prefill_chunk=520, max_seq_len=576)
+    assert eng.tc_prompt[0]
+    plans = ([520], [63, 130, 257, 3, 60], [300, 200])                     # the rest one by one
+    fast = [mc.stream_logits(eng, toks, p) for p in plans]
+    eng.force_plain_attn = True
+    eng.lib.prl_attn_any_tensor_cores(0)
+    try:
+        plain = mc.stream_logits(eng, toks, [520])
+    finally:
+        eng.lib.prl_attn_any_tensor_cores(1)
+    for f in fast:
+        assert mc.rel_err(f, plain) < 0.5 * BF16_TOL and mc.rel_err(f, ref) < BF16_TOL
+    assert (fast[0] != plain).any()
+
+
+@pytest.mark.parametrize("shift", [0.0, -150.0, 150.0])
+@pytest.mark.parametrize("heads,kv_heads,pos0,rows,window", [(4, 2, 0, 200, 37), (2, 2, 130, 300, 64), (8, 1, 77, 40, 129), (4, 4, 500, 150, 0)])
+def test_tcgen05_prompt_attention_alone(cuda_device, shift, heads, kv_heads, pos0, rows, window):
+    """The tcgen05 prompt kernel alone, with and without a sink and gates, on scores that are all far below (or far above) zero:
+    rows of a tile that see nothing in its first steps must take their reference from the first step they do see."""
+    from pipelinerl_b200 import _lib
+    lib, d = _lib.load(), cuda_device
+    g = torch.Generator().manual_seed(rows)
+    S, R = pos0 + rows, heads // kv_heads
+    c = torch.sign(torch.randn(128, generator=g))
+    q = mc.bf16_round(torch.randn(rows, heads, 128, generator=g) * 0.3 + c * (0.5 if shift else 0.0))
+    k = mc.bf16_round(torch.randn(S, kv_heads, 128, generator=g) * 0.3 + c * (shift / 64.0))
+    v = mc.bf16_round(torch.randn(S, kv_heads, 128, generator=g))
+    sink, gate = torch.randn(heads, generator=g) + shift, torch.randn(rows, heads, generator=g)
+    pages = -(-S // 64)
+    order = torch.randperm(pages, generator=g) + 1
+    kv = torch.zeros(2, pages + 1, kv_heads, 64, 128, dtype=torch.bfloat16)
+    for t in range(S):
+        kv[0, order[t // 64], :, t % 64], kv[1, order[t // 64], :, t % 64] = k[t].bfloat16(), v[t].bfloat16()
+    scale = 1.0                                                             # scores around `shift`
+    i32 = dict(dtype=torch.int32, device=d)
+    bt = order.int().view(1, -1).to(d)
+    one = lambda x: torch.tensor([x], **i32)
+    ss, sl, sp, slot = one(0), one(rows), one(pos0), one(0)
+    qd, kvd, sd, gd = q.bfloat16().to(d), kv.to(d), sink.to(d), gate.to(d)
+    for use in (False, True):
+        out = torch.zeros(rows, heads, 128, dtype=torch.bfloat16, device=d)
+        _lib.check(lib.prl_paged_attn_prefill_tc_gated(qd.data_ptr(), rows, kvd.data_ptr(), pages + 1, 1, 0, bt.data_ptr(), pages, ss.data_ptr(),
+                                                       sl.data_ptr(), sp.data_ptr(), slot.data_ptr(), 1, rows, heads, kv_heads, 128, 64, scale,
+                                                       window, sd.data_ptr() if use else None, gd.data_ptr() if use else None, heads,
+                                                       out.data_ptr(), _lib.stream_ptr()))
+        back = (pos0 + torch.arange(rows))[:, None] - torch.arange(S)[None, :]
+        see = (back >= 0) & ((back < window) if window else torch.ones_like(back, dtype=torch.bool))
+        ref = torch.zeros(rows, heads, 128, dtype=torch.float64)
+        for h in range(heads):
+            s = (q[:, h].double() @ k[:, h // R].double().T * scale).masked_fill(~see, -math.inf)
+            if use:
+                s = torch.cat([s, sink[h].double().expand(rows, 1)], 1)
+            w = torch.softmax(s, 1)[:, :S]
+            ref[:, h] = w @ v[:, h // R].double() * (torch.sigmoid(gate[:, h].double())[:, None] if use else 1.0)
+        err = (out.double().cpu() - ref).abs().max().item()
+        assert err < 0.03, (use, err)
 
 
 def test_long_decoding(cuda_device):
