@@ -21,11 +21,11 @@
 //        O = G * (Q S_0) + E D,                   E_ts = (G_t / G_s) (q_t . k_s) for s <= t
 //        S_end = G_end S_0 + (K * (G_end / G))^T D
 //    so that D = U - W S_0 with U = (I + A)^(-1) (b * V), W = (I + A)^(-1) (b * G * K).  Four kernels: the front end
-//    (convolution, unit vectors, gates); per piece and head A, E and, by forward substitution with one column per thread, U
+//    (convolution, unit vectors, gates); per piece and head A, E and, by forward substitution with two columns per thread, U
 //    and W; the walk over the pieces of a segment, which only carries S (two products per piece, a tile of 16 value columns per
 //    CTA) and leaves D and every piece's S_0; the read-out, per piece and head again, with the head norm and the gate.  All
-//    products are register-blocked fp32 FMAs (a warp's shared-memory reads cost by the bytes its lanes receive, broadcast or
-//    not, so the tiles are as square and as large as the work leaves threads for).  Decays enter as differences of running sums of logarithms, which are never
+//    products are register-blocked fp32 FMAs on the CUDA cores; the piece kernel issues two per instruction (fma.rn.f32x2), on
+//    pairs of neighbouring channels or columns.  Decays enter as differences of running sums of logarithms, which are never
 //    positive, so nothing overflows.
 #include "prl_common.cuh"
 #include <math.h>
@@ -57,6 +57,26 @@ __device__ __forceinline__ void cp16z(float* dst, const float* src, int bytes) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ float4 lds4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+
+// two fp32 numbers in a 64-bit register
+typedef unsigned long long pair_t;
+__device__ __forceinline__ pair_t fma2(pair_t a, pair_t b, pair_t c) {
+  pair_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ pair_t pack2(float x, float y) {
+  pair_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+  return d;
+}
+__device__ __forceinline__ float2 unpack2(pair_t a) {
+  float2 v;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(v.x), "=f"(v.y) : "l"(a));
+  return v;
+}
+__device__ __forceinline__ float sum2(pair_t a) { const float2 v = unpack2(a); return v.x + v.y; }
+__device__ __forceinline__ ulonglong2 ldp(const float* p) { return *reinterpret_cast<const ulonglong2*>(p); }
 
 // rows x cols floats (row stride ld_src) into shared rows of stride ld_dst; rows from `live` on and columns from `cols` to
 // `cols_pad` are zero.  `vec`: every source row starts on a 16-byte boundary and cols is a multiple of four.
@@ -429,27 +449,12 @@ __global__ void __launch_bounds__(kThreads) gated_delta_front_tile_kernel(SplitA
 }
 
 // A, E, U and W of one (piece, value head); the running sums of the log decays replace them in `gates`.
-// Row s of two columns is final: take its part out of the rows behind it.  At[s][t] = A_ts (zero at and above the diagonal).
-constexpr int kPieceLd = kPieceMax + 4;
-template <int s>
-__device__ __forceinline__ void substitute(float (&x)[2][kPieceMax], const float* At) {
-  if constexpr (s < kPieceMax - 1) {
-#pragma unroll
-    for (int t4 = (s + 1) / 4 * 4; t4 < kPieceMax; t4 += 4) {
-      const float4 c4 = lds4(At + s * kPieceLd + t4);
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        if (t4 > s) x[u][t4] = fmaf(-c4.x, x[u][s], x[u][t4]);
-        if (t4 + 1 > s) x[u][t4 + 1] = fmaf(-c4.y, x[u][s], x[u][t4 + 1]);
-        if (t4 + 2 > s) x[u][t4 + 2] = fmaf(-c4.z, x[u][s], x[u][t4 + 2]);
-        if (t4 + 3 > s) x[u][t4 + 3] = fmaf(-c4.w, x[u][s], x[u][t4 + 3]);
-      }
-    }
-    substitute<s + 1>(x, At);
-  }
-}
-
+// A is kept negated and doubled (each entry as a pair), as the ten 16 x 16 blocks on and below its diagonal: block (b, q) at
+// b (b + 1) / 2 + q, entry (column s, row t) at 32 s + 2 t.
 constexpr int kPieceThreads = 128;
+constexpr int kBlk = 16, kBlkFloats = kBlk * kBlk * 2;
+__device__ __forceinline__ int blk_at(int b, int q) { return (b * (b + 1) / 2 + q) * kBlkFloats; }
+
 __global__ void __launch_bounds__(kPieceThreads, 2) gated_delta_piece_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -457,10 +462,9 @@ __global__ void __launch_bounds__(kPieceThreads, 2) gated_delta_piece_kernel(Spl
   const int64_t row0 = a.sub_start[piece];
   const int dk = a.dk, dv = a.dv, H = a.heads, tid = threadIdx.x;
   const int dk4 = (dk + 3) & ~3, ldk = dk4 + 4, ch = 2 * a.kh * dk + H * dv, kvh = head / (H / a.kh);
-  constexpr int ldA = kPieceLd;
-  float* Ks = sm;                                 // [64][ldk]
-  float* Qs = Ks + kPieceMax * ldk;               // [64][ldk]
-  float* At = Qs + kPieceMax * ldk;               // [64][ldA]: At[s][t] = A_ts
+  float* As = sm;                                 // 10 blocks
+  float* Ks = As + 10 * kBlkFloats;               // [64][ldk]
+  float* Qs = Ks + kPieceMax * ldk;               // [64][ldk], later X: rows 0 .. 47 of the thread's two columns [48][256]
   __shared__ float cum[kPieceMax], beta[kPieceMax], bg[kPieceMax];      // running log decay, step, step times decay
   const float* C = a.C + row0 * ch;
   stage_tile(Ks, ldk, C + a.kh * dk + kvh * dk, ch, kPieceMax, len, dk, dk4, a.vec);
@@ -490,24 +494,22 @@ __global__ void __launch_bounds__(kPieceThreads, 2) gated_delta_piece_kernel(Spl
   {   // one half of the CTA forms K K^T, the other Q K^T, 8 x 8 entries per thread
     const bool query = tid >= 64;
     const int ty = tid >> 3 & 7, tx = tid & 7;
-    const float* As = query ? Qs : Ks;
-    float acc[8][8];
+    const float* rows = query ? Qs : Ks;
+    pair_t acc[8][8];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
+      for (int j = 0; j <= i; ++j) acc[i][j] = 0ull;
     for (int c = 0; c < dk4; c += 4) {
-      float4 s4[8];
+      ulonglong2 s4[8];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) s4[j] = lds4(Ks + (tx + 8 * j) * ldk + c);
+      for (int j = 0; j < 8; ++j) s4[j] = ldp(Ks + (tx + 8 * j) * ldk + c);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const float4 a4 = lds4(As + (ty + 8 * i) * ldk + c);
+        const ulonglong2 r4 = ldp(rows + (ty + 8 * i) * ldk + c);
 #pragma unroll
-        for (int j = 0; j <= i; ++j) {            // blocks above the diagonal are not needed
-          acc[i][j] = fmaf(a4.x, s4[j].x, acc[i][j]); acc[i][j] = fmaf(a4.y, s4[j].y, acc[i][j]);
-          acc[i][j] = fmaf(a4.z, s4[j].z, acc[i][j]); acc[i][j] = fmaf(a4.w, s4[j].w, acc[i][j]);
-        }
+        for (int j = 0; j <= i; ++j)              // blocks above the diagonal are not needed
+          acc[i][j] = fma2(r4.y, s4[j].y, fma2(r4.x, s4[j].x, acc[i][j]));
       }
     }
 #pragma unroll
@@ -516,43 +518,85 @@ __global__ void __launch_bounds__(kPieceThreads, 2) gated_delta_piece_kernel(Spl
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int s = tx + 8 * j;
-        const float e = s <= t ? expf(cum[t] - cum[s]) * acc[i][j] : 0.f;
-        if (!query) At[s * ldA + t] = s < t ? beta[t] * e : 0.f;      // rows past the piece have beta = 0
-        else if (t < len) a.E[((row0 + t) * H + head) * kPieceMax + s] = s < len ? e : 0.f;
+        const float e = j <= i && s <= t ? expf(cum[t] - cum[s]) * sum2(acc[i][j <= i ? j : 0]) : 0.f;
+        if (query) {
+          if (t < len) a.E[((row0 + t) * H + head) * kPieceMax + s] = s < len ? e : 0.f;
+        } else if (i / 2 >= j / 2) {              // a block on or below the diagonal; rows past the piece have beta = 0
+          const float v = s < t ? -beta[t] * e : 0.f;
+          *reinterpret_cast<float2*>(As + blk_at(i / 2, j / 2) + 32 * (s & 15) + 2 * (t & 15)) = make_float2(v, v);
+        }
       }
     }
   }
   __syncthreads();
-  // forward substitution, two columns of [b V | b G K] per thread, all 64 rows in registers
+  // forward substitution for two neighbouring columns of [b V | b G K] per thread, sixteen rows at a time: the rows done so
+  // far come back from shared memory (only the thread itself reads them)
   const float* V = C + 2 * a.kh * dk + head * dv;
-  for (int base = tid; base < dv + dk; base += 2 * kPieceThreads) {
-    float x[2][kPieceMax];
+  float* X = Qs + 2 * tid;
+  for (int col = 2 * tid; col < dv + dk; col += 2 * kPieceThreads) {
+    const bool two = col + 1 < dv + dk, same = a.vec;      // vec: dv is even, so both columns are in one matrix
+#pragma unroll 1
+    for (int b = 0; b < kPieceMax / kBlk; ++b) {
+      if (b * kBlk >= len) break;                 // rows past the piece are zero and nobody reads them
+      pair_t r[kBlk];
+      if (same && col < dv) {
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int col = base + u * kPieceThreads;
-      if (col < dv) {
-#pragma unroll
-        for (int t = 0; t < kPieceMax; ++t) x[u][t] = t < len ? V[(int64_t)t * ch + col] : 0.f;
-#pragma unroll
-        for (int t = 0; t < kPieceMax; ++t) x[u][t] *= beta[t];
-      } else if (col < dv + dk) {
-#pragma unroll
-        for (int t = 0; t < kPieceMax; ++t) x[u][t] = bg[t] * Ks[t * ldk + col - dv];
+        for (int t = 0; t < kBlk; ++t) {
+          const int tt = b * kBlk + t;
+          const float2 v = tt < len ? *reinterpret_cast<const float2*>(V + (int64_t)tt * ch + col) : make_float2(0.f, 0.f);
+          r[t] = pack2(beta[tt] * v.x, beta[tt] * v.y);
+        }
       } else {
 #pragma unroll
-        for (int t = 0; t < kPieceMax; ++t) x[u][t] = 0.f;
+        for (int t = 0; t < kBlk; ++t) {
+          const int tt = b * kBlk + t;
+          float v[2];
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const int c = col + u;
+            v[u] = c < dv ? (tt < len ? beta[tt] * V[(int64_t)tt * ch + c] : 0.f) : c < dv + dk ? bg[tt] * Ks[tt * ldk + c - dv] : 0.f;
+          }
+          r[t] = pack2(v[0], v[1]);
+        }
       }
-    }
-    substitute<0>(x, At);
+#pragma unroll 1
+      for (int q = 0; q < b; ++q) {
+        const float* blk = As + blk_at(b, q);
+#pragma unroll 4
+        for (int s = 0; s < kBlk; ++s) {
+          const pair_t x = *reinterpret_cast<const pair_t*>(X + (q * kBlk + s) * 2 * kPieceThreads);
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int col = base + u * kPieceThreads;
-      if (col >= dv + dk) continue;
-      float* dst = col < dv ? a.D + (row0 * H + head) * dv + col : a.W + (row0 * H + head) * dk + col - dv;
-      const int64_t step = (int64_t)H * (col < dv ? dv : dk);
+          for (int t = 0; t < kBlk; t += 2) {
+            const ulonglong2 w = ldp(blk + 32 * s + 2 * t);
+            r[t] = fma2(w.x, x, r[t]);
+            r[t + 1] = fma2(w.y, x, r[t + 1]);
+          }
+        }
+      }
+      const float* blk = As + blk_at(b, b);
 #pragma unroll
-      for (int t = 0; t < kPieceMax; ++t)
-        if (t < len) dst[t * step] = x[u][t];
+      for (int s = 0; s < kBlk - 1; ++s) {
+#pragma unroll
+        for (int t = (s + 1) / 2 * 2; t < kBlk; t += 2) {
+          const ulonglong2 w = ldp(blk + 32 * s + 2 * t);
+          if (t > s) r[t] = fma2(w.x, r[s], r[t]);
+          if (t + 1 > s) r[t + 1] = fma2(w.y, r[s], r[t + 1]);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < kBlk; ++t) {
+        const int tt = b * kBlk + t;
+        if (b + 1 < kPieceMax / kBlk) *reinterpret_cast<pair_t*>(X + tt * 2 * kPieceThreads) = r[t];
+        if (tt >= len) continue;
+        const float2 v = unpack2(r[t]);
+        float* u = a.D + ((row0 + tt) * H + head) * dv;
+        float* w = a.W + ((row0 + tt) * H + head) * dk - dv;
+        if (same) *reinterpret_cast<float2*>((col < dv ? u : w) + col) = v;
+        else {
+          (col < dv ? u : w)[col] = v.x;
+          if (two) (col + 1 < dv ? u : w)[col + 1] = v.y;
+        }
+      }
     }
   }
 }
@@ -735,9 +779,8 @@ __global__ void __launch_bounds__(kThreads, 2) gated_delta_walk_kernel(SplitArgs
 
 // O = G * (Q S_0) + E D of one (piece, value head), 128 value columns per pass; NORM (dv <= 128): the head norm, the gain and
 // the gate, into `out`; otherwise the raw read-out replaces D.
-constexpr int kReadThreads = 128;
 template <typename T, bool NORM>
-__global__ void __launch_bounds__(kReadThreads, 3) gated_delta_read_kernel(SplitArgs a) {
+__global__ void __launch_bounds__(kThreads, 2) gated_delta_read_kernel(SplitArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   constexpr int kStep = 32, lda = kStep + 4, ldb = kOutCols + 4;
@@ -764,16 +807,16 @@ __global__ void __launch_bounds__(kReadThreads, 3) gated_delta_read_kernel(Split
     }
     cp_commit();
   };
-  const int ty = tid >> 4, tx = tid & 15;         // rows ty + 8 m, columns 4 tx .. and 64 + 4 tx ..
-  float acc[8][8];
+  const int ty = tid >> 4, tx = tid & 15;         // rows ty + 16 m, columns 4 tx .. and 64 + 4 tx ..
+  float acc[4][8];
 #pragma unroll
-  for (int m = 0; m < 8; ++m)
+  for (int m = 0; m < 4; ++m)
 #pragma unroll
     for (int c = 0; c < 8; ++c) acc[m][c] = 0.f;
-  float up[8];                                    // G_t
+  float up[4];                                    // G_t
 #pragma unroll
-  for (int m = 0; m < 8; ++m) {
-    const int t = ty + 8 * m;
+  for (int m = 0; m < 4; ++m) {
+    const int t = ty + 16 * m;
     up[m] = t < len ? expf(a.gates[(row0 + t) * 2 * H + head]) : 0.f;
   }
   stage(0);
@@ -783,21 +826,21 @@ __global__ void __launch_bounds__(kReadThreads, 3) gated_delta_read_kernel(Split
     __syncthreads();
     if (i == n1)
 #pragma unroll
-      for (int m = 0; m < 8; ++m)
+      for (int m = 0; m < 4; ++m)
 #pragma unroll
         for (int c = 0; c < 8; ++c) acc[m][c] *= up[m];
     const float* as = As + (i & 1) * kPieceMax * lda;
     const float* bs = Bs + (i & 1) * kStep * ldb;
 #pragma unroll
     for (int k = 0; k < kStep; k += 4) {
-      float4 q[8];
+      float4 q[4];
 #pragma unroll
-      for (int m = 0; m < 8; ++m) q[m] = lds4(as + (ty + 8 * m) * lda + k);
+      for (int m = 0; m < 4; ++m) q[m] = lds4(as + (ty + 16 * m) * lda + k);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float4 b0 = lds4(bs + (k + e) * ldb + 4 * tx), b1 = lds4(bs + (k + e) * ldb + 64 + 4 * tx);
 #pragma unroll
-        for (int m = 0; m < 8; ++m) {
+        for (int m = 0; m < 4; ++m) {
           const float w = e == 0 ? q[m].x : e == 1 ? q[m].y : e == 2 ? q[m].z : q[m].w;
           acc[m][0] = fmaf(w, b0.x, acc[m][0]); acc[m][1] = fmaf(w, b0.y, acc[m][1]); acc[m][2] = fmaf(w, b0.z, acc[m][2]); acc[m][3] = fmaf(w, b0.w, acc[m][3]);
           acc[m][4] = fmaf(w, b1.x, acc[m][4]); acc[m][5] = fmaf(w, b1.y, acc[m][5]); acc[m][6] = fmaf(w, b1.z, acc[m][6]); acc[m][7] = fmaf(w, b1.w, acc[m][7]);
@@ -808,8 +851,8 @@ __global__ void __launch_bounds__(kReadThreads, 3) gated_delta_read_kernel(Split
   }
   cp_wait<0>();
 #pragma unroll
-  for (int m = 0; m < 8; ++m) {
-    const int t = ty + 8 * m;
+  for (int m = 0; m < 4; ++m) {
+    const int t = ty + 16 * m;
     if constexpr (NORM) {
       float ss = 0.f;                             // columns past dv are zero
 #pragma unroll
@@ -921,7 +964,8 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
   else PRL_CUDA(launch_pdl(gated_delta_front_kernel, dim3(n_rows), dim3(kThreads), (size_t)0, s, a));
   PRL_LAUNCH_CHECK();
   const int dk4 = (dk + 3) & ~3, ldk = dk4 + 4;
-  const size_t sm_piece = ((size_t)2 * kPieceMax * ldk + kPieceMax * (kPieceMax + 4)) * sizeof(float);
+  const size_t x_rows = (size_t)(kPieceMax - kBlk) * 2 * kPieceThreads, q_rows = (size_t)kPieceMax * ldk;
+  const size_t sm_piece = (10 * (size_t)kBlkFloats + q_rows + (q_rows > x_rows ? q_rows : x_rows)) * sizeof(float);
   static SmemAttr at_piece = {};
   PRL_CUDA(ensure_smem(gated_delta_piece_kernel, (int)sm_piece, at_piece));
   PRL_CUDA(launch_pdl(gated_delta_piece_kernel, dim3(n_sub, heads), dim3(kPieceThreads), sm_piece, s, a));
@@ -946,7 +990,7 @@ extern "C" int prl_gated_delta_split(const float* P, int64_t ldp, int32_t off, i
 #define PRL_GR(T, NORM, I)                                                                                   \
   do {                                                                                                       \
     PRL_CUDA(ensure_smem((gated_delta_read_kernel<T, NORM>), (int)sm_read, at_read[I]));                     \
-    PRL_CUDA(launch_pdl((gated_delta_read_kernel<T, NORM>), gr, dim3(kReadThreads), sm_read, s, a));             \
+    PRL_CUDA(launch_pdl((gated_delta_read_kernel<T, NORM>), gr, dim3(kThreads), sm_read, s, a));             \
   } while (0)
   if (dv > kOutCols) PRL_GR(float, false, 0);
   else if (f32) PRL_GR(float, true, 1);
