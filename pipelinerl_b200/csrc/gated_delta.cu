@@ -143,6 +143,27 @@ __global__ void __launch_bounds__(512) gated_delta_step_kernel(StepArgs a) {
   __shared__ float red[16], unit[2];
   const float* p = a.P + row * a.ldp;
   const int ch = 2 * a.kh * dk + a.heads * dv, keep = a.taps - 1;
+  const int grp = tid >> 8, t = tid & 255, cg = t >> 3, l8 = t & 7;
+  float4 S[CPT][R];
+  auto load = [&](const float* S0, int col0) {    // columns col0 + cg + 32 u of a head's state
+#pragma unroll
+    for (int u = 0; u < CPT; ++u) {
+      const int col = col0 + cg + 32 * u;
+      const float* s = S0 + (int64_t)col * dk;
+#pragma unroll
+      for (int j = 0; j < R; ++j) {
+        const int i = 4 * (l8 + 8 * j);
+        if (VEC) S[u][j] = (col < dv && i < dk) ? *reinterpret_cast<const float4*>(s + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        else {
+          const bool in = col < dv;
+          S[u][j] = make_float4(in && i < dk ? s[i] : 0.f, in && i + 1 < dk ? s[i + 1] : 0.f, in && i + 2 < dk ? s[i + 2] : 0.f,
+                                in && i + 3 < dk ? s[i + 3] : 0.f);
+        }
+      }
+    }
+  };
+  // the first states are on their way while the convolution runs
+  if (grp < rep) load(a.state + ((int64_t)slot * a.heads + kvh * rep + grp) * dv * dk, 0);
   for (int i = tid; i < 2 * (dkp - dk); i += blockDim.x) (i < dkp - dk ? qs + dk + i : ks + dk + i - (dkp - dk))[0] = 0.f;
   for (int i = tid; i < 2 * dk + rep * dv; i += blockDim.x) {
     const int c = i < dk ? kvh * dk + i : i < 2 * dk ? a.kh * dk + kvh * dk + i - dk : 2 * a.kh * dk + kvh * rep * dv + i - 2 * dk;
@@ -170,7 +191,6 @@ __global__ void __launch_bounds__(512) gated_delta_step_kernel(StepArgs a) {
   __syncthreads();
   for (int i = tid; i < dk; i += blockDim.x) { qs[i] *= unit[0]; ks[i] *= unit[1]; }
   __syncthreads();
-  const int grp = tid >> 8, t = tid & 255, cg = t >> 3, l8 = t & 7;
   for (int r0 = 0; r0 < rep; r0 += groups) {
     const bool on = r0 + grp < rep;               // uniform over the group's warps
     const int head = kvh * rep + r0 + grp;
@@ -180,22 +200,7 @@ __global__ void __launch_bounds__(512) gated_delta_step_kernel(StepArgs a) {
       const float g = expf(log_decay(a.A_log[head], p[a.off_a + head] + a.dt_bias[head]));
       float* S0 = a.state + ((int64_t)slot * a.heads + head) * dv * dk;
       for (int col0 = 0; col0 < dv; col0 += 32 * CPT) {
-        float4 S[CPT][R];
-#pragma unroll
-        for (int u = 0; u < CPT; ++u) {
-          const int col = col0 + cg + 32 * u;
-          const float* s = S0 + (int64_t)col * dk;
-#pragma unroll
-          for (int j = 0; j < R; ++j) {
-            const int i = 4 * (l8 + 8 * j);
-            if (VEC) S[u][j] = (col < dv && i < dk) ? *reinterpret_cast<const float4*>(s + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-            else {
-              const bool in = col < dv;
-              S[u][j] = make_float4(in && i < dk ? s[i] : 0.f, in && i + 1 < dk ? s[i + 1] : 0.f, in && i + 2 < dk ? s[i + 2] : 0.f,
-                                    in && i + 3 < dk ? s[i + 3] : 0.f);
-            }
-          }
-        }
+        if (r0 + col0 > 0) load(S0, col0);
         float dot[CPT], rd[CPT];
 #pragma unroll
         for (int u = 0; u < CPT; ++u) { dot[u] = 0.f; rd[u] = 0.f; }

@@ -146,24 +146,26 @@ __device__ __forceinline__ void choose_row(const float* z, int E, const ChoiceRu
       if (gs[e / size] != -INFINITY) c[e] = -INFINITY;     // still ranked: a closed group
     __syncwarp();
   }
-  float total = 0.f;
+  float total = 0.f, mine = 0.f;                           // lane k keeps choice k until the sum is known (up to 32 of them)
   for (int k = 0; k < r.top; ++k) {
     const int e = best_of(c, E);
     const bool ok = e < E;                                 // always, for finite logits
     const float w = ok ? score(e) : 0.f;
     total += w;
-    if (lane == 0) {
+    if (lane == (k & 31)) {
+      mine = w * r.scale;
       sel[(int64_t)k * n + t] = ok ? e : 0;
-      wsel[(int64_t)k * n + t] = w * r.scale;
+      if (r.top > 32) wsel[(int64_t)k * n + t] = mine;
       if (ok) c[e] = -INFINITY;
     }
     __syncwarp();
   }
-  if (r.renorm && lane == 0)
-    for (int k = 0; k < r.top; ++k) {
-      const float w = wsel[(int64_t)k * n + t];            // written by this lane
-      wsel[(int64_t)k * n + t] = w / (total + 1e-20f);
-    }
+  const float div = r.renorm ? total + 1e-20f : 1.f;
+  if (r.top <= 32) {
+    if (lane < r.top) wsel[(int64_t)lane * n + t] = mine / div;
+  } else if (r.renorm) {
+    for (int k = lane; k < r.top; k += 32) wsel[(int64_t)k * n + t] /= div;      // written by this lane
+  }
 }
 
 // Choice from ready logits, one warp per row.
@@ -180,7 +182,7 @@ __global__ void __launch_bounds__(kChooseWarps * 32) moe_choose_kernel(const flo
   choose_row(logits + (int64_t)t * ld, E, rule, c, c + E, n, t, sel, wsel);
 }
 
-// Router and choice in one kernel: logits[e] = x . Wr[e] in fp32 (block per row, the row staged in shared memory, warps
+// Router and choice in one kernel: logits[e] = x . Wr[e] in fp32 (block per row, warps
 // take experts in turn, a lane sums every 32nd group of channels, then the warp's shuffle tree: a fixed order), then the top-k
 // pass of moe_route_kernel over the logits in shared memory (RULED: choose_row instead, with scratch behind the logits).
 template <typename TX, typename TW, bool RULED>
@@ -193,14 +195,28 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const TX* __restrict__ 
   float* xs = rsm;
   float* z = rsm + W;
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  for (int c = threadIdx.x; c < W; c += blockDim.x) xs[c] = to_f32(x[(int64_t)t * W + c]);
-  __syncthreads();
   constexpr int V = 16 / sizeof(TW);              // router weights per 16-byte load
   const bool vec = W % V == 0 && ((uintptr_t)Wr & 15) == 0;
+  // one element type and aligned rows: the row is read beside the weights (from L1 for all warps but the first), not staged
+  const bool direct = sizeof(TX) == sizeof(TW) && vec && ((uintptr_t)x & 15) == 0;
+  if (!direct) {
+    for (int c = threadIdx.x; c < W; c += blockDim.x) xs[c] = to_f32(x[(int64_t)t * W + c]);
+    __syncthreads();
+  }
   for (int e = warp; e < E; e += nw) {
     const TW* w = Wr + (int64_t)e * W;
     float a = 0.f;
-    if (vec) {                                    // a lane sums its channels in ascending order
+    if (direct) {                                 // a lane sums its channels in ascending order
+      const TX* xr = x + (int64_t)t * W;
+#pragma unroll 4
+      for (int c = V * lane; c < W; c += 32 * V) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(w + c), xraw = *reinterpret_cast<const uint4*>(xr + c);
+        const TW* wv = reinterpret_cast<const TW*>(&raw);
+        const TX* xv = reinterpret_cast<const TX*>(&xraw);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a = fmaf(to_f32(xv[j]), to_f32(wv[j]), a);
+      }
+    } else if (vec) {
 #pragma unroll 4
       for (int c = V * lane; c < W; c += 32 * V) {
         const uint4 raw = *reinterpret_cast<const uint4*>(w + c);
@@ -303,6 +319,75 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
       if (mine) perm[at + __popc(mask & ((1u << lane) - 1u))] = p;
       at += __popc(mask);
     }
+  }
+}
+
+// The same for up to kGroupExperts experts: every warp counts a run of the pairs, then places them behind the runs of the warps
+// before it (a warp finds its lanes of one expert with a match, so the order stays that of the pairs).
+constexpr int kGroupExperts = 256, kGroupWarps = 32;
+__global__ void __launch_bounds__(32 * kGroupWarps) moe_group_runs_kernel(const int32_t* __restrict__ sel, int pairs, int E, int tile_rows,
+                                                                         int32_t* __restrict__ perm, int32_t* __restrict__ meta,
+                                                                         int32_t* __restrict__ tiles) {
+  pdl_wait();
+  extern __shared__ int32_t cnt[];      // [warps][E] counts, then first places; [E] totals; [E] first place and first tile
+  int32_t* total = cnt + kGroupWarps * E;
+  int32_t* off = total + E;
+  int32_t* tile0 = off + E;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int32_t* mine = cnt + warp * E;
+  for (int i = tid; i < kGroupWarps * E; i += blockDim.x) cnt[i] = 0;
+  __syncthreads();
+  const int run = (pairs + 32 * kGroupWarps - 1) / (32 * kGroupWarps) * 32, p_end = min(pairs, (warp + 1) * run);
+  for (int p0 = warp * run; p0 < p_end; p0 += 32) {
+    const int p = p0 + lane, e = p < p_end ? sel[p] : 0x7fffffff;
+    const uint32_t same = __match_any_sync(0xffffffffu, e);
+    if (e < E && lane == __ffs(same) - 1) mine[e] += __popc(same);       // a choice past the experts belongs to none of them
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = tid; e < E; e += blockDim.x) {
+    int at = 0;
+    for (int w = 0; w < kGroupWarps; ++w) {
+      const int c = cnt[w * E + e];
+      cnt[w * E + e] = at;
+      at += c;
+    }
+    total[e] = at;
+  }
+  __syncthreads();
+  if (warp == 0) {                      // first place and first tile of every expert: running sums, 32 experts at a time
+    int at = 0, nt = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int c = e0 + lane < E ? total[e0 + lane] : 0, k = (c + tile_rows - 1) / tile_rows;
+      int sc = c, sk = k;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int vc = __shfl_up_sync(0xffffffffu, sc, o), vk = __shfl_up_sync(0xffffffffu, sk, o);
+        if (lane >= o) { sc += vc; sk += vk; }
+      }
+      if (e0 + lane < E) { off[e0 + lane] = at + sc - c; tile0[e0 + lane] = nt + sk - k; }
+      at += __shfl_sync(0xffffffffu, sc, 31);
+      nt += __shfl_sync(0xffffffffu, sk, 31);
+    }
+    if (lane == 0) { meta[0] = nt; meta[1] = at; }
+  }
+  __syncthreads();
+  for (int e = tid; e < E; e += blockDim.x)
+    for (int r0 = 0, i = tile0[e]; r0 < total[e]; r0 += tile_rows, ++i) {
+      tiles[3 * i] = e;
+      tiles[3 * i + 1] = off[e] + r0;
+      tiles[3 * i + 2] = min(tile_rows, total[e] - r0);
+    }
+  for (int p0 = warp * run; p0 < p_end; p0 += 32) {
+    const int p = p0 + lane, e = p < p_end ? sel[p] : 0x7fffffff;
+    const uint32_t same = __match_any_sync(0xffffffffu, e);
+    const int first = e < E ? mine[e] : 0;
+    __syncwarp();
+    if (e < E) {
+      perm[off[e] + first + __popc(same & ((1u << lane) - 1u))] = p;
+      if (lane == __ffs(same) - 1) mine[e] = first + __popc(same);
+    }
+    __syncwarp();
   }
 }
 
@@ -567,6 +652,15 @@ __global__ void moe_glu_out_kernel(const float* __restrict__ gu, int64_t ld, int
 using namespace prl;
 typedef __nv_bfloat16 bf16;
 
+static cudaError_t launch_group(const int32_t* sel, int pairs, int experts, int tile_rows, int32_t* perm, int32_t* meta, int32_t* tiles,
+                                cudaStream_t s) {
+  if (experts <= kGroupExperts)
+    return launch_pdl(moe_group_runs_kernel, dim3(1), dim3(32 * kGroupWarps), (size_t)(kGroupWarps + 3) * experts * sizeof(int32_t), s, sel,
+                      pairs, experts, tile_rows, perm, meta, tiles);
+  return launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, sel, pairs, experts, tile_rows, perm,
+                    meta, tiles);
+}
+
 extern "C" int64_t prl_moe_max_tiles(int64_t pairs, int32_t experts) { return (pairs + kTile - 1) / kTile + experts; }
 
 extern "C" int prl_moe_route(const float* logits, int64_t ld, const float* bias, int32_t n, int32_t experts, int32_t top,
@@ -578,7 +672,7 @@ extern "C" int prl_moe_route(const float* logits, int64_t ld, const float* bias,
   cudaStream_t s = (cudaStream_t)st;
   PRL_CUDA(launch_pdl(moe_route_kernel, dim3((n + 7) / 8), dim3(256), (size_t)0, s, logits, ld, bias, n, experts, top, softmax_weights, sel, wsel));
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, kTile, perm, meta, tiles));
+  PRL_CUDA(launch_group(sel, n * top, experts, kTile, perm, meta, tiles, s));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -613,7 +707,7 @@ static int moe_router_impl(const void* x, int32_t x_is_f32, const void* Wr, int3
 #undef PRL_RT2
 #undef PRL_RT
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, tile_rows, perm, meta, tiles));
+  PRL_CUDA(launch_group(sel, n * top, experts, tile_rows, perm, meta, tiles, s));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
@@ -657,7 +751,7 @@ extern "C" int prl_moe_choose(const float* logits, int64_t ld, const float* corr
   PRL_CUDA(launch_pdl(moe_choose_kernel, dim3((n + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32),
                       (size_t)kChooseWarps * (outputs + groups) * sizeof(float), s, logits, ld, n, outputs, rule, sel, wsel));
   PRL_LAUNCH_CHECK();
-  PRL_CUDA(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)(2 * experts * sizeof(int32_t)), s, (const int32_t*)sel, n * top, experts, tile_rows, perm, meta, tiles));
+  PRL_CUDA(launch_group(sel, n * top, experts, tile_rows, perm, meta, tiles, s));
   PRL_LAUNCH_CHECK();
   return PRL_OK;
 }
