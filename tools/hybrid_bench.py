@@ -124,14 +124,14 @@ def futetar_config(s):
 def modadra_config(s):
     """Eight layers of windowed attention (heads of 128, 64 rotated channels, window 1024) beside the gated delta rule (heads
     of 128 x 128 on half as many q / k heads, four taps), as in the Kolotar model, every layer with routed experts of the
-    dense ff's active width (four of sixteen experts of ff / 4, three of four groups)."""
+    dense ff's active width (four of sixteen experts of ff / 4, six of eight groups)."""
     W, ff, H, G = s["width"], s["ff"], s["heads"], s["kv"]
-    routed = dict(kind="moe", router=dict(experts=16, top=4, scale=1.5, groups=dict(count=4, keep=3)), expert=dict(ff=ff // 4))
+    routed = dict(kind="moe", router=dict(experts=16, top=4, scale=1.25, groups=dict(count=8, keep=6)), expert=dict(ff=ff // 4))
     par = dict(type="parallel", mlp=routed,
                mixer=dict(left=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024),
                                     rot=dict(base=1e6, dims=64)),
                           right=dict(heads=W // 128, kv_heads=max(1, W // 256), dim=128, vdim=128, conv=4)))
-    return dict(architecture="Modadra", vocab=s["vocab"], width=W, norm=dict(eps=1e-5), residual_mult=0.5, logit_softcap=30.0,
+    return dict(architecture="Modadra", vocab=s["vocab"], width=W, norm=dict(eps=1e-5), residual_mult=0.5, logit_softcap=40.0,
                 layers=[par] * s["layers"])
 
 
